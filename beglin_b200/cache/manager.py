@@ -12,7 +12,7 @@ has one pool of pages (shared by its stages: page p of every stage of the group 
 request and the same positions) and one block table per request.  What a page holds is the need's
 business (`page_shape`): keys and values per kv head, or one latent row per position.  A group with a window gives back
 the pages that lie wholly behind the window as a request advances (one whose queries read their own block of positions
-only, the pages in front of the newest block).  A group of fixed state has one
+only, the pages in front of the newest block), except those with the first positions that its window keeps for good.  A group of fixed state has one
 slab [stages, slots, ...]; a request's slot is zeroed when the request starts.  A stage whose mixer is made of
 branches (attention beside a recurrence) hands in a composite need: each of its needs joins the group of its kind,
 and the stage's view is the tuple of the branches' views.
@@ -92,6 +92,10 @@ class _KVGroup:
         if self.need.block is not None:                # a query reads its own block of positions only
             lo = max(lo, first_query_pos - first_query_pos % self.need.block)
         return lo // page_size
+
+    def kept_pages(self, page_size: int) -> int:
+        """How many pages at a request's start are never given back (they hold the positions a window keeps for good)."""
+        return -(-getattr(self.need, "keep_first", 0) // page_size)
 
     @property
     def gives_back(self) -> bool:
@@ -252,7 +256,7 @@ class CacheManager:
         """(page indexes to give back, number of page indexes to add) for one group."""
         table = g.tables[rid]
         first = g.first_needed_page(first_query_pos, self.page_size)
-        drop = [i for i in range(min(first, len(table))) if table[i] >= 0] if first > 0 else ()
+        drop = [i for i in range(g.kept_pages(self.page_size), min(first, len(table))) if table[i] >= 0] if first > 0 else ()
         want_pages = -(-new_len // self.page_size)
         add = max(0, want_pages - len(table))
         return drop, add

@@ -19,6 +19,10 @@
 // enlarged by one, as if the row saw one more key of score 0 that carries no value: the merge starts its running
 // maximum at 0 and its sum at exp(0 - m), and nothing else changes.  With `sink_w` the extra key's score is a learned
 // number of the query head, sink_w[h], in place of 0.  With `softcap` c > 0 a score s is replaced by c tanh(s / c).
+//
+// With `slopes` [nh] the score of the key at position j falls by slopes[h] for every position that it lies behind the
+// query.  With `keep` k > 0 a window never loses the sequence's first k positions: a query at `pos` sees t <= pos with
+// t >= first_visible(pos, window) or t < k, the tiles and splits between the two ranges being passed over.
 #include "common.cuh"
 
 namespace bg {
@@ -47,6 +51,8 @@ struct AttnParams {
     int bq;                 // rows per query block (upper bound)
     float scale;
     float softcap;          // c > 0: scores pass c * tanh(s / c); 0: they stay as they are
+    int keep;               // positions 0 .. keep - 1 stay visible behind a window
+    const float* slopes;    // [nh] or null
     unsigned* status;
 };
 
@@ -75,9 +81,9 @@ attention_partial_kernel(AttnParams p) {
     const int pos_first = p.positions[row0];
     const int pos_last = p.positions[row0 + nq - 1];
     const int lo_first = first_visible(pos_first, p.window);
-    const int k_begin = max(sp * p.split, lo_first);
+    const int k_first = sp * p.split;
     const int k_end = min((sp + 1) * p.split, pos_last + 1);       // exclusive
-    if (k_begin >= k_end) return;
+    if (k_first >= k_end || (lo_first >= k_end && k_first >= p.keep)) return;      // no key of the split is seen
 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int n_rows = nq * group;
@@ -94,15 +100,15 @@ attention_partial_kernel(AttnParams p) {
     const size_t page_elems = (size_t)p.nkv * p.page_size * (hd + vd);
     const size_t v_off = (size_t)p.nkv * p.page_size * hd;
     const int tile = p.tile;
-    const int t_first = (k_begin / tile) * tile;
-
-    for (int t0 = t_first; t0 < k_end; t0 += tile) {
+    // (a split is a whole number of tiles)
+    for (int t0 = k_first; t0 < k_end; t0 += tile) {
+        if (t0 + tile <= lo_first && t0 >= p.keep) continue;       // wholly in front of every row's window
         __syncthreads();
-        // element offset of each key's K row in the pool, or -1 for a key outside [k_begin, k_end)
+        // element offset of each key's K row in the pool, or -1 for a key that no row of the block may see
         for (int j = tid; j < tile; j += ATT_THREADS) {
             int key = t0 + j;
             long long off = -1, voff = -1;
-            if (key >= k_begin && key < k_end) {
+            if (key < k_end && key_seen(key, lo_first, p.keep)) {
                 int page = p.block_table[(size_t)req * p.max_pages + key / p.page_size];
                 if (page < 0 || page >= p.num_pages) {
                     if (p.status) atomicOr(p.status, BG_STATUS_BAD_PAGE);
@@ -140,12 +146,13 @@ attention_partial_kernel(AttnParams p) {
                 int j = c * 32 + lane;
                 if (j < tile) {
                     int key = t0 + j;
-                    if (key >= lo && key <= pos && key >= k_begin && key < k_end && base_s[j] >= 0) {
+                    if (key_seen(key, lo, p.keep) && key <= pos && key < k_end && base_s[j] >= 0) {
                         const float* kr = k_s + j * kstride;
                         float dot = 0.0f;
                         for (int d = 0; d < hd; ++d) dot = fmaf(qr[d], kr[d], dot);
                         s[c] = dot * p.scale;
                         if (p.softcap > 0.0f) s[c] = p.softcap * tanhf(s[c] / p.softcap);
+                        if (p.slopes) s[c] -= p.slopes[kvh * group + r % group] * (float)(pos - key);
                     }
                 }
                 tmax = fmaxf(tmax, s[c]);
@@ -198,7 +205,7 @@ attention_partial_kernel(AttnParams p) {
         const int qi = r / group, g = r - qi * group;
         const int pos = p.positions[row0 + qi];
         const int lo = first_visible(pos, p.window);
-        if (pos < sp * p.split || lo >= (sp + 1) * p.split) continue;
+        if (pos < sp * p.split || (lo >= (sp + 1) * p.split && sp * p.split >= p.keep)) continue;
         const size_t prow = ((size_t)(row0 + qi) * p.nh + (size_t)kvh * group + g) * p.max_splits + sp;
         for (int d = lane; d < vd; d += 32) p.part_o[prow * vd + d] = acc_s[(size_t)r * vd + d];
         if (lane == 0) { p.part_ml[prow * 2 + 0] = m_s[r]; p.part_ml[prow * 2 + 1] = l_s[r]; }
@@ -215,7 +222,7 @@ template <typename TO, int DPL, int BATCH>
 __global__ void attention_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                        const int* __restrict__ positions, TO* __restrict__ out, int out_stride,
                                        int T, int nh, int hd, int max_splits, int split_arg, int window, int sink,
-                                       const float* __restrict__ sink_w) {
+                                       const float* __restrict__ sink_w, int keep) {
     pdl_launch();
     pdl_wait();
     const int w = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
@@ -225,20 +232,23 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_o, const f
     const int pos = positions[t];
     const int split = keys_per_split(split_arg, pos + 1, max_splits);
     const int lo = first_visible(pos, window);
-    const int s_lo = lo / split, s_hi = pos / split;
+    const int s_win = lo / split, s_hi = pos / split;
+    const int s_lo = keep > 0 ? 0 : s_win;
+    auto seen = [&](int s) { return s <= s_hi && (s >= s_win || s * split < keep); };     // splits that the row has results of
     const size_t prow = (size_t)w * max_splits;
     // the maxima and sums of the first 32 * MERGE_GROUPS splits of the row: lane j holds split s_lo + 32 g + j
     float ms_r[MERGE_GROUPS], ls_r[MERGE_GROUPS];
 #pragma unroll
     for (int g = 0; g < MERGE_GROUPS; ++g) {
         const int sidx = s_lo + 32 * g + lane;
-        const float2 ml = sidx <= s_hi ? *reinterpret_cast<const float2*>(part_ml + (prow + sidx) * 2) : make_float2(-INFINITY, 0.0f);
+        const float2 ml = seen(sidx) ? *reinterpret_cast<const float2*>(part_ml + (prow + sidx) * 2) : make_float2(-INFINITY, 0.0f);
         ms_r[g] = ml.x; ls_r[g] = ml.y;
     }
     float m = -INFINITY;
 #pragma unroll
     for (int g = 0; g < MERGE_GROUPS; ++g) m = fmaxf(m, ms_r[g]);
-    for (int sidx = s_lo + 32 * MERGE_GROUPS + lane; sidx <= s_hi; sidx += 32) m = fmaxf(m, part_ml[(prow + sidx) * 2]);
+    for (int sidx = s_lo + 32 * MERGE_GROUPS + lane; sidx <= s_hi; sidx += 32)
+        if (seen(sidx)) m = fmaxf(m, part_ml[(prow + sidx) * 2]);
     m = warp_max(m);
     const float sv = (sink && sink_w) ? sink_w[h] : 0.0f;      // the score of the key without a value
     if (sink) m = fmaxf(m, sv);
@@ -254,7 +264,7 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_o, const f
         if (grp < MERGE_GROUPS) {
 #pragma unroll
             for (int g = 0; g < MERGE_GROUPS; ++g) if (g == grp) { ms = ms_r[g]; l_mine = ls_r[g]; }
-        } else if (mine <= s_hi) {
+        } else if (seen(mine)) {
             ms = part_ml[(prow + mine) * 2];
             l_mine = part_ml[(prow + mine) * 2 + 1];
         }
@@ -269,7 +279,7 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_o, const f
 #pragma unroll
                 for (int i = 0; i < DPL; ++i) {
                     int d = i * 32 + lane;
-                    v[jj][i] = (j0 + jj < n && d < hd) ? po[d] : 0.0f;
+                    v[jj][i] = (j0 + jj < n && d < hd && seen(s0 + j0 + jj)) ? po[d] : 0.0f;
                 }
             }
 #pragma unroll
@@ -320,15 +330,17 @@ extern "C" int bg_attention_partial(const void* q, int q_dtype, int q_stride, co
                                     int num_pages, int page_size, const int* block_table, int max_pages,
                                     const int* positions, const int* qblk, int n_qblk, float* part_o, float* part_ml,
                                     int max_splits, int n_splits_launch, int nh, int nkv, int hd, int vd, int window, int split,
-                                    int tile, int bq, float scale, float softcap, unsigned* status, cudaStream_t stream) {
+                                    int tile, int bq, float scale, float softcap, int keep, const float* slopes, unsigned* status,
+                                    cudaStream_t stream) {
     if (n_qblk <= 0 || n_splits_launch <= 0) return BG_OK;
     if (nh % nkv != 0 || hd > 32 * ATT_MAX_DPL || vd <= 0 || vd > 32 * ATT_MAX_DPL || (tile != 32 && tile != 64) || split % tile != 0) return BG_ERR_SHAPE;
-    if (n_splits_launch > max_splits || n_splits_launch > 65535 || nkv > 65535) return BG_ERR_SHAPE;
+    if (n_splits_launch > max_splits || n_splits_launch > 65535 || nkv > 65535 || keep < 0) return BG_ERR_SHAPE;
     AttnParams p;
     p.q = q; p.q_stride = q_stride; p.kv_pool = kv_pool; p.num_pages = num_pages; p.page_size = page_size;
     p.block_table = block_table; p.max_pages = max_pages; p.positions = positions; p.qblk = qblk;
     p.part_o = part_o; p.part_ml = part_ml; p.max_splits = max_splits; p.nh = nh; p.nkv = nkv; p.hd = hd; p.vd = vd;
     p.group = nh / nkv; p.window = window; p.split = split; p.tile = tile; p.bq = bq; p.scale = scale; p.softcap = softcap; p.status = status;
+    p.keep = keep; p.slopes = slopes;
     size_t smem = attention_smem_bytes(bq, p.group, hd, vd, tile);
     if (smem > 227 * 1024) return BG_ERR_UNSUPPORTED;
     dim3 grid(n_qblk, nkv, n_splits_launch);
@@ -357,7 +369,7 @@ template <typename TO, int NS>
 __global__ void attention_merge_few_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                            const int* __restrict__ positions, TO* __restrict__ out, int out_stride,
                                            int T, int nh, int hd, int max_splits, int split_arg, int window, int sink,
-                                       const float* __restrict__ sink_w) {
+                                           const float* __restrict__ sink_w, int keep) {
     pdl_launch();
     const int w = (blockIdx.x * blockDim.x + threadIdx.x) >> 5;
     const int lane = threadIdx.x & 31;
@@ -388,7 +400,7 @@ __global__ void attention_merge_few_kernel(const float* __restrict__ part_o, con
     float m = sink ? sv : -INFINITY;
 #pragma unroll
     for (int s = 0; s < NS; ++s) {
-        if (s < s_lo || s > s_hi) ms[s] = -INFINITY;          // not written for this row: whatever was read is dropped
+        if ((s < s_lo && s * split >= keep) || s > s_hi) ms[s] = -INFINITY;          // not written for this row: whatever was read is dropped
         m = fmaxf(m, ms[s]);
     }
     float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f}, l = sink ? expf(sv - m) : 0.0f;
@@ -423,7 +435,7 @@ __global__ void __launch_bounds__(32 * MERGE_WARPS)
 attention_merge_block_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                              const int* __restrict__ positions, TO* __restrict__ out, int out_stride,
                              int T, int nh, int hd, int max_splits, int split_arg, int window, int sink,
-                                       const float* __restrict__ sink_w) {
+                             const float* __restrict__ sink_w, int keep) {
     __shared__ float4 acc_s[MERGE_WARPS][32];
     __shared__ float2 ml_s[MERGE_WARPS];
     pdl_launch();
@@ -434,7 +446,8 @@ attention_merge_block_kernel(const float* __restrict__ part_o, const float* __re
     const int pos = positions[t];
     const int split = keys_per_split(split_arg, pos + 1, max_splits);
     const int lo = first_visible(pos, window);
-    const int s_lo = lo / split, s_hi = pos / split;
+    const int s_win = lo / split, s_hi = pos / split;
+    const int s_lo = keep > 0 ? 0 : s_win;
     pdl_wait();
     const size_t prow = (size_t)w * max_splits;
     const int d = lane * 4;
@@ -447,7 +460,7 @@ attention_merge_block_kernel(const float* __restrict__ part_o, const float* __re
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
             const int sidx = g * 8 + j;
-            const bool have = sidx >= s_lo && sidx <= s_hi;
+            const bool have = sidx <= s_hi && (sidx >= s_win || sidx * split < keep);
             const float2 ml = have ? *reinterpret_cast<const float2*>(part_ml + (prow + sidx) * 2) : make_float2(-INFINITY, 0.0f);
             ms[j] = ml.x; ls[j] = ml.y;
             v[j] = (have && live) ? *reinterpret_cast<const float4*>(part_o + (prow + sidx) * hd + d)
@@ -504,7 +517,7 @@ attention_merge_block_kernel(const float* __restrict__ part_o, const float* __re
 
 extern "C" int bg_attention_merge(const float* part_o, const float* part_ml, const int* positions, void* out,
                                   int out_dtype, int out_stride, int T, int nh, int hd, int max_splits, int split,
-                                  int window, int sink, const float* sink_w, cudaStream_t stream) {
+                                  int window, int sink, const float* sink_w, int keep, cudaStream_t stream) {
     if (T <= 0) return BG_OK;
     long long warps = (long long)T * nh;
     unsigned blocks = (unsigned)((warps * 32 + 255) / 256);
@@ -519,24 +532,24 @@ extern "C" int bg_attention_merge(const float* part_o, const float* part_ml, con
         // 5 us this way; the decode step of the 1.5B sizes went from 1.372 to 1.214 ms at batch 1, from 1.225 to
         // 1.151 ms at batch 2)
         launch(attention_merge_block_kernel<__nv_bfloat16>, dim3((unsigned)warps), dim3(32 * MERGE_WARPS), 0, stream,
-               part_o, part_ml, positions, (__nv_bfloat16*)out, out_stride, T, nh, hd, max_splits, split, window, sink, sink_w);
+               part_o, part_ml, positions, (__nv_bfloat16*)out, out_stride, T, nh, hd, max_splits, split, window, sink, sink_w, keep);
     } else if (max_splits <= 8 && hd <= 128) {
         BG_DISPATCH_DTYPE(out_dtype, TO, launch(attention_merge_few_kernel<TO, 8>, dim3(few_blocks), dim3(few_threads), 0, stream,
-            part_o, part_ml, positions, (TO*)out, out_stride, T, nh, hd, max_splits, split, window, sink, sink_w));
+            part_o, part_ml, positions, (TO*)out, out_stride, T, nh, hd, max_splits, split, window, sink, sink_w, keep));
     } else if (max_splits <= 16 && hd <= 128) {
         BG_DISPATCH_DTYPE(out_dtype, TO, launch(attention_merge_few_kernel<TO, 16>, dim3(few_blocks), dim3(few_threads), 0, stream,
-            part_o, part_ml, positions, (TO*)out, out_stride, T, nh, hd, max_splits, split, window, sink, sink_w));
+            part_o, part_ml, positions, (TO*)out, out_stride, T, nh, hd, max_splits, split, window, sink, sink_w, keep));
     } else if (block_fits) {
         // bfloat16 rows of few requests with many splits each (the float path keeps one order of summation for
         // every shape of a step, so that its rows do not depend on the batch)
         launch(attention_merge_block_kernel<__nv_bfloat16>, dim3((unsigned)warps), dim3(32 * MERGE_WARPS), 0, stream,
-               part_o, part_ml, positions, (__nv_bfloat16*)out, out_stride, T, nh, hd, max_splits, split, window, sink, sink_w);
+               part_o, part_ml, positions, (__nv_bfloat16*)out, out_stride, T, nh, hd, max_splits, split, window, sink, sink_w, keep);
     } else if (hd <= 128) {
         BG_DISPATCH_DTYPE(out_dtype, TO, launch(attention_merge_kernel<TO, 4, 16>, dim3(blocks), dim3(256), 0, stream,
-            part_o, part_ml, positions, (TO*)out, out_stride, T, nh, hd, max_splits, split, window, sink, sink_w));
+            part_o, part_ml, positions, (TO*)out, out_stride, T, nh, hd, max_splits, split, window, sink, sink_w, keep));
     } else {
         BG_DISPATCH_DTYPE(out_dtype, TO, launch(attention_merge_kernel<TO, ATT_MAX_DPL, 4>, dim3(blocks), dim3(256), 0, stream,
-            part_o, part_ml, positions, (TO*)out, out_stride, T, nh, hd, max_splits, split, window, sink, sink_w));
+            part_o, part_ml, positions, (TO*)out, out_stride, T, nh, hd, max_splits, split, window, sink, sink_w, keep));
     }
     BG_LAUNCH_CHECK();
     return BG_OK;

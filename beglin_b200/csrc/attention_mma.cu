@@ -25,6 +25,10 @@
 //          the instruction and the heads the N side of 8, S^T = K Q^T and O^T = V^T P^T, which halves
 //          the MMAs of a stage (the heads fill 6 of 8 columns instead of 6 of 16 rows); P^T reaches its
 //          operand layout through movmatrix.
+//
+// EXT instances: a score falls by slopes[head] per position that its key lies back, and a window never loses the sequence's
+// first `keep` positions.  The stages of a CTA are then those of its kept keys followed by those of its window's, the
+// stages between the two passed over.
 #include "page_tma.cuh"
 
 namespace bg {
@@ -60,6 +64,8 @@ struct AttnMmaParams {
     int out_stride;         // the finished rows here (no partial results, no merge)
     int use_tma;            // pages are copied as TMA boxes (the page size divides 64)
     int whole_pages;        // a page is a stage (64 positions): keys and values of a stage come in ONE box
+    int keep;               // EXT: positions 0 .. keep - 1 stay visible behind a window
+    const float* slopes;    // EXT: [nh] or null
 };
 
 // A product q . k as the exponent of two that the softmax takes: scaled, squashed when the layer asks for it.
@@ -113,7 +119,7 @@ __device__ __forceinline__ int swz_kv(int row, int c) {
     return (c >> 3) * (AM_STAGE_KEYS * 128) + row * 128 + (((c & 7) ^ (row & 7)) << 4);
 }
 
-template <int HD, bool BY_KEYS, int AM_STAGES, bool SWAP>
+template <int HD, bool BY_KEYS, int AM_STAGES, bool SWAP, bool EXT>
 __global__ void __launch_bounds__(AM_ALL)
 attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_constant__ CUtensorMap map_page, AttnMmaParams p) {
     constexpr int CH = HD / 8;                 // 16-byte columns per row
@@ -181,13 +187,23 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
     }
 
     const int lo_first = first_visible(pos_first, p.window);
-    const int k_begin = direct ? lo_first : max(sp * split, lo_first);
+    const int k_first = direct ? 0 : sp * split;                  // this CTA's range of positions: [k_first, k_end)
+    const int k_begin = max(k_first, lo_first);                   // of which the window's keys are [k_begin, k_end)
     const int k_end = direct ? pos_last + 1 : min((sp + 1) * split, pos_last + 1);
-    if (k_begin >= k_end) return;
+    const int keep = EXT ? p.keep : 0;
+    const int kept_end = min(keep, k_end);                        // and the kept ones [k_first, kept_end), possibly none
+    const bool has_kept = EXT && k_first < kept_end;
+    if (k_begin >= k_end && !has_kept) return;
+    auto in_range = [&](int key) { return key < k_end && (key >= k_begin || (EXT && key >= k_first && key < kept_end)); };
 
     // ---- stage loader: thread t copies 16-byte pieces of key rows of K and of V
-    const int first_stage_key = (k_begin / AM_STAGE_KEYS) * AM_STAGE_KEYS;
-    const int n_stage = (k_end - first_stage_key + AM_STAGE_KEYS - 1) / AM_STAGE_KEYS;
+    const int first_stage_key = ((has_kept ? k_first : k_begin) / AM_STAGE_KEYS) * AM_STAGE_KEYS;
+    // the stages of the kept keys, then those of the window's keys, `skip` positions further on
+    const int n_kept = has_kept ? (kept_end - first_stage_key + AM_STAGE_KEYS - 1) / AM_STAGE_KEYS : 0;
+    const int kept_stop = first_stage_key + n_kept * AM_STAGE_KEYS;
+    const int skip = has_kept ? max((k_begin / AM_STAGE_KEYS) * AM_STAGE_KEYS - kept_stop, 0) : 0;
+    const int n_stage = n_kept + max((k_end - kept_stop - skip + AM_STAGE_KEYS - 1) / AM_STAGE_KEYS, 0);
+    auto stage_key = [&](int s) { return first_stage_key + s * AM_STAGE_KEYS + (EXT && s >= n_kept ? skip : 0); };
     const int last_page = (k_end - 1) / p.page_size;
     int table_group = (first_stage_key / p.page_size) / AM_TABLE;
     if (table_group != pre_group) table_group = -1;               // a window moved the range: fetched by the loader
@@ -209,8 +225,9 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
         const int n_box = (AM_STAGE_KEYS >> shift) * PER_PAGE;
         const int* table = p.block_table + (size_t)req * p.max_pages;
         auto page_of = [&](int s, int o) {               // the page that box o of stage s comes from, or -1
-            const int key_lo = first_stage_key + s * AM_STAGE_KEYS + (o / PER_PAGE) * ps;
-            if (s >= n_stage || o >= n_box || key_lo >= k_end || key_lo + ps <= k_begin || (key_lo >> shift) >= p.max_pages) return -1;
+            const int key_lo = stage_key(s) + (o / PER_PAGE) * ps;
+            if (s >= n_stage || o >= n_box || key_lo >= k_end || (key_lo >> shift) >= p.max_pages) return -1;
+            if (key_lo + ps <= k_begin && !(has_kept && key_lo < kept_end && key_lo + ps > k_first)) return -1;
             return table[key_lo >> shift];
         };
         // stages of old keys only may be asked for before the kernel ahead has finished: all but the one that
@@ -262,7 +279,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
     auto load_stage = [&](int s) {
         if (p.use_tma) return;                                   // the copying warp's job
         if (s < n_stage) {
-            const int stage_key0 = first_stage_key + s * AM_STAGE_KEYS;
+            const int stage_key0 = stage_key(s);
             const int group_of_stage = (stage_key0 / p.page_size) / AM_TABLE;
             if (group_of_stage != table_group) {                 // uniform over the computing warps
                 compute_sync();
@@ -283,7 +300,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
             for (int j = tid / CH; j < AM_STAGE_KEYS; j += ROWS_PER_PASS) {
                 const int key = stage_key0 + j;
                 const __nv_bfloat16* src = nullptr;
-                if (key >= k_begin && key < k_end) {
+                if (in_range(key)) {
                     const int pi = p.page_shift >= 0 ? key >> p.page_shift : key / p.page_size;
                     const int slot = p.page_shift >= 0 ? key & (p.page_size - 1) : key - pi * p.page_size;
                     const int page = table_s[pi - table_group * AM_TABLE];
@@ -327,6 +344,15 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
             lo_r[h] = first_visible(pos_r[h], p.window);
         } else {
             pos_r[h] = -1; lo_r[h] = 0;
+        }
+    }
+    // what the scores of this thread's two rows (or two heads) fall by per position, in powers of two
+    float slope_l2[2] = {0.0f, 0.0f};
+    if (EXT && p.slopes) {
+#pragma unroll
+        for (int h = 0; h < 2; ++h) {
+            const int r = SWAP ? 2 * (lane & 3) + h : row_base + (lane >> 2) + h * 8;
+            if (r < n_rows) slope_l2[h] = p.slopes[kvh * group + r % group] * AM_LOG2E;
         }
     }
     // the span of keys that the rows of this warp can see at all, and the span that ALL its rows see
@@ -376,19 +402,21 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
         const int buf = s % AM_STAGES;
         unsigned char* kt = k_s + buf * BUF_BYTES;
         unsigned char* vt = v_s + buf * BUF_BYTES;
-        const int stage_key0 = first_stage_key + s * AM_STAGE_KEYS;
+        const int stage_key0 = stage_key(s);
         // who reads this stage: the warp alone (keys arrangement) or the four warps together
         const int t0 = BY_KEYS ? lane : tid, nt = BY_KEYS ? 32 : AM_THREADS;
         if (p.use_tma) {
             // A wait that runs out records it and goes on (with whatever the buffer holds; the host raises on
             // the status): every thread then still reaches the barriers below.
             if (!mbar_wait<4000>(&full_bar[buf], (s / AM_STAGES) & 1, &gave_up) && p.status) atomicOr(p.status, BG_STATUS_TIMEOUT);
-            if (stage_key0 < k_begin || stage_key0 + AM_STAGE_KEYS > k_end) {      // uniform over the readers
+            const bool whole_stage = stage_key0 + AM_STAGE_KEYS <= k_end &&
+                (stage_key0 >= k_begin || (has_kept && stage_key0 >= k_first && stage_key0 + AM_STAGE_KEYS <= kept_end));
+            if (!whole_stage) {                                                    // uniform over the readers
                 // whole pages were copied: rows outside the range of keys become zeros (a value row that no
                 // query sees must not hold garbage, since 0 * NaN is NaN)
                 for (int idx = t0; idx < AM_STAGE_KEYS * CH; idx += nt) {
                     const int j = idx / CH, c = idx - j * CH;
-                    if (stage_key0 + j < k_begin || stage_key0 + j >= k_end) {
+                    if (!in_range(stage_key0 + j)) {
                         *reinterpret_cast<uint4*>(kt + swz_kv(j, c)) = make_uint4(0, 0, 0, 0);
                         *reinterpret_cast<uint4*>(vt + swz_kv(j, c)) = make_uint4(0, 0, 0, 0);
                     }
@@ -401,7 +429,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
             for (int idx = lane; idx < AM_STAGE_KEYS * CH; idx += 32) {
                 const int j = idx / CH, c = idx - j * CH, key = stage_key0 + j;
                 const __nv_bfloat16* src = nullptr;
-                if (key >= k_begin && key < k_end) {
+                if (in_range(key)) {
                     const int pi = key / p.page_size, slot = key - pi * p.page_size;
                     const int page = pi < p.max_pages ? p.block_table[(size_t)req * p.max_pages + pi] : -1;
                     if (page < 0 || page >= p.num_pages) {
@@ -429,7 +457,8 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
         const int w_key0 = stage_key0;
         const int vis_lo = max(max(w_key0, k_begin), warp_lo);                   // keys some row of the warp sees
         const int vis_hi = min(min(w_key0 + 16 * KB, k_end), warp_pos_hi + 1);
-        if (SWAP && vis_lo < vis_hi) {
+        const bool kept_here = has_kept && w_key0 < kept_end && w_key0 <= warp_pos_hi;     // (kept keys of the stage that a row sees)
+        if (SWAP && (vis_lo < vis_hi || kept_here)) {
             // ---- S^T = K Q^T: per block of 16 keys a 16 x 8 tile; c[kb][e]: key kb * 16 + lane / 4 + 8 (e >> 1), head r0 + (e & 1)
             float c[KB][4];
 #pragma unroll
@@ -452,8 +481,9 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int key = w_key0 + kb * 16 + (lane >> 2) + 8 * (e >> 1);
-                    const bool ok = all_seen || (key <= pos && key >= lo && key >= k_begin && key < k_end);
-                    const float v = (ok && r0 + (e & 1) < n_rows) ? am_score(c[kb][e], p) : -INFINITY;
+                    const bool ok = all_seen || (key <= pos && key_seen(key, lo, keep) && in_range(key));
+                    float v = (ok && r0 + (e & 1) < n_rows) ? am_score(c[kb][e], p) : -INFINITY;
+                    if (EXT) v = fmaf(slope_l2[e & 1], (float)(key - pos), v);
                     c[kb][e] = v;
                     tmax[e & 1] = fmaxf(tmax[e & 1], v);
                 }
@@ -499,7 +529,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
                 }
             }
         }
-        if (!SWAP && vis_lo < vis_hi) {                                          // warp-uniform
+        if (!SWAP && (vis_lo < vis_hi || kept_here)) {                           // warp-uniform
             // ---- scores of 16 rows x 16*KB keys
             // (k-step outermost, so the 2*KB accumulators form independent chains of dependent MMAs)
             float sc[2 * KB][4];
@@ -526,6 +556,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
 #pragma unroll
                     for (int e = 0; e < 4; ++e) {
                         sc[j][e] = am_score(sc[j][e], p);
+                        if (EXT) sc[j][e] = fmaf(slope_l2[e >> 1], (float)(w_key0 + j * 8 + (lane & 3) * 2 + (e & 1) - pos_r[e >> 1]), sc[j][e]);
                         tmax[e >> 1] = fmaxf(tmax[e >> 1], sc[j][e]);
                     }
             } else {
@@ -535,8 +566,9 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
                     for (int e = 0; e < 4; ++e) {
                         const int key = w_key0 + j * 8 + (lane & 3) * 2 + (e & 1);
                         const int h = e >> 1;
-                        const bool ok = key <= pos_r[h] && key >= lo_r[h] && key >= k_begin && key < k_end;
-                        const float v = ok ? am_score(sc[j][e], p) : -INFINITY;
+                        const bool ok = key <= pos_r[h] && key_seen(key, lo_r[h], keep) && in_range(key);
+                        float v = ok ? am_score(sc[j][e], p) : -INFINITY;
+                        if (EXT) v = fmaf(slope_l2[h], (float)(key - pos_r[h]), v);
                         sc[j][e] = v;
                         tmax[h] = fmaxf(tmax[h], v);
                     }
@@ -617,7 +649,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
         for (int h = 0; h < 2; ++h) {
             int r = row_base + (lane >> 2) + h * 8;
             if (r >= n_rows) continue;
-            if (pos_r[h] < sp * split || lo_r[h] >= (sp + 1) * split) continue;
+            if (pos_r[h] < sp * split || (lo_r[h] >= (sp + 1) * split && sp * split >= keep)) continue;
             int qi = r / group, g = r - qi * group;
             size_t prow = ((size_t)(row0 + qi) * p.nh + (size_t)kvh * group + g) * p.max_splits + sp;
             float* po = p.part_o + prow * HD;
@@ -661,7 +693,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
         compute_sync();
         const int pos = pos_first;
         const int lo = first_visible(pos, p.window);
-        if (!(pos < sp * split || lo >= (sp + 1) * split)) {
+        if (!(pos < sp * split || (lo >= (sp + 1) * split && sp * split >= keep))) {
             // every thread takes one feature of all rows and works out the weights of the four warps' parts itself
             // (four exponentials a row: cheaper than a third barrier and a round through shared memory)
             if (tid < HD) {
@@ -696,9 +728,9 @@ static size_t am_smem_bytes() {
     return (size_t)(BY_KEYS ? 16 : 64) * HD * 2 + (size_t)2 * STAGES * AM_STAGE_KEYS * HD * 2 + 1024;
 }
 
-template <int HD, bool BY_KEYS, int STAGES, bool SWAP = false>
+template <int HD, bool BY_KEYS, int STAGES, bool SWAP, bool EXT>
 static int am_launch_stages(const CUtensorMap& map, const CUtensorMap& map5, const AttnMmaParams& p, int n_qblk, int n_splits, cudaStream_t stream) {
-    auto kern = attention_mma_kernel<HD, BY_KEYS, STAGES, SWAP>;
+    auto kern = attention_mma_kernel<HD, BY_KEYS, STAGES, SWAP, EXT>;
     size_t smem = am_smem_bytes<HD, BY_KEYS, STAGES>();
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
@@ -708,11 +740,16 @@ static int am_launch_stages(const CUtensorMap& map, const CUtensorMap& map5, con
     return BG_OK;
 }
 
+template <int HD, bool BY_KEYS, bool EXT>
+static int am_launch_as(const CUtensorMap& map, const CUtensorMap& map5, const AttnMmaParams& p, int n_qblk, int n_splits, cudaStream_t stream) {
+    if (BY_KEYS && p.group <= 8) return am_launch_stages<HD, BY_KEYS, AM_THREADS / 32, BY_KEYS, EXT>(map, map5, p, n_qblk, n_splits, stream);
+    if (BY_KEYS) return am_launch_stages<HD, BY_KEYS, AM_THREADS / 32, false, EXT>(map, map5, p, n_qblk, n_splits, stream);   // a buffer per warp
+    return am_launch_stages<HD, BY_KEYS, 3, false, EXT>(map, map5, p, n_qblk, n_splits, stream);
+}
 template <int HD, bool BY_KEYS>
 static int am_launch(const CUtensorMap& map, const CUtensorMap& map5, const AttnMmaParams& p, int n_qblk, int n_splits, cudaStream_t stream) {
-    if (BY_KEYS && p.group <= 8) return am_launch_stages<HD, BY_KEYS, AM_THREADS / 32, BY_KEYS>(map, map5, p, n_qblk, n_splits, stream);
-    if (BY_KEYS) return am_launch_stages<HD, BY_KEYS, AM_THREADS / 32>(map, map5, p, n_qblk, n_splits, stream);   // a buffer per warp
-    return am_launch_stages<HD, BY_KEYS, 3>(map, map5, p, n_qblk, n_splits, stream);
+    if (p.keep > 0 || p.slopes) return am_launch_as<HD, BY_KEYS, true>(map, map5, p, n_qblk, n_splits, stream);
+    return am_launch_as<HD, BY_KEYS, false>(map, map5, p, n_qblk, n_splits, stream);
 }
 
 }  // namespace bg
@@ -737,7 +774,8 @@ extern "C" int bg_attention_mma_partial(const void* q, int q_stride, const void*
                                         const int* block_table, int max_pages, const int* positions, const int* qblk,
                                         int n_qblk, float* part_o, float* part_ml, int max_splits, int n_splits_launch,
                                         int nh, int nkv, int hd, int window, int split, int by_keys, float scale,
-                                        float softcap, void* direct_out, int out_stride, unsigned* status, cudaStream_t stream) {
+                                        float softcap, void* direct_out, int out_stride, int keep, const float* slopes,
+                                        unsigned* status, cudaStream_t stream) {
     if (n_qblk <= 0 || n_splits_launch <= 0) return BG_OK;
     if (direct_out && (n_splits_launch != 1 || (out_stride % 2) != 0)) return BG_ERR_SHAPE;
     if (nh % nkv != 0 || split % AM_STAGE_KEYS != 0 || (split <= 0 && !by_keys)) return BG_ERR_SHAPE;
@@ -753,6 +791,8 @@ extern "C" int bg_attention_mma_partial(const void* q, int q_stride, const void*
     p.scale_log2 = scale * AM_LOG2E; p.status = status;
     p.cap_log2 = softcap > 0.0f ? softcap * AM_LOG2E : 0.0f; p.scale_over_cap = softcap > 0.0f ? scale / softcap : 0.0f;
     p.out = (__nv_bfloat16*)direct_out; p.out_stride = out_stride;
+    if (keep < 0) return BG_ERR_SHAPE;
+    p.keep = keep; p.slopes = slopes;
     if (by_keys ? p.group > 16 : p.group > 64) return BG_ERR_UNSUPPORTED;
     if (hd != 64 && hd != 128) return BG_ERR_UNSUPPORTED;
     CUtensorMap map;

@@ -61,6 +61,8 @@ struct AttnTcParams {
     float cap_log2;             // c * log2(e) when scores are squashed to c tanh(score / c), else 0
     float cap_k;                // 2 * log2(e) * scale / c
     const float* sink_weight;   // [nh] the sink's score head by head (null: 0), where the denominator is enlarged
+    int keep;                   // EXT: positions 0 .. keep - 1 stay visible behind a window
+    const float* slopes;        // EXT: [nh] what a score falls by per position that its key lies back, or null
     unsigned* status;
 };
 
@@ -85,7 +87,9 @@ __device__ __forceinline__ float at_squash(float x, float cap_log2, float cap_k)
 
 // SINK: the softmax's denominator is enlarged by one (a key of score 0 without a value): the final join takes 0 into the
 // maximum and exp2(0 - maximum) into the sum; nothing else differs, and the plain instance is compiled as before.
-template <int HD, int AT_BK, bool SINK = false>
+// EXT: scores fall with the distance by a slope of the head, and a window never loses the first `keep` positions: the
+// tiles are then those of the kept positions followed by those of the window, the tiles between passed over.
+template <int HD, int AT_BK, bool SINK = false, bool EXT = false>
 __global__ void __launch_bounds__(AT_THREADS)
 attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParams p) {
     constexpr int AT_HALF = AT_BK / 2, AT_STAGES = 256 / AT_BK;
@@ -148,8 +152,11 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
     const int pos_last = pos_first + nq - 1;
     const int k_begin = first_visible(pos_first, p.window);
     const int k_end = pos_last + 1;
-    const int tile0 = k_begin / AT_BK;
-    const int n_tiles = (k_end + AT_BK - 1) / AT_BK - tile0;
+    const int keep = EXT ? p.keep : 0;
+    const int n_kept = EXT ? (min(keep, k_end) + AT_BK - 1) / AT_BK : 0;         // tiles with kept positions
+    const int tile0 = max(k_begin / AT_BK, n_kept);                              // the window's first tile behind those
+    const int n_tiles = n_kept + max((k_end + AT_BK - 1) / AT_BK - tile0, 0);
+    auto tile_key = [&](int i) { return (EXT && i < n_kept ? i : tile0 + i - n_kept) * AT_BK; };
 
     // ---- Q into shared memory: row r, column block cb, 16-byte piece c at r*128 + ((c ^ (r & 7)) * 16)
     for (int idx = tid; idx < AT_BM * (HD / 8); idx += AT_THREADS) {
@@ -270,12 +277,13 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
         float m = -INFINITY, l = 0.0f;
         bool ok = true;
         const bool capped = p.cap_log2 > 0.0f;
-        const float sl2 = capped ? 1.0f : p.scale_log2;
+        const float sl2 = (capped || EXT) ? 1.0f : p.scale_log2;
+        const float slope_l2 = (EXT && p.slopes && real) ? p.slopes[kvh * group + r % group] * AT_LOG2E : 0.0f;
         const int i_first = ALT ? grp : 0;                   // this group's first tile
         for (int i = i_first; i < n_tiles && ok; i += (ALT ? 2 : 1)) {
             const int b = i % NSB;
             const unsigned s_col = (unsigned)b * AT_BK + (ALT ? 0u : (unsigned)grp * AT_HALF);    // this group's scores of the tile, and its P
-            const int key0 = (tile0 + i) * AT_BK + (ALT ? 0 : grp * AT_HALF);
+            const int key0 = tile_key(i) + (ALT ? 0 : grp * AT_HALF);
             ok = mbar_wait(&s_full[b], (i / NSB) & 1);
             if (!ok) break;
             tc_fence_after();
@@ -286,13 +294,18 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
 #pragma unroll
                 for (int q = 0; q < GK; ++q) s[q] = at_squash(s[q], p.cap_log2, p.cap_k);
             }
+            if constexpr (EXT) {                         // exponents of two, less the head's slope times the distance
+                const float at0 = slope_l2 * (float)(key0 - pos), unit = capped ? 1.0f : p.scale_log2;
+#pragma unroll
+                for (int q = 0; q < GK; ++q) s[q] = fmaf(s[q], unit, fmaf(slope_l2, (float)q, at0));
+            }
             // only a half that some row of the warp sees in part is masked element by element
             float tm[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
-            if (key0 + GK - 1 > warp_pos_min || key0 < warp_lo_max) {
+            if (key0 + GK - 1 > warp_pos_min || (key0 < warp_lo_max && !(EXT && key0 + GK <= keep))) {
 #pragma unroll
                 for (int q = 0; q < GK; ++q) {
                     const int key = key0 + q;
-                    s[q] = (key <= pos && key >= lo) ? s[q] : -INFINITY;
+                    s[q] = (key <= pos && key_seen(key, lo, keep)) ? s[q] : -INFINITY;
                     tm[q & 3] = fmaxf(tm[q & 3], s[q]);
                 }
             } else {
@@ -393,13 +406,13 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
         unsigned landed_phase = 0;                       // bit s: parity of stage s's "landed" barrier
         constexpr int ROUNDS = AT_BK / 32;               // a lane holds the page of up to ROUNDS of a tile's pages (pages of one key)
         auto fetch_pages = [&](int i, int (&pg)[ROUNDS]) {
-            const int key0 = (tile0 + i) * AT_BK;
+            const int key0 = tile_key(i);
 #pragma unroll
             for (int h = 0; h < ROUNDS; ++h) {
                 const int k = h * 32 + lane;
                 const int pi = (key0 >> sh) + k;
                 pg[h] = -1;
-                if (i < n_tiles && k < n_pg && pi < p.max_pages && key0 + k * ps < k_end && key0 + (k + 1) * ps > k_begin)
+                if (i < n_tiles && k < n_pg && pi < p.max_pages && key0 + k * ps < k_end && (key0 + (k + 1) * ps > k_begin || key0 + k * ps < keep))
                     pg[h] = p.block_table[(size_t)req * p.max_pages + pi];
             }
         };
@@ -411,7 +424,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
                 ok = mbar_wait(&empty[st], ((i / AT_STAGES) - 1) & 1);
                 if (!ok) break;
             }
-            const int key0 = (tile0 + i) * AT_BK;
+            const int key0 = tile_key(i);
             unsigned char* dst = ring + st * KV_BYTES;
             // page numbers of the tile (fetched one tile ahead): lanes 0..n_pg-1 hold one each, in rounds of 32
             int pg[ROUNDS];
@@ -429,7 +442,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
             // Key rows that no query may see need no care (their scores are masked, whatever they are); value rows
             // do: 0 * garbage can be NaN.  So a ragged tile of values lands on a barrier of its own, the rows
             // outside the range or in pages that are not held are zeroed, and only then is the tile released.
-            const bool direct = !which || (n_have == n_pg && key0 >= k_begin && key0 + AT_BK <= k_end);
+            const bool direct = !which || (n_have == n_pg && (key0 >= k_begin || key0 + AT_BK <= keep) && key0 + AT_BK <= k_end);
             unsigned long long* bar = direct ? &full[st] : &kv_landed[st];
             if (lane == 0) {
                 if (n_have > 0) mbar_expect_tx(bar, (unsigned)n_have * ps * HD * 2);
@@ -458,7 +471,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
 #pragma unroll
                     for (int h = 1; h < ROUNDS; ++h) mask = (k >> 5) == h ? have[h] : mask;
                     const int held = (mask >> (k & 31)) & 1;
-                    if (!held || key < k_begin || key >= k_end)
+                    if (!held || !key_seen(key, k_begin, keep) || key >= k_end)
                         *reinterpret_cast<uint4*>(dst + (c >> 3) * KV_BLOCK + jrow * 128 + (((c & 7) ^ (jrow & 7)) << 4)) = make_uint4(0, 0, 0, 0);
                 }
                 fence_proxy_async();
@@ -477,9 +490,9 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
     if (tid == 0 && failed && p.status) atomicOr(p.status, BG_STATUS_TIMEOUT);
 }
 
-template <int HD, int BK, bool SINK = false>
+template <int HD, int BK, bool SINK = false, bool EXT = false>
 static int at_launch(const CUtensorMap& map, const AttnTcParams& p, int n_qblk, cudaStream_t stream) {
-    auto kern = attention_tcgen05_kernel<HD, BK, SINK>;
+    auto kern = attention_tcgen05_kernel<HD, BK, SINK, EXT>;
     // Q, and two rings (keys, values) of 256 keys each
     const size_t smem = (size_t)(HD / 64) * AT_BM * 128 + (size_t)2 * 256 * (HD / 64) * 128 + 1024;
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
@@ -511,7 +524,8 @@ extern "C" int bg_attention_tc_plan(int group, int hd, int page_size, int* bq_ou
 static int attention_tc(const void* q, int q_stride, const void* kv_pool, int num_pages, int page_size,
                         const int* block_table, int max_pages, const int* positions, const int* qblk, int n_qblk,
                         void* out, int out_stride, int nh, int nkv, int hd, int window, float scale, int max_position,
-                        bool sink, unsigned* status, cudaStream_t stream, const float* sink_weight = nullptr, float softcap = 0.0f) {
+                        bool sink, unsigned* status, cudaStream_t stream, const float* sink_weight = nullptr, float softcap = 0.0f,
+                        int keep = 0, const float* slopes = nullptr) {
     if (n_qblk <= 0) return BG_OK;
     if ((sink_weight && !sink) || softcap < 0.0f) return BG_ERR_SHAPE;
     if (nh % nkv != 0 || (hd != 64 && hd != 128) || nh / nkv > 128 || !(scale > 0.0f)) return BG_ERR_UNSUPPORTED;
@@ -527,12 +541,20 @@ static int attention_tc(const void* q, int q_stride, const void* kv_pool, int nu
     p.window = window; p.scale_log2 = scale * AT_LOG2E; p.status = status;
     p.cap_log2 = softcap > 0.0f ? softcap * AT_LOG2E : 0.0f; p.cap_k = softcap > 0.0f ? 2.0f * AT_LOG2E * scale / softcap : 0.0f;
     p.sink_weight = sink_weight;
+    const bool ext = keep > 0 || slopes != nullptr;
+    if (keep < 0) return BG_ERR_SHAPE;
+    if (ext && sink) return BG_ERR_UNSUPPORTED;              // (no instance with both)
+    p.keep = keep; p.slopes = slopes;
     CUtensorMap map;
     int rc = pt_pool_map(&map, kv_pool, num_pages, nkv, page_size, hd);
     if (rc != BG_OK) return rc;
     // tiles of 128 keys where a block may walk many of them (max_position bounds the positions of the step's rows)
     const int reach = window != 0 ? abs(window) : max_position + 1;          // the most keys a row can see
     const bool wide = (reach < max_position + 1 ? reach : max_position + 1) >= at_wide_from();
+    if (ext) {
+        if (hd == 128) return wide ? at_launch<128, 128, false, true>(map, p, n_qblk, stream) : at_launch<128, 64, false, true>(map, p, n_qblk, stream);
+        return wide ? at_launch<64, 128, false, true>(map, p, n_qblk, stream) : at_launch<64, 64, false, true>(map, p, n_qblk, stream);
+    }
     if (sink) {
         if (hd == 128) return wide ? at_launch<128, 128, true>(map, p, n_qblk, stream) : at_launch<128, 64, true>(map, p, n_qblk, stream);
         return wide ? at_launch<64, 128, true>(map, p, n_qblk, stream) : at_launch<64, 64, true>(map, p, n_qblk, stream);
@@ -559,12 +581,14 @@ extern "C" int bg_attention_tc_sink(const void* q, int q_stride, const void* kv_
 }
 
 // The same with what a layer may add to the softmax: a sink's score for every query head (float [nh]; null with `sink`
-// set: a score of 0; `sink` 0: none) and scores squashed to softcap * tanh(score / softcap) (0: as they are).
+// set: a score of 0; `sink` 0: none), scores squashed to softcap * tanh(score / softcap) (0: as they are), scores that fall
+// by slopes[head] (float [nh], or null) per position of distance, and `keep` first positions that a window never loses.
 extern "C" int bg_attention_tc_ext(const void* q, int q_stride, const void* kv_pool, int num_pages, int page_size,
                                    const int* block_table, int max_pages, const int* positions, const int* qblk, int n_qblk,
                                    void* out, int out_stride, int nh, int nkv, int hd, int window, float scale, int max_position,
-                                   int sink, const float* sink_weight, float softcap, unsigned* status, cudaStream_t stream) {
+                                   int sink, const float* sink_weight, float softcap, int keep, const float* slopes, unsigned* status,
+                                   cudaStream_t stream) {
     return attention_tc(q, q_stride, kv_pool, num_pages, page_size, block_table, max_pages, positions, qblk, n_qblk, out, out_stride,
                         nh, nkv, hd, window, scale, max_position, sink != 0 || sink_weight != nullptr, status, stream, sink_weight,
-                        softcap);
+                        softcap, keep, slopes);
 }

@@ -23,6 +23,7 @@
 #define BG_STATUS_BAD_TOKEN 1u      // a token id outside [0, vocab)
 #define BG_STATUS_BAD_PAGE 2u       // a block-table entry outside [0, num_pages)
 #define BG_STATUS_TIMEOUT 4u        // a bounded wait ran out
+#define BG_STATUS_BAD_POSITION 8u   // a position outside the table of position vectors
 
 // Dynamic shared memory from which a kernel asks for more than the default: the default limit of 48 KB holds for
 // a kernel's static and dynamic shared memory together, so a request of exactly 48 KB beside a few static
@@ -119,6 +120,10 @@ __host__ __device__ __forceinline__ int first_visible(int pos, int window) {
     if (window < 0) return pos - pos % (-window);
     return 0;
 }
+
+// Whether a query whose window begins at `lo` sees the position `key` (at or before its own): the window never loses the
+// sequence's first `keep` positions.
+__host__ __device__ __forceinline__ bool key_seen(int key, int lo, int keep) { return key >= lo || key < keep; }
 
 template <typename T> __device__ __forceinline__ float to_float(T v);
 template <> __device__ __forceinline__ float to_float<float>(float v) { return v; }

@@ -418,7 +418,9 @@ static size_t decay_chunk_out_smem(int np, int nvp) {
 // ---------------------------------------------------------------------------------------------------------------
 // x[t] (= or +=) sum_i scale_i * term_i[t], term_i a [T, d] tensor of either type or the float partial sums of a
 // split product; then, when asked, the rows of x RMS-normed with one or two weight vectors (the two norms of a layer
-// whose sublayers read the same stream share the statistics).  The sum and the statistics are float.
+// whose sublayers read the same stream share the statistics).  The sum and the statistics are float.  A term may itself be
+// RMS-normed over the row first, with a float weight vector (a branch whose result is normed before it is added).  With
+// `center` the norm of the rows is a layer norm: the mean is taken off first, and a shift vector may follow the weight.
 constexpr int MAX_TERMS = 6;
 struct TermsParams {
     float* x;
@@ -427,6 +429,9 @@ struct TermsParams {
     const void* w1; const void* w2; int w_dtype; float eps;
     void* out1; void* out2; int out_dtype;
     int d;
+    const float* nw[MAX_TERMS]; float neps[MAX_TERMS];        // weights of a normed term (null: the term as it is)
+    int any_normed, center;
+    const void* b1; const void* b2;                           // shift vectors of the weights' type, or null
 };
 
 __device__ __forceinline__ float term_value(const TermsParams& p, int i, size_t at) {
@@ -440,47 +445,112 @@ __device__ __forceinline__ void store_value(void* out, int dtype, size_t at, flo
     if (dtype == BG_DTYPE_F32) ((float*)out)[at] = v; else ((__nv_bfloat16*)out)[at] = __float2bfloat16_rn(v);
 }
 
+// What every term of row t is multiplied by besides its weight: its constant, and for a normed term the reciprocal of its
+// root mean square.  Every thread of the block comes here; `mult` is read after the call.
+__device__ __forceinline__ void term_multipliers(const TermsParams& p, size_t t, float* mult, float* red) {
+    for (int i = 0; i < p.n_terms; ++i) {
+        float f = p.scale[i];
+        if (p.nw[i]) {
+            float ss = 0.0f;
+            for (int j = threadIdx.x; j < p.d; j += blockDim.x) {
+                const float v = term_value(p, i, t * p.d + j);
+                ss += v * v;
+            }
+            ss = block_sum(ss, red);
+            f /= sqrtf(ss / (float)p.d + p.neps[i]);
+        }
+        if (threadIdx.x == 0) mult[i] = f;
+    }
+    __syncthreads();
+}
+
 __global__ void __launch_bounds__(256) add_terms_norm_kernel(TermsParams p) {
     extern __shared__ float row_s[];
     __shared__ float red[32];
+    __shared__ float mult[MAX_TERMS];
     pdl_launch();
     pdl_wait();
     const size_t t = blockIdx.x;
-    float ss = 0.0f;
+    float ss = 0.0f, sum = 0.0f;
+    term_multipliers(p, t, mult, red);
     for (int j = threadIdx.x; j < p.d; j += blockDim.x) {
         const size_t at = t * p.d + j;
         float v = p.assign ? 0.0f : p.x[at];
-        for (int i = 0; i < p.n_terms; ++i) v = fmaf(p.scale[i], term_value(p, i, at), v);
+        for (int i = 0; i < p.n_terms; ++i) v = fmaf(p.nw[i] ? mult[i] * p.nw[i][j] : mult[i], term_value(p, i, at), v);
         if (p.n_terms > 0 || p.assign) p.x[at] = v;
         row_s[j] = v;
         ss += v * v;
+        sum += v;
     }
     if (!p.out1) return;
+    float mean = 0.0f;
+    if (p.center) {
+        mean = block_sum(sum, red) / (float)p.d;
+        ss = 0.0f;
+        for (int j = threadIdx.x; j < p.d; j += blockDim.x) { const float v = row_s[j] - mean; ss += v * v; }
+    }
     ss = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)p.d + p.eps);
     for (int j = threadIdx.x; j < p.d; j += blockDim.x) {
-        const float v = row_s[j] * inv;
-        store_value(p.out1, p.out_dtype, t * p.d + j, v * weight_value(p.w1, p.w_dtype, j));
-        if (p.out2) store_value(p.out2, p.out_dtype, t * p.d + j, v * weight_value(p.w2, p.w_dtype, j));
+        const float v = (row_s[j] - mean) * inv;
+        store_value(p.out1, p.out_dtype, t * p.d + j, fmaf(v, weight_value(p.w1, p.w_dtype, j), p.b1 ? weight_value(p.b1, p.w_dtype, j) : 0.0f));
+        if (p.out2) store_value(p.out2, p.out_dtype, t * p.d + j, fmaf(v, weight_value(p.w2, p.w_dtype, j), p.b2 ? weight_value(p.b2, p.w_dtype, j) : 0.0f));
     }
 }
 
 // The same, four columns a thread at a time (d a multiple of 4, every pointer 16-byte aligned): the terms are walked
 // outside the columns, so a term's type and its number of partial sums are looked at once per group of four.
+// The sum of the partial sums of term i, four columns from element `at` on.
+__device__ __forceinline__ float4 term_value4(const TermsParams& p, int i, size_t at) {
+    float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+    for (int q = 0; q < p.parts[i]; ++q) {
+        float4 a;
+        if (p.dtype[i] == BG_DTYPE_F32) {
+            a = *reinterpret_cast<const float4*>((const float*)p.term[i] + at + (size_t)q * p.part_stride[i]);
+        } else {
+            const uint2 raw = *reinterpret_cast<const uint2*>((const __nv_bfloat16*)p.term[i] + at + (size_t)q * p.part_stride[i]);
+            const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+            const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+            a = make_float4(lo.x, lo.y, hi.x, hi.y);
+        }
+        v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+    }
+    return v;
+}
+
 __global__ void __launch_bounds__(1024) add_terms_norm_vec4_kernel(TermsParams p) {
     extern __shared__ __align__(16) float row_s[];
     __shared__ float red[32];
+    __shared__ float mult[MAX_TERMS];
     pdl_launch();
     pdl_wait();
     const size_t t = blockIdx.x;
     const int d4 = p.d >> 2;
-    float ss = 0.0f;
+    float ss = 0.0f, sum = 0.0f;
+    if (p.any_normed) {
+        for (int i = 0; i < p.n_terms; ++i) {
+            float q = 0.0f;
+            if (!p.nw[i]) continue;
+            for (int j = threadIdx.x; j < d4; j += blockDim.x) {
+                const float4 a = term_value4(p, i, t * p.d + (size_t)j * 4);
+                q += a.x * a.x + a.y * a.y + a.z * a.z + a.w * a.w;
+            }
+            q = block_sum(q, red);
+            if (threadIdx.x == 0) mult[i] = p.scale[i] / sqrtf(q / (float)p.d + p.neps[i]);
+        }
+        __syncthreads();
+    }
     for (int j = threadIdx.x; j < d4; j += blockDim.x) {
         const size_t at = t * p.d + (size_t)j * 4;
         float4 v = p.assign ? make_float4(0.0f, 0.0f, 0.0f, 0.0f) : *reinterpret_cast<const float4*>(p.x + at);
         for (int i = 0; i < p.n_terms; ++i) {
             const float sc = p.scale[i];
-            if (p.dtype[i] == BG_DTYPE_F32) {
+            if (p.nw[i]) {                                   // a normed term: its columns have weights of their own
+                const float4 a = term_value4(p, i, at);
+                const float4 w = *reinterpret_cast<const float4*>(p.nw[i] + (size_t)j * 4);
+                const float f = mult[i];
+                v.x = fmaf(f * w.x, a.x, v.x); v.y = fmaf(f * w.y, a.y, v.y); v.z = fmaf(f * w.z, a.z, v.z); v.w = fmaf(f * w.w, a.w, v.w);
+            } else if (p.dtype[i] == BG_DTYPE_F32) {
                 const float* base = (const float*)p.term[i] + at;
 #pragma unroll 4
                 for (int q = 0; q < p.parts[i]; ++q) {
@@ -501,22 +571,38 @@ __global__ void __launch_bounds__(1024) add_terms_norm_vec4_kernel(TermsParams p
         if (p.n_terms > 0 || p.assign) *reinterpret_cast<float4*>(p.x + at) = v;
         *reinterpret_cast<float4*>(row_s + (size_t)j * 4) = v;
         ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+        sum += (v.x + v.y) + (v.z + v.w);
     }
     if (!p.out1) return;
+    float mean = 0.0f;
+    if (p.center) {
+        mean = block_sum(sum, red) / (float)p.d;
+        ss = 0.0f;
+        for (int j = threadIdx.x; j < d4; j += blockDim.x) {           // (every thread reads the columns it wrote)
+            const float4 v = *reinterpret_cast<const float4*>(row_s + (size_t)j * 4);
+            const float a = v.x - mean, b = v.y - mean, c = v.z - mean, e = v.w - mean;
+            ss += a * a + b * b + c * c + e * e;
+        }
+    }
     ss = block_sum(ss, red);
     const float inv = 1.0f / sqrtf(ss / (float)p.d + p.eps);
     for (int j = threadIdx.x; j < d4; j += blockDim.x) {
         const float4 v = *reinterpret_cast<const float4*>(row_s + (size_t)j * 4);
-        const float r[4] = {v.x * inv, v.y * inv, v.z * inv, v.w * inv};
+        const float r[4] = {(v.x - mean) * inv, (v.y - mean) * inv, (v.z - mean) * inv, (v.w - mean) * inv};
         const size_t at = t * p.d + (size_t)j * 4;
 #pragma unroll
         for (int o = 0; o < 2; ++o) {
             void* out = o == 0 ? p.out1 : p.out2;
             const void* w = o == 0 ? p.w1 : p.w2;
+            const void* b = o == 0 ? p.b1 : p.b2;
             if (!out) continue;
             float y[4];
 #pragma unroll
             for (int k = 0; k < 4; ++k) y[k] = r[k] * weight_value(w, p.w_dtype, j * 4 + k);
+            if (b) {
+#pragma unroll
+                for (int k = 0; k < 4; ++k) y[k] += weight_value(b, p.w_dtype, j * 4 + k);
+            }
             if (p.out_dtype == BG_DTYPE_F32) {
                 *reinterpret_cast<float4*>((float*)out + at) = make_float4(y[0], y[1], y[2], y[3]);
             } else {
@@ -618,16 +704,19 @@ extern "C" int bg_decay_attention_chunked(const void* src, int src_dtype, int sr
 extern "C" int bg_add_terms_norm(float* x, int n_rows, int d, int assign, int n_terms, const void* const* terms, const int* dtypes,
                                  const int* parts, const long long* part_strides, const float* scales, const void* w1,
                                  const void* w2, int w_dtype, float eps, void* out1, void* out2, int out_dtype,
-                                 cudaStream_t stream) {
+                                 const float* const* term_weights, const float* term_eps, int center, const void* b1,
+                                 const void* b2, cudaStream_t stream) {
     if (n_rows <= 0 || d <= 0) return BG_OK;
     if (n_terms < 0 || n_terms > MAX_TERMS || (out2 && !out1) || (out1 && !w1) || (out2 && !w2)) return BG_ERR_SHAPE;
     TermsParams p;
     p.x = x; p.n_terms = n_terms; p.assign = assign; p.w1 = w1; p.w2 = w2; p.w_dtype = w_dtype; p.eps = eps; p.out1 = out1;
-    p.out2 = out2; p.out_dtype = out_dtype; p.d = d;
+    p.out2 = out2; p.out_dtype = out_dtype; p.d = d; p.center = center; p.b1 = b1; p.b2 = b2; p.any_normed = 0;
     for (int i = 0; i < MAX_TERMS; ++i) {
         const bool have = i < n_terms;
         p.term[i] = have ? terms[i] : nullptr; p.dtype[i] = have ? dtypes[i] : BG_DTYPE_F32; p.parts[i] = have ? parts[i] : 0;
         p.part_stride[i] = have ? (size_t)part_strides[i] : 0; p.scale[i] = have ? scales[i] : 0.0f;
+        p.nw[i] = have && term_weights ? term_weights[i] : nullptr; p.neps[i] = have && term_eps ? term_eps[i] : 0.0f;
+        if (p.nw[i]) p.any_normed = 1;
         if (have && (parts[i] < 1 || (dtypes[i] != BG_DTYPE_F32 && dtypes[i] != BG_DTYPE_BF16))) return BG_ERR_SHAPE;
     }
     const size_t smem = (size_t)d * sizeof(float);
@@ -639,7 +728,7 @@ extern "C" int bg_add_terms_norm(float* x, int n_rows, int d, int assign, int n_
     }
     bool vec = d % 4 == 0 && ((uintptr_t)x % 16) == 0 && (!out1 || (uintptr_t)out1 % 16 == 0) && (!out2 || (uintptr_t)out2 % 16 == 0);
     for (int i = 0; i < n_terms; ++i)
-        vec = vec && ((uintptr_t)terms[i] % 16) == 0 && (part_strides[i] % 4) == 0;
+        vec = vec && ((uintptr_t)terms[i] % 16) == 0 && (part_strides[i] % 4) == 0 && ((uintptr_t)p.nw[i] % 16) == 0;
     // steps of few rows cannot fill the device with rows: a row's groups of four columns then get a thread each
     const int vthreads = n_rows >= 512 ? 256 : (d / 4 + 31) / 32 * 32 < 64 ? 64 : (d / 4 + 31) / 32 * 32 > 1024 ? 1024 : (d / 4 + 31) / 32 * 32;
     if (vec) launch(add_terms_norm_vec4_kernel, dim3(n_rows), dim3(vthreads), smem, stream, p);

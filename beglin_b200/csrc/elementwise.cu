@@ -10,10 +10,12 @@ namespace bg {
 
 // ---------------------------------------------------------------------------------------------
 // x[t, :] = table[ids[t], :] * scale   (qwen_infer.c:1438-1439, where the scale is 1).  An id outside the
-// table sets a status bit and yields a row of zeros.
+// table sets a status bit and yields a row of zeros.  With `pos_table` [n_pos, d] the row of the token's position is added,
+// unscaled; a position outside it sets a status bit and adds nothing.
 template <typename TT>
 __global__ void embed_gather_kernel(const TT* __restrict__ table, const int* __restrict__ ids,
-                                    float* __restrict__ out, int d, int vocab, float scale, unsigned* status) {
+                                    float* __restrict__ out, int d, int vocab, float scale, const TT* __restrict__ pos_table,
+                                    const int* __restrict__ positions, int n_pos, unsigned* status) {
     pdl_launch();
     pdl_wait();
     const int t = blockIdx.x;
@@ -25,7 +27,13 @@ __global__ void embed_gather_kernel(const TT* __restrict__ table, const int* __r
         return;
     }
     const TT* row = table + (size_t)id * d;
-    for (int i = threadIdx.x; i < d; i += blockDim.x) o[i] = to_float(row[i]) * scale;
+    const TT* at = nullptr;
+    if (pos_table) {
+        const int pos = positions[t];
+        if (pos >= 0 && pos < n_pos) at = pos_table + (size_t)pos * d;
+        else if (threadIdx.x == 0 && status) atomicOr(status, BG_STATUS_BAD_POSITION);
+    }
+    for (int i = threadIdx.x; i < d; i += blockDim.x) o[i] = to_float(row[i]) * scale + (at ? to_float(at[i]) : 0.0f);
 }
 
 // Random weights on the device: out[i] = mean + std * x(key, first + i), x approximately normal, a function of the
@@ -320,11 +328,14 @@ __global__ void add_residual_kernel(float* __restrict__ x, const TD* __restrict_
 // approximations (ex2.approx and the approximate division: relative error about 2^-21), which makes the kernel bound by memory
 // instead of by these two functions; a float result is computed with expf and a division.
 // ACT 0: silu.  ACT 1: the tanh form of GELU, 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))), which is
-// g * sigmoid(2 sqrt(2/pi) (g + 0.044715 g^3)); a float result takes tanhf.
+// g * sigmoid(2 sqrt(2/pi) (g + 0.044715 g^3)); a float result takes tanhf.  ACT 2: the square of relu.
 template <typename TO, int ACT> __device__ __forceinline__ float silu_mul(float g, float u) {
     if constexpr (ACT == 0) {
         if constexpr (std::is_same<TO, float>::value) return (g / (1.0f + expf(-g))) * u;
         else return __fdividef(g, 1.0f + __expf(-g)) * u;
+    } else if constexpr (ACT == 2) {
+        const float z = fmaxf(g, 0.0f);
+        return z * z * u;
     } else {
         const float z = 0.7978845608028654f * (g + 0.044715f * g * g * g);
         if constexpr (std::is_same<TO, float>::value) return 0.5f * g * (1.0f + tanhf(z)) * u;
@@ -620,10 +631,12 @@ __global__ void rope_kv_append_heads_kernel(const TS* __restrict__ src, int src_
 using namespace bg;
 
 extern "C" int bg_embed_gather(const void* table, int table_dtype, const int* ids, float* out, int T,
-                               int d, int vocab, float scale, unsigned* status, cudaStream_t stream) {
+                               int d, int vocab, float scale, const void* pos_table, const int* positions, int n_pos,
+                               unsigned* status, cudaStream_t stream) {
     if (T <= 0) return BG_OK;
+    if (pos_table && !positions) return BG_ERR_SHAPE;
     BG_DISPATCH_DTYPE(table_dtype, TT, launch(embed_gather_kernel<TT>, dim3(T), dim3(256), 0, stream,
-        (const TT*)table, ids, out, d, vocab, scale, status));
+        (const TT*)table, ids, out, d, vocab, scale, (const TT*)pos_table, positions, n_pos, status));
     BG_LAUNCH_CHECK();
     return BG_OK;
 }
@@ -814,8 +827,9 @@ static int activation_launch(const void* z, int parts, size_t part_stride, void*
 extern "C" int bg_activation(const void* z, int in_dtype, int parts, long long part_stride, void* out, int out_dtype, long long total,
                              int act, cudaStream_t stream) {
     if (total <= 0) return BG_OK;
-    if (parts < 1 || act < 0 || act > 1) return BG_ERR_SHAPE;
+    if (parts < 1 || act < 0 || act > 2) return BG_ERR_SHAPE;
     BG_DISPATCH_DTYPE(in_dtype, TI, BG_DISPATCH_DTYPE(out_dtype, TO, {
+        if (act == 2) return activation_launch<TI, TO, 2>(z, parts, (size_t)part_stride, out, (size_t)total, stream);
         if (act == 0) return activation_launch<TI, TO, 0>(z, parts, (size_t)part_stride, out, (size_t)total, stream);
         return activation_launch<TI, TO, 1>(z, parts, (size_t)part_stride, out, (size_t)total, stream);
     }));

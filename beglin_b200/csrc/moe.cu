@@ -20,12 +20,14 @@
 
 namespace bg {
 
-// How the router's logits become scores (`mode`): 0 the logit itself, 1 its sigmoid, 2 the softmax over all E logits.
+// How the router's logits become scores (`mode`): 0 the logit itself, 1 its sigmoid, 2 the softmax over all E logits, 3 the
+// softmax over the chosen logits only (the choice is made on the logits themselves).
 struct RouteRule {
     int mode;
     int renorm;             // the chosen scores are divided by their sum
     const float* bias;      // [E] or null: added to the scores for the CHOICE only; the weights are the scores without it
     float scale;            // multiplies the weights
+    const float* logit_bias;    // [E] or null: part of the logits
 };
 
 // One warp chooses for one token: `sc` holds the token's E logits in shared memory and is used up.  Without a bias and
@@ -36,6 +38,10 @@ __device__ __forceinline__ void choose_experts(float* sc, int E, int top, RouteR
                                                float* __restrict__ weights, size_t t, int lane) {
     float total = 0.0f;
     float zmax = 0.0f, inv = 1.0f;
+    if (rule.logit_bias) {
+        for (int e = lane; e < E; e += 32) sc[e] += rule.logit_bias[e];
+        __syncwarp();
+    }
     if (rule.mode == 2) {                                  // softmax over all experts, float
         float m = -INFINITY;
         for (int e = lane; e < E; e += 32) m = fmaxf(m, sc[e]);
@@ -46,7 +52,7 @@ __device__ __forceinline__ void choose_experts(float* sc, int E, int top, RouteR
     }
     const bool on_scores = rule.mode == 2 || rule.bias != nullptr;
     auto score_of = [&](float z) {
-        return rule.mode == 2 ? expf(z - zmax) * inv : (rule.mode == 1 ? 1.0f / (1.0f + expf(-z)) : z);
+        return rule.mode >= 2 ? expf(z - zmax) * inv : (rule.mode == 1 ? 1.0f / (1.0f + expf(-z)) : z);
     };
     for (int j = 0; j < top; ++j) {
         float best = -INFINITY;
@@ -63,6 +69,7 @@ __device__ __forceinline__ void choose_experts(float* sc, int E, int top, RouteR
             if (ob > best || (ob == best && oa < arg)) { best = ob; arg = oa; }
         }
         if (arg == 0x7fffffff) arg = 0;                     // (every score NaN or -inf: a defined choice)
+        if (rule.mode == 3 && j == 0) zmax = sc[arg];           // (without a choice bias the first choice is the largest)
         const float score = score_of(on_scores ? sc[arg] : best);
         __syncwarp();
         if (lane == 0) {
@@ -73,7 +80,7 @@ __device__ __forceinline__ void choose_experts(float* sc, int E, int top, RouteR
         total += score;
         __syncwarp();
     }
-    if (rule.renorm && lane < top) weights[(size_t)t * top + lane] /= total;
+    if ((rule.renorm || rule.mode == 3) && lane < top) weights[(size_t)t * top + lane] /= total;
 }
 
 __global__ void route_topk_kernel(const float* __restrict__ logits, int T, int E, int top, RouteRule rule,
@@ -502,10 +509,10 @@ extern "C" int bg_route_logits(const void* A, int a_dtype, int lda, const float*
 }
 
 extern "C" int bg_route_topk(const float* logits, int T, int E, int top, int mode, int renorm, const float* bias, float scale,
-                             int* ids, float* weights, cudaStream_t stream) {
+                             const float* logit_bias, int* ids, float* weights, cudaStream_t stream) {
     if (T <= 0) return BG_OK;
-    if (E <= 0 || top <= 0 || top > E || top > 32 || mode < 0 || mode > 2) return BG_ERR_SHAPE;
-    const RouteRule rule = {mode, renorm, bias, scale};
+    if (E <= 0 || top <= 0 || top > E || top > 32 || mode < 0 || mode > 3 || (mode == 3 && bias)) return BG_ERR_SHAPE;
+    const RouteRule rule = {mode, renorm, bias, scale, logit_bias};
     const int warps = 4;
     const size_t smem = (size_t)warps * E * sizeof(float);
     if (smem > 40 * 1024) return BG_ERR_UNSUPPORTED;
@@ -517,10 +524,11 @@ extern "C" int bg_route_topk(const float* logits, int T, int E, int top, int mod
 
 // The router in one kernel: float logits of h [T, d] (either type, row stride ldh) against W [E, d] float, and the choice.
 extern "C" int bg_route(const void* h, int h_dtype, int ldh, const float* W, int T, int d, int E, int top, int mode, int renorm,
-                        const float* bias, float scale, int* ids, float* weights, float* logits_out, cudaStream_t stream) {
+                        const float* bias, float scale, const float* logit_bias, int* ids, float* weights, float* logits_out,
+                        cudaStream_t stream) {
     if (T <= 0) return BG_OK;
-    if (E <= 0 || top <= 0 || top > E || top > 32 || d <= 0 || mode < 0 || mode > 2) return BG_ERR_SHAPE;
-    const RouteRule rule = {mode, renorm, bias, scale};
+    if (E <= 0 || top <= 0 || top > E || top > 32 || d <= 0 || mode < 0 || mode > 3 || (mode == 3 && bias)) return BG_ERR_SHAPE;
+    const RouteRule rule = {mode, renorm, bias, scale, logit_bias};
     const size_t smem = (size_t)ROUTE_TOKENS * E * sizeof(float);
     if (smem > 40 * 1024) return BG_ERR_UNSUPPORTED;
     const dim3 grid((T + ROUTE_TOKENS - 1) / ROUTE_TOKENS), block(32 * ROUTE_TOKENS);

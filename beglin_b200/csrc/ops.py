@@ -14,13 +14,14 @@ import torch
 from . import build as _build
 
 F32, BF16 = 0, 1
-STATUS_BAD_TOKEN, STATUS_BAD_PAGE, STATUS_TIMEOUT = 1, 2, 4
+STATUS_BAD_TOKEN, STATUS_BAD_PAGE, STATUS_TIMEOUT, STATUS_BAD_POSITION = 1, 2, 4, 8
 
 _c_int, _c_float, _c_void_p, _c_ll = ctypes.c_int, ctypes.c_float, ctypes.c_void_p, ctypes.c_longlong
 _c_ull = ctypes.c_ulonglong
 
 _SIGNATURES = {
-    "bg_embed_gather": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_void_p],
+    "bg_embed_gather": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_void_p, _c_int,
+                        _c_void_p, _c_void_p],
     "bg_softcap": [_c_void_p, _c_ll, _c_float, _c_void_p],
     "bg_fill_normal": [_c_void_p, _c_int, _c_ll, _c_ull, _c_ll, _c_float, _c_float, _c_void_p],
     "bg_add_rmsnorm": [_c_void_p, _c_void_p, _c_int, _c_int, _c_ll, _c_void_p, _c_int, _c_float, _c_void_p, _c_int,
@@ -35,9 +36,10 @@ _SIGNATURES = {
     "bg_attention_plan": [_c_int, _c_int, _c_int, ctypes.POINTER(_c_int), ctypes.POINTER(_c_int)],
     "bg_attention_partial": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int,
                              _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
-                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_void_p, _c_void_p],
+                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_void_p, _c_void_p,
+                             _c_void_p],
     "bg_attention_merge": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
-                           _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
+                           _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p],
     "bg_rmsnorm_add": [_c_void_p, _c_void_p, _c_int, _c_int, _c_ll, _c_void_p, _c_int, _c_float, _c_void_p, _c_int, _c_int,
                        _c_int, _c_void_p],
     "bg_rmsnorm_add_routed": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_float, _c_void_p,
@@ -48,9 +50,10 @@ _SIGNATURES = {
                                _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p,
                                _c_void_p],
     "bg_route_logits": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p],
-    "bg_route_topk": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_void_p],
+    "bg_route_topk": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_void_p,
+                      _c_void_p],
     "bg_route": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_float,
-                 _c_void_p, _c_void_p, _c_void_p, _c_void_p],
+                 _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p],
     "bg_route_combine_ext": [_c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p,
                              _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
     "bg_glu_clamped": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_float, _c_float, _c_void_p],
@@ -80,17 +83,21 @@ _SIGNATURES = {
                                    _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int,
                                    _c_void_p],
     "bg_add_terms_norm": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p,
-                          _c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_void_p, _c_int, _c_void_p],
+                          _c_void_p, _c_void_p, _c_int, _c_float, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int,
+                          _c_void_p, _c_void_p, _c_void_p],
+    "bg_gla_walk": [_c_void_p, _c_void_p, _c_int, _c_void_p],
+    "bg_gla_chunk_plan": [_c_int, _c_int, ctypes.POINTER(_c_int)],
+    "bg_gla_chunked": [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p],
     "bg_attention_mma_plan": [_c_int, _c_int, _c_int, ctypes.POINTER(_c_int)],
     "bg_attention_mma_partial": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p,
                                  _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
-                                 _c_int, _c_float, _c_float, _c_void_p, _c_int, _c_void_p, _c_void_p],
+                                 _c_int, _c_float, _c_float, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p],
     "bg_attention_tc_plan": [_c_int, _c_int, _c_int, ctypes.POINTER(_c_int)],
     "bg_attention_tc": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int,
                         _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p],
     "bg_attention_tc_ext": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int,
                             _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void_p, _c_float,
-                            _c_void_p, _c_void_p],
+                            _c_int, _c_void_p, _c_void_p, _c_void_p],
     "bg_attention_tc_sink": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int,
                              _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p],
     "bg_gemm_f32_nt": [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
@@ -107,7 +114,7 @@ _SIGNATURES = {
                            _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p,
                            _c_void_p],
     "bg_add_layernorm": [_c_void_p, _c_void_p, _c_int, _c_int, _c_ll, _c_void_p, _c_int, _c_float, _c_void_p, _c_int,
-                         _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
+                         _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
     "bg_depth_mix": [_c_void_p, _c_void_p, _c_int, _c_int, _c_ll, _c_void_p, _c_ll, _c_void_p, _c_int, _c_int, _c_ll, _c_void_p],
     "bg_xielu": [_c_void_p, _c_int, _c_int, _c_ll, _c_void_p, _c_int, _c_void_p, _c_int, _c_ll, _c_void_p],
     "bg_rmsnorm_slice": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_float, _c_void_p, _c_int, _c_int,
@@ -325,6 +332,8 @@ def raise_on_status(status: torch.Tensor) -> None:
         what.append("a token id outside the vocabulary")
     if v & STATUS_BAD_PAGE:
         what.append("a block-table entry outside the page pool")
+    if v & STATUS_BAD_POSITION:
+        what.append("a position outside the table of position vectors")
     if v & STATUS_TIMEOUT:
         what.append("a bounded wait inside a kernel ran out")
     raise KernelError("a kernel recorded: " + "; ".join(what or [f"status {v}"]))
@@ -332,16 +341,23 @@ def raise_on_status(status: torch.Tensor) -> None:
 
 # ------------------------------------------------------------------------------------------------
 def embed_gather(table: torch.Tensor, ids: torch.Tensor, out: torch.Tensor, status: Optional[torch.Tensor],
-                 scale: float = 1.0) -> None:
-    """out[t] = table[ids[t]] * scale as float32; an id outside the table sets BG_STATUS_BAD_TOKEN."""
-    _cuda(table, ids, out)
+                 scale: float = 1.0, pos_table: Optional[torch.Tensor] = None, positions: Optional[torch.Tensor] = None) -> None:
+    """out[t] = table[ids[t]] * scale (+ pos_table[positions[t]]) as float32; an id outside the table sets
+    BG_STATUS_BAD_TOKEN, a position outside the table of position vectors BG_STATUS_BAD_POSITION."""
+    _cuda(table, ids, out, pos_table, positions)
     _i32(ids, "ids")
+    if pos_table is not None:
+        _i32(positions, "positions")
+        if pos_table.dtype != table.dtype or pos_table.shape[1] != table.shape[1] or not pos_table.is_contiguous() \
+                or positions.numel() != ids.numel():
+            raise KernelError("embed_gather: pos_table contiguous [positions, d] of the table's type, one position per id")
     T, d = ids.numel(), table.shape[1]
     if out.dtype != torch.float32 or tuple(out.shape) != (T, d) or not out.is_contiguous() or not table.is_contiguous():
         raise KernelError("embed_gather: out must be contiguous float32 [T, d] and the table contiguous")
     with phase("emb_gather"):
-        _check(lib().bg_embed_gather(_p(table), _dt(table), _p(ids), _p(out), T, d, table.shape[0], float(scale), _p(status),
-                                     _stream()), "embed_gather")
+        _check(lib().bg_embed_gather(_p(table), _dt(table), _p(ids), _p(out), T, d, table.shape[0], float(scale), _p(pos_table),
+                                     _p(positions), 0 if pos_table is None else pos_table.shape[0], _p(status), _stream()),
+               "embed_gather")
 
 
 def fill_normal(out: torch.Tensor, key: int, mean: float, std: float, first: int = 0) -> None:
@@ -405,6 +421,7 @@ def add_residual(x: torch.Tensor, delta: torch.Tensor) -> None:
 
 
 GLU_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
+ACTIVATIONS = dict(GLU_ACTIVATIONS, relu2=2)          # of a feed-forward without a gate branch
 
 
 def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0, activation: str = "silu") -> None:
@@ -428,15 +445,16 @@ def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0, activation:
 
 
 def activation(z: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
-    """out = act(z), z [rows, n] or its float partial sums [parts, rows, n]; act is silu or the tanh form of GELU."""
-    if activation not in GLU_ACTIVATIONS:
-        raise KernelError(f"activation: unknown activation '{activation}' ({', '.join(GLU_ACTIVATIONS)})")
+    """out = act(z), z [rows, n] or its float partial sums [parts, rows, n]; act is silu, the tanh form of GELU or
+    the square of relu."""
+    if activation not in ACTIVATIONS:
+        raise KernelError(f"activation: unknown activation '{activation}' ({', '.join(ACTIVATIONS)})")
     _cuda(z, out)
     parts, stride = _parts(z, "activation: z")
     if tuple(out.shape) != tuple(z.shape[-2:]) or not z.is_contiguous() or not out.is_contiguous():
         raise KernelError("activation: z and out contiguous and of one shape")
     with phase("swiglu"):
-        _check(lib().bg_activation(_p(z), _dt(z), parts, stride, _p(out), _dt(out), out.numel(), GLU_ACTIVATIONS[activation],
+        _check(lib().bg_activation(_p(z), _dt(z), parts, stride, _p(out), _dt(out), out.numel(), ACTIVATIONS[activation],
                                    _stream()), "activation")
 
 
@@ -578,7 +596,8 @@ def _attention(q: torch.Tensor, q_stride: int, kv_pool: torch.Tensor, block_tabl
               positions: torch.Tensor, qblk: torch.Tensor, n_qblk: int, max_position: int, n_rows: int, nh: int,
               nkv: int, hd: int, window: int, split: int, tile: int, bq: int, scale: float, out: torch.Tensor,
               status: Optional[torch.Tensor], kernel: str = "generic", vd: Optional[int] = None, sink: bool = False,
-              sink_weight: Optional[torch.Tensor] = None, softcap: float = 0.0) -> None:
+              sink_weight: Optional[torch.Tensor] = None, softcap: float = 0.0, keep: int = 0,
+              slopes: Optional[torch.Tensor] = None) -> None:
     """Paged grouped-query attention of a step's rows; out is [T, nh*hd].  `kernel`, `bq` and `tile`
     come from `attention_plan`; `qblk` must be cut for that `bq`; `max_position` is the largest
     position among the rows (or a bound on it).
@@ -589,8 +608,15 @@ def _attention(q: torch.Tensor, q_stride: int, kv_pool: torch.Tensor, block_tabl
     query block and write `out` directly.
 
     `sink`: the softmax's denominator also holds exp(b) for a key that has no value, b = 0, or `sink_weight`[head]
-    (float32 [nh]) when given.  `softcap` c > 0: a score s becomes c tanh(s / c)."""
-    _cuda(q, kv_pool, block_table, positions, qblk, out, sink_weight)
+    (float32 [nh]) when given.  `softcap` c > 0: a score s becomes c tanh(s / c).  `slopes` (float32 [nh]): a score falls by
+    slopes[head] for every position its key lies back.  `keep` k > 0: a window never loses the first k positions."""
+    _cuda(q, kv_pool, block_table, positions, qblk, out, sink_weight, slopes)
+    if slopes is not None and (slopes.dtype != torch.float32 or slopes.numel() != nh or not slopes.is_contiguous()):
+        raise KernelError("attention: the slopes are contiguous float32, one per query head")
+    if keep < 0 or (keep and window < 0):
+        raise KernelError("attention: kept first positions go with a sliding window")
+    if kernel == "tc_rows" and (keep or slopes is not None) and (sink or sink_weight is not None):
+        raise KernelError("attention: the tcgen05 kernel takes a sink or falling scores and kept positions, not both")
     if sink_weight is not None:
         sink = True
         if sink_weight.dtype != torch.float32 or sink_weight.numel() != nh or not sink_weight.is_contiguous():
@@ -627,11 +653,11 @@ def _attention(q: torch.Tensor, q_stride: int, kv_pool: torch.Tensor, block_tabl
     if kernel == "tc_rows":
         if q.dtype != torch.bfloat16 or kv_pool.dtype != torch.bfloat16 or out.dtype != torch.bfloat16:
             raise KernelError("attention: the tcgen05 kernel takes bfloat16 queries, caches and outputs")
-        if learned or softcap:
+        if learned or softcap or keep or slopes is not None:
             _check(L.bg_attention_tc_ext(
                 _p(q), q_stride, _p(kv_pool), num_pages, page_size, _p(block_table), block_table.shape[1], _p(positions),
                 _p(qblk), n_qblk, _p(out), out.stride(0), nh, nkv, hd, window, float(scale), int(max_position),
-                1 if sink else 0, _p(sink_weight), float(softcap), _p(status), _stream()), "attention_tcgen05")
+                1 if sink else 0, _p(sink_weight), float(softcap), int(keep), _p(slopes), _p(status), _stream()), "attention_tcgen05")
             return
         _check((L.bg_attention_tc_sink if sink else L.bg_attention_tc)(
             _p(q), q_stride, _p(kv_pool), num_pages, page_size, _p(block_table), block_table.shape[1], _p(positions), _p(qblk),
@@ -644,7 +670,7 @@ def _attention(q: torch.Tensor, q_stride: int, kv_pool: torch.Tensor, block_tabl
         _check(L.bg_attention_mma_partial(_p(q), q_stride, _p(kv_pool), num_pages, page_size, _p(block_table),
                                           block_table.shape[1], _p(positions), _p(qblk), n_qblk, None, None, 1, 1,
                                           nh, nkv, hd, window, split, 0, float(scale), float(softcap), _p(out), out.stride(0),
-                                          _p(status), _stream()), "attention_mma")
+                                          int(keep), _p(slopes), _p(status), _stream()), "attention_mma")
         return
     if kernel == "mma_keys":
         split, n_splits = 0, decode_splits(n_qblk * nkv, max_position + 1)
@@ -654,7 +680,7 @@ def _attention(q: torch.Tensor, q_stride: int, kv_pool: torch.Tensor, block_tabl
             _check(L.bg_attention_mma_partial(_p(q), q_stride, _p(kv_pool), num_pages, page_size, _p(block_table),
                                               block_table.shape[1], _p(positions), _p(qblk) if qblk is not None else None,
                                               n_qblk, None, None, 1, 1, nh, nkv, hd, window, 0, 1, float(scale), float(softcap), _p(out),
-                                              out.stride(0), _p(status), _stream()), "attention_mma_keys")
+                                              out.stride(0), int(keep), _p(slopes), _p(status), _stream()), "attention_mma_keys")
             return
     else:
         n_splits = max_position // split + 1
@@ -664,7 +690,8 @@ def _attention(q: torch.Tensor, q_stride: int, kv_pool: torch.Tensor, block_tabl
         _check(L.bg_attention_partial(_p(q), _dt(q), q_stride, _p(kv_pool), _dt(kv_pool), num_pages, page_size,
                                       _p(block_table), block_table.shape[1], _p(positions), _p(qblk), n_qblk,
                                       _p(part_o), _p(part_ml), n_splits, n_splits, nh, nkv, hd, vd, window, split, tile,
-                                      bq, float(scale), float(softcap), _p(status), _stream()), "attention_partial")
+                                      bq, float(scale), float(softcap), int(keep), _p(slopes), _p(status), _stream()),
+               "attention_partial")
     elif kernel in ("mma_keys", "mma_rows"):
         # (the kernels that write finished rows know the plain softmax only: with the enlarged denominator their rows
         # go through partial results, also when there is one range of keys, and the merge adds the sink's share)
@@ -675,11 +702,12 @@ def _attention(q: torch.Tensor, q_stride: int, kv_pool: torch.Tensor, block_tabl
                                           n_qblk, _p(part_o),
                                           _p(part_ml), n_splits, n_splits, nh, nkv, hd, window, split,
                                           1 if kernel == "mma_keys" else 0,
-                                          float(scale), float(softcap), None, 0, _p(status), _stream()), "attention_mma_partial")
+                                          float(scale), float(softcap), None, 0, int(keep), _p(slopes), _p(status), _stream()),
+               "attention_mma_partial")
     else:
         raise KernelError(f"unknown attention kernel '{kernel}'")
     _check(L.bg_attention_merge(_p(part_o), _p(part_ml), _p(positions), _p(out), _dt(out), out.stride(0), n_rows, nh,
-                                vd, n_splits, split, window, 1 if sink else 0, _p(sink_weight), _stream()), "attention_merge")
+                                vd, n_splits, split, window, 1 if sink else 0, _p(sink_weight), int(keep), _stream()), "attention_merge")
 
 
 def gemm_f32_nt(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
@@ -935,10 +963,12 @@ def sample(logits: torch.Tensor, temperature: Optional[torch.Tensor], uniform: O
 # ------------------------------------------------------------------------------------------------
 # Layer norm, depth-weighted average, xIELU, norms of slices, output gates
 def add_layernorm(x: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Tensor, eps: float, out: torch.Tensor,
-                  rows: Optional[torch.Tensor] = None, update: bool = True) -> None:
-    """As add_rmsnorm, with a layer norm (mean taken off, no bias): v = x[s] (+ delta[s], or the sum of its
-    partial sums); x[s] = v when update; out[r] = (v - mean) / sqrt(var + eps) * weight, s = rows[r] or r."""
-    _cuda(x, delta, weight, out, rows)
+                  rows: Optional[torch.Tensor] = None, update: bool = True, bias: Optional[torch.Tensor] = None) -> None:
+    """As add_rmsnorm, with a layer norm (mean taken off): v = x[s] (+ delta[s], or the sum of its
+    partial sums); x[s] = v when update; out[r] = (v - mean) / sqrt(var + eps) * weight (+ bias), s = rows[r] or r."""
+    _cuda(x, delta, weight, out, rows, bias)
+    if bias is not None and (bias.dtype != weight.dtype or bias.numel() != weight.numel() or not bias.is_contiguous()):
+        raise KernelError("add_layernorm: the shift vector is contiguous and of the weight's type and size")
     d = x.shape[1]
     n = rows.numel() if rows is not None else x.shape[0]
     if x.dtype != torch.float32 or not x.is_contiguous() or not out.is_contiguous() or not weight.is_contiguous():
@@ -955,7 +985,7 @@ def add_layernorm(x: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.
     with phase("layernorm"):
         _check(lib().bg_add_layernorm(_p(x), _p(delta), _dt(delta) if delta is not None else F32, parts, stride, _p(weight),
                                       _dt(weight), float(eps), _p(out), _dt(out), _p(rows), n, d, 1 if update else 0,
-                                      _stream()), "add_layernorm")
+                                      _p(bias), _stream()), "add_layernorm")
 
 
 def depth_mix(x: torch.Tensor, delta: Optional[torch.Tensor], history: torch.Tensor, weight: torch.Tensor, terms: int) -> None:
@@ -1417,12 +1447,23 @@ def decay_attention(src: torch.Tensor, q_col: int, k_col: int, v_col: int, decay
 
 def add_terms_norm(x: torch.Tensor, terms, assign: bool = False, weight1: Optional[torch.Tensor] = None,
                    weight2: Optional[torch.Tensor] = None, eps: float = 0.0, out1: Optional[torch.Tensor] = None,
-                   out2: Optional[torch.Tensor] = None) -> None:
+                   out2: Optional[torch.Tensor] = None, center: bool = False, bias1: Optional[torch.Tensor] = None,
+                   bias2: Optional[torch.Tensor] = None) -> None:
     """x (= or +=) sum_i scale_i * term_i for `terms` = [(tensor, scale), ...], each tensor [T, d] of either type or float
     partial sums [parts, T, d]; then out1 = rmsnorm(x) * weight1 and out2 = rmsnorm(x) * weight2 when given (one pass
-    over the rows for the sum and both norms).  x is the float32 residual [T, d]."""
+    over the rows for the sum and both norms).  x is the float32 residual [T, d].  A term may also be an object with
+    `rows`, `weight` (float32 [d]) and `eps` in the tensor's place: its rows are RMS-normed, times the weight, before they
+    are added.  `center`: the norms of x are layer norms, with the shift vectors `bias1`, `bias2` (of the weights' type)."""
+    normed = [(t.weight, float(t.eps)) if hasattr(t, "rows") else (None, 0.0) for t, _ in terms]
+    terms = [(getattr(t, "rows", t), c) for t, c in terms]
     tensors = [t for t, _ in terms]
-    _cuda(x, weight1, weight2, out1, out2, *tensors)
+    _cuda(x, weight1, weight2, out1, out2, bias1, bias2, *tensors, *[w for w, _ in normed])
+    for w, _ in normed:
+        if w is not None and (w.dtype != torch.float32 or w.numel() != x.shape[1] or not w.is_contiguous()):
+            raise KernelError("add_terms_norm: a normed term's weight is contiguous float32 [d]")
+    for b, w in ((bias1, weight1), (bias2, weight2)):
+        if b is not None and (not center or w is None or b.dtype != w.dtype or b.numel() != w.numel() or not b.is_contiguous()):
+            raise KernelError("add_terms_norm: a shift vector goes with a layer norm's weight, of its type and size")
     T, d = x.shape
     if x.dtype != torch.float32 or not x.is_contiguous():
         raise KernelError("add_terms_norm: x is contiguous float32")
@@ -1445,7 +1486,74 @@ def add_terms_norm(x: torch.Tensor, terms, assign: bool = False, weight1: Option
         _check(lib().bg_add_terms_norm(_p(x), T, d, 1 if assign else 0, k, arr(_c_void_p, ptrs), arr(_c_int, dts), arr(_c_int, parts),
                                        arr(_c_ll, strides), arr(_c_float, scales), _p(weight1), _p(weight2),
                                        _dt(weight1) if weight1 is not None else F32, float(eps), _p(out1), _p(out2),
-                                       _dt(out1) if out1 is not None else F32, _stream()), "add_terms_norm")
+                                       _dt(out1) if out1 is not None else F32, arr(_c_void_p, [_p(w) for w, _ in normed]),
+                                       arr(_c_float, [e for _, e in normed]), 1 if center else 0, _p(bias1), _p(bias2), _stream()),
+               "add_terms_norm")
+
+
+# ---------------------------------------------------------------------------------------------------- gated linear attention
+class _GlaArgs(ctypes.Structure):
+    _fields_ = [("src", _c_void_p), ("src_stride", _c_ll), ("q_col", _c_int), ("k_col", _c_int), ("v_col", _c_int), ("g_col", _c_int),
+                ("forget", _c_int), ("q_silu", _c_int), ("r_col", _c_int), ("rank", _c_int), ("q_scale", _c_float), ("power", _c_float),
+                ("eps", _c_float), ("pad", _c_float), ("bias", _c_void_p), ("lower", _c_void_p), ("wa", _c_void_p), ("norm_w", _c_void_p),
+                ("state", _c_void_p), ("slot_stride", _c_ll), ("slots", _c_void_p), ("out", _c_void_p), ("out_dtype", _c_int),
+                ("H", _c_int), ("n", _c_int), ("nv", _c_int)]
+
+
+def gla_chunk(n: int, nv: int) -> int:
+    """The number of tokens in a chunk of the chunked kernels for heads of n x nv values, 0 when they do not take them."""
+    c = _c_int(0)
+    return c.value if lib().bg_gla_chunk_plan(int(n), int(nv), ctypes.byref(c)) == 0 else 0
+
+
+def gated_linear_attention(src: torch.Tensor, q_col: int, k_col: int, v_col: int, bias: torch.Tensor, norm_weight: torch.Tensor, eps: float,
+                           state: torch.Tensor, slots: torch.Tensor, reqs: Optional[torch.Tensor], n_req: int, out: torch.Tensor, H: int,
+                           n: int, nv: int, *, lower: Optional[torch.Tensor] = None, decay_matrix: Optional[torch.Tensor] = None,
+                           r_col: int = 0, power: float = 1.0, q_silu: bool = False, q_scale: float = 1.0, g_col: int = -1,
+                           chunks: Optional[torch.Tensor] = None, n_chunks: int = 0, longs: Optional[torch.Tensor] = None,
+                           n_long: int = 0) -> None:
+    """Linear attention with a decay per key channel, its head norm and its gate.  `src` float32 [T, W] holds the products of
+    the mixer's input: from `q_col` the queries' [H, n] (q = q_scale times the product, or times its silu with `q_silu`), from
+    `k_col` either the forget gate's [H, n] (with `lower`, float32 [H n]: a = l + (1 - l) sigmoid(f + bias), k = 1 - a) or the
+    keys' (with `decay_matrix`, float32 [H n, rank], and a short row of `rank` values from `r_col`:
+    a = sigmoid(decay_matrix r + bias)^power), from `v_col` the values [H, nv], and from `g_col` (if not negative) the
+    gate's [H, nv].  Per request and head, for its rows in turn: S <- diag(a) S + k v^T, o = S^T q, with S [n, nv] float32 at
+    state[slots[request], h * n * nv ...]; out[t] = o / rms(o) * norm_weight (float32 [nv]) (* silu(gate)), [T, H nv] in either
+    type.  `reqs` [n_req, 3], or `chunks` and `longs` for requests of many rows, as in `decay_attention`."""
+    _cuda(src, bias, norm_weight, state, slots, reqs, out, lower, decay_matrix, chunks, longs)
+    _i32(slots, "slots")
+    T, W = src.shape
+    if src.dtype != torch.float32 or src.stride(1) != 1:
+        raise KernelError("gated_linear_attention: src is float32 rows")
+    if (lower is None) == (decay_matrix is None):
+        raise KernelError("gated_linear_attention: either the forget gate's lower bounds or a decay matrix")
+    rank = 0 if decay_matrix is None else decay_matrix.shape[1]
+    if max(q_col + H * n, k_col + H * n, v_col + H * nv, g_col + H * nv if g_col >= 0 else 0, r_col + rank) > W:
+        raise KernelError("gated_linear_attention: the rows do not hold the products at the columns given")
+    for t, count in ((bias, H * n), (norm_weight, nv), (lower, H * n), (decay_matrix, H * n * rank)):
+        if t is not None and (t.dtype != torch.float32 or t.numel() != count or not t.is_contiguous()):
+            raise KernelError("gated_linear_attention: bias, lower bounds, decay matrix and norm weight are contiguous float32")
+    if state.dtype != torch.float32 or state.dim() != 2 or state.stride(1) != 1 or state.shape[1] < H * n * nv:
+        raise KernelError(f"gated_linear_attention: the state slab is float32 [slots, >= {H * n * nv}]")
+    if tuple(out.shape) != (T, H * nv) or not out.is_contiguous():
+        raise KernelError(f"gated_linear_attention: out is {(T, H * nv)}")
+    a = _GlaArgs(_p(src), src.stride(0), q_col, k_col, v_col, g_col, 1 if lower is not None else 0, 1 if q_silu else 0, r_col, rank,
+                 float(q_scale), float(power), float(eps), 0.0, _p(bias), _p(lower), _p(decay_matrix), _p(norm_weight), _p(state),
+                 state.stride(0), _p(slots), _p(out), _dt(out), H, n, nv)
+    with phase("scan"):
+        if n_req:
+            _i32(reqs, "reqs")
+            _check(lib().bg_gla_walk(ctypes.byref(a), _p(reqs), n_req, _stream()), "gla_walk")
+        if n_chunks:
+            _i32(chunks, "chunks"); _i32(longs, "longs")
+            if chunks.shape[0] < n_chunks or longs.shape[0] < n_long or n_long < 1:
+                raise KernelError("gated_linear_attention: the lists of chunks and of long requests are shorter than their counts")
+            f32 = dict(dtype=torch.float32, device=out.device)
+            work, decay = torch.empty((n_chunks, H, n * nv), **f32), torch.empty((n_chunks, H, n), **f32)
+            alpha = torch.empty((T, H * n), **f32) if lower is None else None
+            _check(lib().bg_gla_chunked(ctypes.byref(a), T, _p(chunks), n_chunks, _p(longs), n_long, _p(work), _p(decay), _p(alpha),
+                                        _stream()), "gla_chunked")
+            count_launches(2 if lower is not None else 3)
 
 
 # ---------------------------------------------------------------------------------------------------- routed experts
@@ -1464,39 +1572,44 @@ def route_logits(h: torch.Tensor, router: torch.Tensor, out: torch.Tensor) -> No
         _check(lib().bg_route_logits(_p(h), _dt(h), h.stride(0), _p(router), d, _p(out), E, T, E, d, _stream()), "route_logits")
 
 
-ROUTER_MODES = {"none": 0, "sigmoid": 1, "softmax": 2}
+ROUTER_MODES = {"none": 0, "sigmoid": 1, "softmax": 2, "softmax_chosen": 3}
 
 
-def _route_rule(E: int, sigmoid, bias: Optional[torch.Tensor], what: str) -> int:
-    """The kernels' score mode from `sigmoid` (True, False, or one of ROUTER_MODES), with the choice bias checked."""
+def _route_rule(E: int, sigmoid, bias: Optional[torch.Tensor], what: str, logit_bias: Optional[torch.Tensor] = None) -> int:
+    """The kernels' score mode from `sigmoid` (True, False, or one of ROUTER_MODES), with the biases checked."""
     mode = ROUTER_MODES[sigmoid] if isinstance(sigmoid, str) else (1 if sigmoid else 0)
-    if bias is not None and (bias.dtype != torch.float32 or bias.numel() != E or not bias.is_contiguous()):
-        raise KernelError(f"{what}: the choice bias is contiguous float32, one number per expert")
+    for b in (bias, logit_bias):
+        if b is not None and (b.dtype != torch.float32 or b.numel() != E or not b.is_contiguous()):
+            raise KernelError(f"{what}: a bias is contiguous float32, one number per expert")
+    if mode == 3 and bias is not None:
+        raise KernelError(f"{what}: the softmax over the chosen logits takes no choice bias")
     return mode
 
 
 def route_topk(logits: torch.Tensor, top: int, ids: torch.Tensor, weights: torch.Tensor, sigmoid=True,
-               renorm: bool = False, bias: Optional[torch.Tensor] = None, scale: float = 1.0) -> None:
+               renorm: bool = False, bias: Optional[torch.Tensor] = None, scale: float = 1.0,
+               logit_bias: Optional[torch.Tensor] = None) -> None:
     """Per row of float logits [T, E]: the `top` experts of largest score into ids [T, top] (int32) and their scores
-    into weights [T, top] (float32).  `sigmoid` may name the score: "none", "sigmoid" or "softmax" (over all E).  `bias`
-    [E] is added to the scores for the choice only; `scale` multiplies the weights."""
-    _cuda(logits, ids, weights)
+    into weights [T, top] (float32).  `sigmoid` may name the score: "none", "sigmoid", "softmax" (over all E) or
+    "softmax_chosen" (over the chosen logits only).  `bias` [E] is added to the scores for the choice only; `logit_bias` [E] is
+    part of the logits; `scale` multiplies the weights."""
+    _cuda(logits, ids, weights, bias, logit_bias)
     T, E = logits.shape
     _i32(ids, "ids")
     if logits.dtype != torch.float32 or weights.dtype != torch.float32 or not logits.is_contiguous() \
             or tuple(ids.shape) != (T, top) or tuple(weights.shape) != (T, top) or not ids.is_contiguous() or not weights.is_contiguous():
         raise KernelError("route_topk: logits float32 [T, E], ids int32 [T, top], weights float32 [T, top]")
     with phase("router"):
-        _check(lib().bg_route_topk(_p(logits), T, E, top, _route_rule(E, sigmoid, bias, "route_topk"), 1 if renorm else 0, _p(bias),
-                                   float(scale), _p(ids), _p(weights), _stream()), "route_topk")
+        _check(lib().bg_route_topk(_p(logits), T, E, top, _route_rule(E, sigmoid, bias, "route_topk", logit_bias),
+                                   1 if renorm else 0, _p(bias), float(scale), _p(logit_bias), _p(ids), _p(weights), _stream()), "route_topk")
 
 
 def route(h: torch.Tensor, router: torch.Tensor, top: int, ids: torch.Tensor, weights: torch.Tensor, sigmoid=True,
           renorm: bool = False, logits: Optional[torch.Tensor] = None, bias: Optional[torch.Tensor] = None,
-          scale: float = 1.0) -> None:
+          scale: float = 1.0, logit_bias: Optional[torch.Tensor] = None) -> None:
     """`route_logits` and `route_topk` as one kernel: h [T, d] in either type, router float32 [E, d], ids int32 [T, top],
-    weights float32 [T, top]; `logits`, when given, receives the float logits [T, E]."""
-    _cuda(h, router, ids, weights, logits, bias)
+    weights float32 [T, top]; `logits`, when given, receives the float logits [T, E] (without `logit_bias`)."""
+    _cuda(h, router, ids, weights, logits, bias, logit_bias)
     T, d = h.shape
     E = router.shape[0]
     _i32(ids, "ids")
@@ -1507,8 +1620,8 @@ def route(h: torch.Tensor, router: torch.Tensor, top: int, ids: torch.Tensor, we
     if logits is not None and (logits.dtype != torch.float32 or tuple(logits.shape) != (T, E) or not logits.is_contiguous()):
         raise KernelError("route: logits float32 [T, E]")
     with phase("router"):
-        _check(lib().bg_route(_p(h), _dt(h), h.stride(0), _p(router), T, d, E, top, _route_rule(E, sigmoid, bias, "route"),
-                              1 if renorm else 0, _p(bias), float(scale), _p(ids), _p(weights), _p(logits), _stream()), "route")
+        _check(lib().bg_route(_p(h), _dt(h), h.stride(0), _p(router), T, d, E, top, _route_rule(E, sigmoid, bias, "route", logit_bias),
+                              1 if renorm else 0, _p(bias), float(scale), _p(logit_bias), _p(ids), _p(weights), _p(logits), _stream()), "route")
 
 
 def route_sort(ids: torch.Tensor, E: int, offsets: torch.Tensor, row_of: torch.Tensor, src_of: torch.Tensor) -> None:

@@ -1,5 +1,5 @@
 // Small kernels around the residual stream and the activations that the Qwen2 parts do not have:
-// the centred norm (LayerNorm without a shift) with the residual add in front of it, the depth-weighted average of the layer results,
+// the centred norm (LayerNorm, with or without a shift vector) with the residual add in front of it, the depth-weighted average of the layer results,
 // the xIELU activation, an RMS norm over a slice of a product's rows, and the per-head output gate.
 // All statistics and sums are float; every row's sums run in an order fixed by the sizes alone.
 #include "common.cuh"
@@ -8,12 +8,12 @@ namespace bg {
 
 // For output row r (source row s = rows ? rows[r] : r):
 //   v = x[s] + sum_p delta[p][s];  if update: x[s] = v;
-//   out[r] = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * w
+//   out[r] = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * w (+ b)
 // One block per row; the row is held in shared memory between the passes (sum, squared deviations, output).
 template <typename TD, typename TW, typename TO>
 __global__ void add_layernorm_kernel(float* __restrict__ x, const TD* __restrict__ delta, int parts, size_t part_stride,
                                      const TW* __restrict__ w, float eps, TO* __restrict__ out,
-                                     const int* __restrict__ rows, int d, int update) {
+                                     const int* __restrict__ rows, int d, int update, const TW* __restrict__ b) {
     extern __shared__ float row_buf[];
     __shared__ float red[32];
     pdl_launch();
@@ -40,7 +40,7 @@ __global__ void add_layernorm_kernel(float* __restrict__ x, const TD* __restrict
     const float inv = 1.0f / sqrtf(sq / (float)d + eps);
     TO* o = out + (size_t)r * d;
     for (int i = threadIdx.x; i < d; i += blockDim.x)
-        o[i] = from_float<TO>((row_buf[i] - mean) * inv * to_float(w[i]));
+        o[i] = from_float<TO>((row_buf[i] - mean) * inv * to_float(w[i]) + (b ? to_float(b[i]) : 0.0f));
 }
 
 // The same for a width that is a multiple of 8 with rows on 16-byte boundaries: a thread holds up to ITER runs of eight
@@ -50,7 +50,7 @@ template <typename TD, typename TW, typename TO, int ITER>
 __global__ void __launch_bounds__(256)
 add_layernorm_vec8_kernel(float* __restrict__ x, const TD* __restrict__ delta, int parts, size_t part_stride,
                           const TW* __restrict__ w, float eps, TO* __restrict__ out, const int* __restrict__ rows, int d,
-                          int update) {
+                          int update, const TW* __restrict__ b) {
     __shared__ float red[32];
     pdl_launch();
     pdl_wait();
@@ -98,6 +98,11 @@ add_layernorm_vec8_kernel(float* __restrict__ x, const TD* __restrict__ delta, i
             load8(w + c * 8, wv);
 #pragma unroll
             for (int k = 0; k < 8; ++k) ov[k] = (v[it][k] - mean) * inv * wv[k];
+            if (b) {
+                load8(b + c * 8, wv);
+#pragma unroll
+                for (int k = 0; k < 8; ++k) ov[k] += wv[k];
+            }
             store8(o + c * 8, ov);
         }
     }
@@ -264,17 +269,17 @@ using namespace bg;
 
 template <typename TD, typename TW>
 static int add_layernorm_out(float* x, const void* delta, int parts, size_t part_stride, const void* w, float eps, void* out,
-                             int out_dtype, const int* rows, int n_rows, int d, int update, cudaStream_t stream) {
+                             int out_dtype, const int* rows, int n_rows, int d, int update, const void* b, cudaStream_t stream) {
     const size_t smem = (size_t)d * sizeof(float);
     if (smem > 200 * 1024) return BG_ERR_SHAPE;
     const bool vec = (d % 8 == 0) && (part_stride % 8 == 0) && ((uintptr_t)x % 16 == 0) && ((uintptr_t)delta % 16 == 0) &&
-                     ((uintptr_t)w % 16 == 0) && ((uintptr_t)out % 16 == 0) && d <= 8192;
+                     ((uintptr_t)w % 16 == 0) && ((uintptr_t)out % 16 == 0) && ((uintptr_t)b % 16 == 0) && d <= 8192;
     if (vec) {
         const int iter = (d / 8 + 255) / 256;
         BG_DISPATCH_DTYPE(out_dtype, TO, {
-            if (iter <= 1) launch(add_layernorm_vec8_kernel<TD, TW, TO, 1>, dim3(n_rows), dim3(256), 0, stream, x, (const TD*)delta, parts, part_stride, (const TW*)w, eps, (TO*)out, rows, d, update);
-            else if (iter <= 2) launch(add_layernorm_vec8_kernel<TD, TW, TO, 2>, dim3(n_rows), dim3(256), 0, stream, x, (const TD*)delta, parts, part_stride, (const TW*)w, eps, (TO*)out, rows, d, update);
-            else launch(add_layernorm_vec8_kernel<TD, TW, TO, 4>, dim3(n_rows), dim3(256), 0, stream, x, (const TD*)delta, parts, part_stride, (const TW*)w, eps, (TO*)out, rows, d, update);
+            if (iter <= 1) launch(add_layernorm_vec8_kernel<TD, TW, TO, 1>, dim3(n_rows), dim3(256), 0, stream, x, (const TD*)delta, parts, part_stride, (const TW*)w, eps, (TO*)out, rows, d, update, (const TW*)b);
+            else if (iter <= 2) launch(add_layernorm_vec8_kernel<TD, TW, TO, 2>, dim3(n_rows), dim3(256), 0, stream, x, (const TD*)delta, parts, part_stride, (const TW*)w, eps, (TO*)out, rows, d, update, (const TW*)b);
+            else launch(add_layernorm_vec8_kernel<TD, TW, TO, 4>, dim3(n_rows), dim3(256), 0, stream, x, (const TD*)delta, parts, part_stride, (const TW*)w, eps, (TO*)out, rows, d, update, (const TW*)b);
         });
         BG_LAUNCH_CHECK();
         return BG_OK;
@@ -283,21 +288,21 @@ static int add_layernorm_out(float* x, const void* delta, int parts, size_t part
         auto kern = add_layernorm_kernel<TD, TW, TO>;
         if (smem > BG_SMEM_OPT_IN) cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         launch(kern, dim3(n_rows), dim3(256), smem, stream, x, (const TD*)delta, parts, part_stride, (const TW*)w, eps,
-               (TO*)out, rows, d, update);
+               (TO*)out, rows, d, update, (const TW*)b);
     });
     BG_LAUNCH_CHECK();
     return BG_OK;
 }
 
-// The arguments of bg_add_rmsnorm, for the centred norm (scale vector, no shift).
+// The arguments of bg_add_rmsnorm, for the centred norm (scale vector and, unless null, a shift vector b of its type).
 extern "C" int bg_add_layernorm(float* x, const void* delta, int delta_dtype, int parts, long long part_stride,
                                 const void* w, int w_dtype, float eps, void* out, int out_dtype, const int* rows,
-                                int n_rows, int d, int update, cudaStream_t stream) {
+                                int n_rows, int d, int update, const void* b, cudaStream_t stream) {
     if (n_rows <= 0) return BG_OK;
     if (!delta) { delta_dtype = BG_DTYPE_F32; parts = 0; }
     BG_DISPATCH_DTYPE(delta_dtype, TD, BG_DISPATCH_DTYPE(w_dtype, TW,
         return (add_layernorm_out<TD, TW>(x, delta, parts, (size_t)part_stride, w, eps, out, out_dtype, rows, n_rows, d,
-                                          update, stream))));
+                                          update, b, stream))));
     return BG_OK;
 }
 

@@ -86,7 +86,8 @@ class Engine:
         QWEN_HF_CONFIG, qwen_infer.c:20121)."""
         ckpt = Checkpoint(folder)
         try:
-            arch, cfg = load_config(config_path or folder, tensor_names=ckpt.names())
+            # (a size that config.json leaves to a tensor's shape is read off there)
+            arch, cfg = load_config(config_path or folder, tensor_names={n: tuple(ckpt.shape(n)) for n in ckpt.names()})
             return cls(arch.build_spec(cfg), ckpt, config=cfg, origin=folder, **kw)
         finally:
             ckpt.close()

@@ -43,8 +43,13 @@ class DecoderModel:
                     if entry.names[role.name] in tensors}
             self.entries.append(cls(entry.part, mine, ctx))
         self.keep_origin = any(getattr(e, "needs_origin", False) for e in self.entries)
-        self.final_norm = registry.norm_class(spec.final_norm.kind)(
-            spec.final_norm, {"weight": tensors[spec.final_norm_name]}, ctx)
+        self.positions = None if spec.position_name is None else ctx.matrix(tensors[spec.position_name])
+        mine = {"weight": tensors[spec.final_norm_name]}
+        if spec.final_norm_bias_name is not None:
+            mine["bias"] = tensors[spec.final_norm_bias_name]
+        if spec.logit_scale != 1.0:        # c E norm(x) = E (c norm(x)): the constant rides in the final norm's vectors, in float
+            mine = {k: t.float() * float(spec.logit_scale) for k, t in mine.items()}
+        self.final_norm = registry.norm_class(spec.final_norm.kind)(spec.final_norm, mine, ctx)
         head_bias = None if spec.head_bias_name is None else tensors[spec.head_bias_name]
         if spec.head_name is None:
             self.head = Linear(self.embed, head_bias, ctx, label="head_gemv")     # ctx.matrix is a no-op on the table: one copy
@@ -84,7 +89,7 @@ class DecoderModel:
                     walk(v, depth)
             elif depth < 3 and hasattr(obj, "__dict__"):
                 for k, v in vars(obj).items():
-                    if k in ("ctx", "spec", "bias_c", "embed"):
+                    if k in ("ctx", "spec", "bias_c", "embed", "positions"):
                         continue
                     walk(v, depth + 1)
 
@@ -105,7 +110,8 @@ class DecoderModel:
         float residual stream [T, hidden] as that stage leaves it (for looking into a model layer by layer; it
         reads what the stream still owes, so it is not for captured steps)."""
         x = torch.empty((batch.n_rows, self.spec.hidden), dtype=torch.float32, device=self.ctx.device)
-        ops.embed_gather(self.embed, batch.token_ids, x, self.ctx.status, scale=self.spec.embed_scale)
+        ops.embed_gather(self.embed, batch.token_ids, x, self.ctx.status, scale=self.spec.embed_scale, pos_table=self.positions,
+                         positions=batch.positions if self.positions is not None else None)
         stream = ResidualStream(x)
         if self.keep_origin:
             stream.origin = x.clone()
@@ -130,7 +136,7 @@ class DecoderModel:
                     rows += stream.pending.float().reshape(-1, *rows.shape).sum(0)
                 if stream.terms is not None:
                     for t, c in stream.terms.items:
-                        rows += c * t.float().reshape(-1, *rows.shape).sum(0)
+                        rows += c * t.float().reshape(-1, *rows.shape).sum(0)      # (a normed term's float() is its normed rows)
                 tap(si, rows)
         if batch.n_logit_rows == 0:
             return None

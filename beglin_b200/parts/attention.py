@@ -10,7 +10,8 @@ product.  All rows' keys and values are in the cache before any row's attention 
 Options of the spec, each off for the plain form: values of another size than keys; an RMS norm of the whole query
 row and of the whole key row of a token before the rotation, or of every head by itself; a softmax whose denominator is
 enlarged by one, or by exp of a learned number per head; scores squashed by c tanh(s / c); queries that see the keys of their
-own block of positions only; a gate, sigmoid of a further
+own block of positions only; scores that fall with the distance by a slope per head; a window that never loses the first few
+positions; a gate, sigmoid of a further
 product of the mixer's input, on the joined heads before the output product, feature by feature or one number per head.  The gate's matrix is
 one more block of rows of the one q/k/v product.  With any of the first two the kernel that norms, rotates and appends
 is `qk_norm_rope_append`.
@@ -72,7 +73,7 @@ class GQAAttention:
         if ctx is None or ctx.compute_dtype != torch.bfloat16 or ctx.attention == "generic":
             return None
         hd, vd = spec.head_dim, spec.value_dim
-        if spec.qk_norm is None and vd == hd and spec.gate is None:
+        if spec.qk_norm is None and vd == hd and spec.gate is None and spec.slopes is None:
             return None                        # the plain form keeps its layout
         if hd == vd and hd in (64, 128):
             return None
@@ -85,15 +86,15 @@ class GQAAttention:
             return None
         stored = GQAAttention.stored_head(spec, ctx)
         if stored is not None:
-            return PagedKVNeed(spec.n_kv_heads, stored, spec.window, None, spec.block)
+            return PagedKVNeed(spec.n_kv_heads, stored, spec.window, None, spec.block, spec.keep_first)
         return PagedKVNeed(spec.n_kv_heads, spec.head_dim, spec.window,
-                           None if spec.value_dim == spec.head_dim else spec.value_dim, spec.block)
+                           None if spec.value_dim == spec.head_dim else spec.value_dim, spec.block, spec.keep_first)
 
     def __init__(self, spec: AttentionSpec, tensors: Dict[str, torch.Tensor], ctx: BuildContext):
         if spec.n_heads % spec.n_kv_heads:
             raise ValueError(f"{spec.n_heads} query heads are not a multiple of {spec.n_kv_heads} kv heads")
-        if spec.head_dim % 2 or spec.head_dim > 256:
-            raise ValueError(f"head_dim={spec.head_dim} must be even and at most 256")
+        if (spec.head_dim % 2 and spec.position.kind != "none") or not 0 < spec.head_dim <= 256:
+            raise ValueError(f"head_dim={spec.head_dim} must be even (where it is rotated) and at most 256")
         self.spec, self.ctx = spec, ctx
         if spec.qk_norm not in (None, "projection", "head"):
             raise ValueError(f"unknown query/key norm '{spec.qk_norm}' (projection, head)")
@@ -109,7 +110,7 @@ class GQAAttention:
         self.qd, self.kvd = self.nh * self.hd, self.nkv * self.hd
         self.od = self.nh * self.vd
         # what the plain form does not have: the step between product and attention is then a kernel of its own
-        self.extended = spec.qk_norm is not None or self.vd != self.hd or spec.gate is not None
+        self.extended = spec.qk_norm is not None or self.vd != self.hd or spec.gate is not None or spec.slopes is not None
         if self.extended and not spec.own_kv:
             raise ValueError("the extended attention has a cache of its own")
         names = ["q_proj"] + (["k_proj", "v_proj"] if spec.own_kv else [])
@@ -142,6 +143,11 @@ class GQAAttention:
                                             learned_sink=self.sink_weight is not None) for d in (False, True)}
         if spec.block is not None and (spec.window is not None or spec.block <= 0):
             raise ValueError("blocks of positions stand in place of a window and hold at least one position")
+        if spec.keep_first < 0 or (spec.keep_first and spec.window is None):
+            raise ValueError("kept first positions go with a window")
+        if spec.slopes is not None and len(spec.slopes) != spec.n_heads:
+            raise ValueError(f"{len(spec.slopes)} slopes for {spec.n_heads} query heads")
+        self.slopes = None if spec.slopes is None else torch.tensor(spec.slopes, dtype=torch.float64).to(torch.float32).to(ctx.device)
         # what the kernels are told: a positive number is a sliding window, a negative one the size of the blocks
         self.window = int(spec.window) if spec.window else (-int(spec.block) if spec.block else 0)
         # the fused q/k/v product can rotate and append itself: whole heads rotated in halves, a cache of its own
@@ -186,15 +192,16 @@ class GQAAttention:
         ops.attention(q, q.stride(0), cache.pool, cache.block_table, batch.positions, qblk, n_qblk,
                       batch.max_position, T, self.nh, self.nkv, khd, self.window, self.ctx.kv_split, tile, bq,
                       self.scale, out, self.ctx.status, kernel, vd=kvd_, sink=bool(self.spec.sink),
-                      sink_weight=self.sink_weight, softcap=self.score_cap)
+                      sink_weight=self.sink_weight, softcap=self.score_cap, keep=self.spec.keep_first, slopes=self.slopes)
         gate_per = self.vd if self.spec.gate == "head" else 1      # one gate per head, or one per feature
         if self.spec.gate is not None and self.stored is None:
             ops.sigmoid_gate(out, qkv, self.gate_col, self.od, gate_per=gate_per)
         elif self.spec.gate is not None:               # the gate's kernel also drops the zeros behind every head
             wide, out = out, torch.empty((T, self.od), dtype=self.ctx.compute_dtype, device=q.device)
             ops.sigmoid_gate(out, qkv, self.gate_col, self.od, src=wide, vd=self.vd, head_stride=self.stored, gate_per=gate_per)
-        elif self.stored is not None:
-            out = out.view(T, self.nh, self.stored)[:, :, :self.vd].reshape(T, self.od)
+        elif self.stored is not None:                  # no gate: the same kernel drops the zeros
+            wide, out = out, torch.empty((T, self.od), dtype=self.ctx.compute_dtype, device=q.device)
+            ops.gate_heads(wide.view(T, self.nh, self.stored).transpose(0, 1)[:, :, :self.vd], None, 0, out)
         if stream is None:
             return self.o_proj.partial(out)
         self.o_proj.into(out, stream)

@@ -129,9 +129,9 @@ class ParallelBlock:
 
     def normed(self, stream: ResidualStream):
         """(norm1(x), norm2(x) or None) of the stream with everything it is owed added."""
-        n1, n2 = self.mixer_norm, self.feed_forward_norm if self.feed_forward is not None else None
-        one_kernel = getattr(n1, "kind", None) == "rmsnorm" and (n2 is None or (
-            getattr(n2, "kind", None) == "rmsnorm" and n2.spec.eps == n1.spec.eps and n2.weight.dtype == n1.weight.dtype))
+        n1, n2 = self.mixer_norm, self.feed_forward_norm
+        one_kernel = getattr(n1, "kind", None) in ("rmsnorm", "layernorm") and (n2 is None or (
+            getattr(n2, "kind", None) == n1.kind and n2.spec.eps == n1.spec.eps and n2.weight.dtype == n1.weight.dtype))
         if not one_kernel:
             stream.settle()
             h1 = NormedInput(stream, n1).tensor()
@@ -143,12 +143,15 @@ class ParallelBlock:
         h1 = torch.empty(x.shape, dtype=dtype, device=x.device)
         h2 = torch.empty(x.shape, dtype=dtype, device=x.device) if n2 is not None else None
         ops.add_terms_norm(x, terms, weight1=n1.weight, weight2=n2.weight if n2 is not None else None, eps=n1.spec.eps,
-                           out1=h1, out2=h2)
+                           out1=h1, out2=h2, center=n1.kind == "layernorm", bias1=getattr(n1, "bias", None),
+                           bias2=getattr(n2, "bias", None))
         stream.pending, stream.terms, stream.ssq, stream.lowp = None, None, None, None
         return h1, h2
 
     def forward(self, stream: ResidualStream, batch, cache) -> None:
         h1, h2 = self.normed(stream)
+        if h2 is None:
+            h2 = h1                        # a layer with one norm: both sublayers read its rows
         owed = Terms()
         if getattr(self.mixer, "takes_stream", False):
             owed.add(self.mixer.forward(h1, batch, cache, None), self.mult)
@@ -166,3 +169,9 @@ class ParallelBlock:
 class ParallelMixerBlock(ParallelBlock):
     """The same layer without a feed-forward: x <- x + m mixer(norm1(x))."""
     SLOTS = (("mixer_norm", "norm"), ("mixer", "mixer"))
+
+
+@register_block("parallel_shared")
+class ParallelSharedBlock(ParallelBlock):
+    """The parallel layer with ONE norm, whose rows both sublayers read: h = norm(x), x <- x + m (mixer(h) + feed_forward(h))."""
+    SLOTS = (("mixer_norm", "norm"), ("mixer", "mixer"), ("feed_forward", "feed_forward"))

@@ -16,12 +16,14 @@ import torch
 class PagedKVNeed:
     """Keys and values of every position (window None) or of the last `window` positions.  `v_head_dim` is given
     when values have another size than keys.  `block` b: a query reads only the positions of its own block of b positions
-    (blocks counted from position 0), so the pages wholly in front of the newest block are given back."""
+    (blocks counted from position 0), so the pages wholly in front of the newest block are given back.  `keep_first` k: the
+    positions 0 .. k - 1 stay readable beside the window, so the pages that hold them are never given back."""
     n_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     v_head_dim: Optional[int] = None
     block: Optional[int] = None
+    keep_first: int = 0
 
     def page_shape(self, page_size: int) -> Tuple[int, ...]:
         """What one page of one stage holds: (2 = keys, values; kv heads; positions; features); with values of

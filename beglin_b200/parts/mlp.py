@@ -59,8 +59,8 @@ class SwiGLU:
 
 @register_feed_forward("dense_act")
 class DenseAct:
-    """m = W_down act(W_up h): one hidden layer without a gate branch.  The activation (xIELU, the tanh form of GELU or
-    silu) is a kernel of its own between the two products; it reads the up product's result (or its partial sums) as floats and writes
+    """m = W_down act(W_up h): one hidden layer without a gate branch.  The activation (xIELU, the tanh form of GELU, silu
+    or the square of relu) is a kernel of its own between the two products; it reads the up product's result (or its partial sums) as floats and writes
     the compute type."""
 
     @staticmethod
@@ -72,9 +72,9 @@ class DenseAct:
         return roles
 
     def __init__(self, spec: DenseActSpec, tensors: Dict[str, torch.Tensor], ctx: BuildContext):
-        if spec.activation != "xielu" and spec.activation not in ops.GLU_ACTIVATIONS:
+        if spec.activation != "xielu" and spec.activation not in ops.ACTIVATIONS:
             raise ValueError(f"unknown activation '{spec.activation}' of a dense feed-forward "
-                             f"(xielu, {', '.join(ops.GLU_ACTIVATIONS)})")
+                             f"(xielu, {', '.join(ops.ACTIVATIONS)})")
         self.spec, self.ctx = spec, ctx
         self.up = Linear(tensors["up.weight"], None, ctx, label="proj_up")
         self.down = Linear(tensors["down.weight"], None, ctx, label="proj_down")

@@ -5,7 +5,8 @@ The branches are ordinary mixers of the registry (attention, a recurrence, ...),
 tensors are called `<label i>.<name>`.  Each branch has the cache its kind asks for: the stage's need is the composite
 of the branches' needs, and the stage's view is the tuple of their views.  The sum is float: the part hands the block
 its branches' results as terms (result, constant), and the kernel that adds a layer's results to the stream adds them
-one by one, so the branches' results are never rounded to a sum of their own.
+one by one, so the branches' results are never rounded to a sum of their own.  Branches whose results are normed before they
+are added hand them on un-normed, with the norm's weight: the same kernel norms them as it adds.
 """
 from __future__ import annotations
 
@@ -17,7 +18,7 @@ from . import registry
 from .cache_need import CompositeNeed
 from .context import BuildContext
 from .spec import ParallelMixersSpec, TensorRole
-from .stream import NormedInput, Terms
+from .stream import NormedInput, NormedTerm, Terms
 
 
 @registry.register_mixer("parallel_mixers")
@@ -34,6 +35,8 @@ class ParallelMixers:
         for label, cls, b in ParallelMixers._branches(spec):
             for r in cls.expected_tensors(b):
                 roles.append(TensorRole(f"{label}.{r.name}", r.shape, r.required, r.matrix, r.role))
+            if spec.out_norm_eps is not None:
+                roles.append(TensorRole(f"{label}.out_norm.weight", (spec.hidden,), role="scale"))
         return roles
 
     cache_need_takes_context = True
@@ -52,6 +55,8 @@ class ParallelMixers:
             mine = {name[len(label) + 1:]: t for name, t in tensors.items() if name.startswith(label + ".")}
             self.parts.append(cls(b, mine, ctx))
         self.scales = [float(c) for c in spec.scales]
+        self.out_norms = [tensors[f"{label}.out_norm.weight"].to(device=ctx.device, dtype=torch.float32).contiguous()
+                          for label in spec.labels] if spec.out_norm_eps is not None else None
 
     takes_stream = True
     gives_terms = True         # forward returns Terms: (result, constant) per branch, to be summed in float by the block
@@ -61,10 +66,12 @@ class ParallelMixers:
             h = h.tensor()
         views = cache if cache is not None else (None,) * len(self.parts)
         terms = Terms()
-        for part, view, scale in zip(self.parts, views, self.scales):
+        for i, (part, view, scale) in enumerate(zip(self.parts, views, self.scales)):
             if getattr(part, "takes_stream", False):
                 a = part.forward(h, batch, view, None)
             else:
                 a = part.forward(h, batch, view)
+            if self.out_norms is not None:
+                a = NormedTerm(a, self.out_norms[i], self.spec.out_norm_eps)
             terms.add(a, scale)
         return terms

@@ -33,12 +33,13 @@ class TensorRole:
 @dataclass(frozen=True)
 class NormSpec:
     """kind "rmsnorm": x * rsqrt(mean(x^2) + eps) * w.  kind "layernorm": centred first,
-    c = x - mean(x), then c * rsqrt(mean(c^2) + eps) * w; there is no shift vector.  `offset` o (rmsnorm): the stored
+    c = x - mean(x), then c * rsqrt(mean(c^2) + eps) * w, with `shift` + b (tensor `bias`).  `offset` o (rmsnorm): the stored
     weight lies around zero and the rows are multiplied by o + w, the sum formed in float."""
     size: int
     eps: float
     kind: str = "rmsnorm"
     offset: float = 0.0
+    shift: bool = False
 
 
 @dataclass(frozen=True)
@@ -76,7 +77,9 @@ class AttentionSpec:
     the queries and of the keys is RMS-normed by itself, with one weight vector of head_dim values for all query heads and one
     for all key heads.  `sink` "learned": the extra key's score is a learned number per query head (tensor `sink`) in place
     of 0.  `score_cap` c: a scaled score s becomes c tanh(s / c) before the softmax.  `block` b (in place of a window): a query
-    at position i sees the keys j <= i with floor(j / b) = floor(i / b), blocks counted from position 0 of the sequence."""
+    at position i sees the keys j <= i with floor(j / b) = floor(i / b), blocks counted from position 0 of the sequence.
+    `keep_first` k (beside a window): the positions 0 .. k - 1 stay visible however far they lie back.  `slopes`: one number
+    per query head; a scaled score falls by it for every position that its key lies behind the query."""
     hidden: int
     n_heads: int
     n_kv_heads: int
@@ -94,6 +97,8 @@ class AttentionSpec:
     gate: Optional[str] = None             # None, "elementwise" or "head"
     score_cap: Optional[float] = None      # None: scores as they are
     block: Optional[int] = None            # None: no blocks of positions
+    keep_first: int = 0                    # 0: a window keeps no position for good
+    slopes: Optional[Tuple[float, ...]] = None
     kind: str = "gqa_attention"
 
     @property
@@ -123,7 +128,11 @@ class RoutedExpertsSpec:
     router outputs.  `choice_bias`: a learned number per router output (tensor `router.bias`) is added to the scores when
     the experts are chosen, and plays no part in the weights.  `route_scale` multiplies the weights.  `identity` n: the
     router has `experts` + n outputs, and the last n stand for experts without weights that return their input.
-    `shared`: an expert that every token passes, added to the sum."""
+    `shared`: an expert that every token passes, added to the sum.
+
+    `activation` "swiglu": an expert has a gate branch, down(silu(gate(h)) * up(h)).  `router_activation` "softmax_chosen": the
+    weights are the softmax over the chosen logits only.  `logit_bias`: a learned number per router output (tensor
+    `router.logit_bias`) that is part of the logits."""
     hidden: int
     intermediate: int
     experts: int
@@ -137,6 +146,7 @@ class RoutedExpertsSpec:
     route_scale: float = 1.0
     identity: int = 0
     shared: Optional[SharedExpertSpec] = None
+    logit_bias: bool = False
     kind: str = "routed_experts"
 
 
@@ -198,14 +208,39 @@ class DecayAttentionSpec:
 
 
 @dataclass(frozen=True)
+class GatedLinearAttentionSpec:
+    """Linear attention with a decay per key channel: `n_heads` heads with queries of `dim` features and values of `vdim`; per
+    head a state S <- diag(a) S + k v^T [dim, vdim] that is read out as S^T q.  q is `query_scale` times a product of the
+    mixer's input, or times its silu (`query_silu`).  `write` "forget": one product f, with a bias and a lower bound l per
+    channel, gives a = l + (1 - l) sigmoid(f) and k = 1 - a.  `write` "key": k is a product of its own, and
+    a = sigmoid(z)^`decay_power` with z = W2 (W1 h) + bias through `decay_rank` features.  Every head's result is RMS-normed by
+    itself (one weight vector of `vdim` values, `eps`); with `gated` the joined heads are multiplied by silu of a further
+    product; then they are projected."""
+    hidden: int
+    n_heads: int
+    dim: int
+    vdim: int
+    eps: float
+    write: str = "forget"
+    query_silu: bool = False
+    query_scale: float = 1.0
+    decay_rank: int = 0
+    decay_power: float = 1.0
+    gated: bool = False
+    kind: str = "gated_linear_attention"
+
+
+@dataclass(frozen=True)
 class ParallelMixersSpec:
     """Several mixers side by side that read the same input; the result is sum_i scales[i] * mixer_i(h).  `labels` name the
     branches: branch i's tensors are called `<labels[i]>.<the mixer's own name>`.  Every branch has a cache of its own
-    kind (pages, state) or none."""
+    kind (pages, state) or none.  `out_norm_eps`: every branch's result is RMS-normed over the width first, with a weight of
+    its own (tensor `<labels[i]>.out_norm.weight`)."""
     hidden: int
     branches: Tuple[object, ...]
     scales: Tuple[float, ...]
     labels: Tuple[str, ...]
+    out_norm_eps: Optional[float] = None
     kind: str = "parallel_mixers"
 
 
@@ -245,15 +280,15 @@ class SharedExpertSpec:
     """An expert of the routed experts' form that every token passes; its result is multiplied by sigmoid of one number per
     token, a product of the feed-forward's input, when `gated`."""
     intermediate: int
-    limit: float
+    limit: float = 0.0                     # of the clamped activation; the others have none
     gated: bool = True
 
 
 @dataclass(frozen=True)
 class DenseActSpec:
     """Feed-forward with one hidden layer, down(act(up(h))), no gate branch.  `activation` "xielu": a parabola
-    above zero and a scaled exponential below, with two learned numbers (tensor `act`); "gelu_tanh" and "silu" have no
-    tensor of their own."""
+    above zero and a scaled exponential below, with two learned numbers (tensor `act`); "gelu_tanh", "silu" and "relu2" (the
+    square of relu) have no tensor of their own."""
     hidden: int
     intermediate: int
     activation: str = "xielu"
@@ -345,3 +380,6 @@ class ModelSpec:
     #                                       the final norm reads their sum (blocks of a "lanes" kind tie the sublayers to them)
     extra: Dict[str, object] = field(default_factory=dict)
     entries: List[EntrySpec] = field(default_factory=list)   # parts that stages name in `enter`
+    position_name: Optional[str] = None   # a table [max_positions, hidden] whose row of the token's position joins the embedded row
+    final_norm_bias_name: Optional[str] = None
+    logit_scale: float = 1.0              # multiplies the logits

@@ -10,6 +10,7 @@ the layer (the norms) and their launches are gone.
 """
 from __future__ import annotations
 
+from dataclasses import dataclass
 from typing import Optional
 
 import torch
@@ -29,6 +30,19 @@ class Terms:
 
     def scaled(self, scale: float) -> "Terms":
         return Terms([(t, c * scale) for t, c in self.items])
+
+
+@dataclass
+class NormedTerm:
+    """A result that is RMS-normed over its rows (weight float32, eps) before it is added: in the place of a term's tensor."""
+    rows: torch.Tensor                                 # [T, d] or partial sums [parts, T, d]
+    weight: torch.Tensor
+    eps: float
+
+    def float(self) -> torch.Tensor:
+        """The normed rows, formed by torch operations (for looking into a model; the kernels norm as they add)."""
+        v = self.rows.float().reshape(-1, *self.rows.shape[-2:]).sum(0)
+        return v * torch.rsqrt((v * v).mean(-1, keepdim=True) + self.eps) * self.weight
 
 
 class ResidualStream:

@@ -48,6 +48,8 @@ def expected_tensors(spec: ModelSpec) -> Dict[str, TensorRole]:
     import beglin_b200.parts  # noqa: F401  (registers the built-in parts)
     out: Dict[str, TensorRole] = {}
     out[spec.embed_name] = TensorRole(spec.embed_name, (spec.vocab, spec.hidden), True, True)
+    if spec.position_name is not None:
+        out[spec.position_name] = TensorRole(spec.position_name, (spec.max_positions, spec.hidden), True, True)
     for li, layer in enumerate(spec.layers):
         for qualified, role in layer_roles(layer):
             if qualified not in layer.names:
@@ -60,8 +62,8 @@ def expected_tensors(spec: ModelSpec) -> Dict[str, TensorRole]:
             out[entry.names[role.name]] = role
     norm_cls = registry.norm_class(spec.final_norm.kind)
     for role in norm_cls.expected_tensors(spec.final_norm):
-        # a norm has one tensor, "weight"; the final norm's checkpoint name is given whole
-        out[spec.final_norm_name if role.name == "weight" else f"{spec.final_norm_name}.{role.name}"] = role
+        # the checkpoint names of the final norm's tensors, its weight and (a layer norm's) shift vector, are given whole
+        out[{"weight": spec.final_norm_name, "bias": spec.final_norm_bias_name}[role.name]] = role
     if spec.head_name is not None:
         out[spec.head_name] = TensorRole(spec.head_name, (spec.vocab, spec.hidden), True, True)
     if spec.head_bias_name is not None:
