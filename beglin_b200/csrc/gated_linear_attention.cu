@@ -86,33 +86,31 @@ __device__ __forceinline__ void gla_load_token(const GlaParams& p, const float* 
     for (int i = tid; i < nv; i += blockDim.x) vs[i] = row[p.v_col + h * nv + i];
 }
 
-// The state in registers: thread (slice, column) holds the rows slice, slice + slices, ... of its column, at most R of them.
-// `slices` threads share a column (blockDim.x / nv of them, whole columns only).
+// The state in registers: thread (slice, column) holds the R rows from slice R on of its column; `slices` threads share a
+// column (blockDim.x / nv of them, whole columns only, slices R >= n).  q, k and a are padded with zeros up to slices R, so
+// that a thread reads them four at a time and without a condition.
 template <int R>
-__global__ void __launch_bounds__(512) gla_walk_kernel(GlaParams p) {
-    extern __shared__ float ga_s[];
+__global__ void __launch_bounds__(512) gla_walk_kernel(GlaParams p, int slices) {
+    extern __shared__ __align__(16) float ga_s[];
     __shared__ float scratch[32];
-    const int n = p.n, nv = p.nv;
-    const int slices = (int)blockDim.x / nv;
-    float* qs = ga_s;                      // [n]
-    float* ks = qs + n;                    // [n]
-    float* as = ks + n;                    // [n]
-    float* vs = as + n;                    // [nv]
+    const int n = p.n, nv = p.nv, np = slices * R;
+    float* qs = ga_s;                      // [np]
+    float* ks = qs + np;                   // [np]
+    float* as = ks + np;                   // [np]
+    float* vs = as + np;                   // [nv]
     float* red = vs + nv;                  // [slices][nv]
     pdl_launch();
     const int h = blockIdx.x, r = blockIdx.y;
     const int req = p.reqs[r * 3 + 0], row0 = p.reqs[r * 3 + 1], rows = p.reqs[r * 3 + 2];
     const int tid = threadIdx.x;
-    const int sl = tid / nv, c = tid - sl * nv;
-    const bool own = sl < slices;
+    const int sl = tid / nv, c = tid - sl * nv, i0 = sl * R;
+    const bool own = sl < slices && rows > 0;
     // the state was left by an earlier step: it is on its way while the product ahead still runs
-    float* st = p.state + (size_t)p.slots[req] * p.slot_stride + (size_t)h * n * nv + c;
+    float* st = p.state + (size_t)p.slots[req] * p.slot_stride + (size_t)h * n * nv + (size_t)i0 * nv + c;
     float S[R];
 #pragma unroll
-    for (int k = 0; k < R; ++k) {
-        const int i = sl + k * slices;
-        S[k] = (own && rows > 0 && i < n) ? st[(size_t)i * nv] : 0.0f;
-    }
+    for (int k = 0; k < R; ++k) S[k] = (own && i0 + k < n) ? st[(size_t)k * nv] : 0.0f;
+    for (int i = n + tid; i < np; i += blockDim.x) { qs[i] = 0.0f; ks[i] = 0.0f; as[i] = 0.0f; }
     pdl_wait();
     if (rows <= 0) return;
     for (int t = 0; t < rows; ++t) {
@@ -122,16 +120,17 @@ __global__ void __launch_bounds__(512) gla_walk_kernel(GlaParams p) {
         __syncthreads();
         if (own) {
             const float v = vs[c];
-            float acc = 0.0f;
+            float acc0 = 0.0f, acc1 = 0.0f;
 #pragma unroll
-            for (int k = 0; k < R; ++k) {
-                const int i = sl + k * slices;
-                if (i < n) {
-                    S[k] = fmaf(as[i], S[k], ks[i] * v);
-                    acc = fmaf(S[k], qs[i], acc);
-                }
+            for (int k = 0; k < R; k += 4) {
+                const float4 a = *reinterpret_cast<const float4*>(as + i0 + k), kk = *reinterpret_cast<const float4*>(ks + i0 + k);
+                const float4 q = *reinterpret_cast<const float4*>(qs + i0 + k);
+                S[k + 0] = fmaf(a.x, S[k + 0], kk.x * v); acc0 = fmaf(S[k + 0], q.x, acc0);
+                S[k + 1] = fmaf(a.y, S[k + 1], kk.y * v); acc1 = fmaf(S[k + 1], q.y, acc1);
+                S[k + 2] = fmaf(a.z, S[k + 2], kk.z * v); acc0 = fmaf(S[k + 2], q.z, acc0);
+                S[k + 3] = fmaf(a.w, S[k + 3], kk.w * v); acc1 = fmaf(S[k + 3], q.w, acc1);
             }
-            red[tid] = acc;
+            red[sl * nv + c] = acc0 + acc1;
         }
         __syncthreads();
         float o = 0.0f;
@@ -142,11 +141,11 @@ __global__ void __launch_bounds__(512) gla_walk_kernel(GlaParams p) {
                       o * (1.0f / sqrtf(ss / (float)nv + p.eps)) * p.norm_w[tid] * gla_gate(p, row, h, tid));
     }
     if (own) {
+        int stride = nv;
+        asm volatile("" : "+r"(stride));   // the addresses are worked out again here: kept from the loads, they would fill the registers
 #pragma unroll
-        for (int k = 0; k < R; ++k) {
-            const int i = sl + k * slices;
-            if (i < n) st[(size_t)i * nv] = S[k];
-        }
+        for (int k = 0; k < R; ++k)
+            if (i0 + k < n) st[(size_t)k * stride] = S[k];
     }
 }
 
@@ -579,20 +578,21 @@ extern "C" int bg_gla_walk(const GlaArgs* args, const int* reqs, int n_req, cuda
     if (n_req > 65535) return BG_ERR_SHAPE;
     p.reqs = reqs;
     const dim3 grid(p.H, n_req);
-    // whole columns per block: 512 threads, fewer where a head has too few rows to give each some
+    // whole columns per block of up to 512 threads, four to 64 rows of its column a thread
     if (p.nv <= 512) {
-        int slices = 512 / p.nv;
-        const int few = (p.n + 7) / 8;                      // at least eight rows a thread where the head has them
-        if (slices > few) slices = few;
-        if (slices * p.nv < 32) slices = (32 + p.nv - 1) / p.nv;
+        int slices = 512 / p.nv, R = 4;
+        while (R < 64 && slices * R < p.n) R *= 2;
+        slices = (p.n + R - 1) / R < slices ? (p.n + R - 1) / R : slices;
         const int threads = (slices * p.nv + 31) / 32 * 32;
-        const int per = (p.n + threads / p.nv - 1) / (threads / p.nv);
-        const size_t smem = ((size_t)3 * p.n + p.nv + threads) * sizeof(float);
-        if (per <= 64 && threads <= 512 && smem <= 40 * 1024) {
-            if (per <= 8) launch(gla_walk_kernel<8>, grid, dim3(threads), smem, stream, p);
-            else if (per <= 16) launch(gla_walk_kernel<16>, grid, dim3(threads), smem, stream, p);
-            else if (per <= 32) launch(gla_walk_kernel<32>, grid, dim3(threads), smem, stream, p);
-            else launch(gla_walk_kernel<64>, grid, dim3(threads), smem, stream, p);
+        const size_t smem = ((size_t)3 * slices * R + p.nv + (size_t)slices * p.nv) * sizeof(float);
+        if (slices * R >= p.n && smem <= BG_SMEM_OPT_IN) {
+            switch (R) {
+                case 4: launch(gla_walk_kernel<4>, grid, dim3(threads), smem, stream, p, slices); break;
+                case 8: launch(gla_walk_kernel<8>, grid, dim3(threads), smem, stream, p, slices); break;
+                case 16: launch(gla_walk_kernel<16>, grid, dim3(threads), smem, stream, p, slices); break;
+                case 32: launch(gla_walk_kernel<32>, grid, dim3(threads), smem, stream, p, slices); break;
+                default: launch(gla_walk_kernel<64>, grid, dim3(threads), smem, stream, p, slices); break;
+            }
             BG_LAUNCH_CHECK();
             return BG_OK;
         }

@@ -430,10 +430,35 @@ def tuzupel_config(width, heads, layers, vocab=32768):
             "layers": [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": moe} for i in range(layers)]}
 
 
+# The Dinatar decoder beside another design at equal layer sizes (--design dinatar): layers in the order linear attention with a
+# forget gate, two mixers side by side, linear attention with rooted decays, side by side, ...: width / 128 heads of 128 x 128
+# values of state; grouped-query attention with heads of 128 features, a window of 1,024 positions that keeps the first four
+# and a slope per head, beside a Mamba-2 recurrence of the model's width with a state of 128.  The first of every three
+# feed-forwards is dense (two matrices with the weights of the Qwen2 layer's three), the others eight routed experts with a gate
+# branch of which two are chosen and a shared one, the chosen two and the shared one together with those weights.  Two of the
+# layers are passed twice, so that the number of layer runs is the other model's number of layers.  Random weights.
+def dinatar_config(width, heads, layers, vocab=32768, max_positions=32768):
+    kv = max(1, heads // 4 if heads % 4 == 0 and heads > 12 else heads // 6)
+    h = width // 128
+    att = {"heads": heads, "kv_heads": kv, "dim": 128, "vdim": 128, "scale": 128 ** -0.5, "mask": {"size": 1024, "keep_first": 4}}
+    mam = {"heads": h, "vdim": 128, "state": 128, "groups": 1, "conv": 4, "norm_groups": 1}
+    par = ("parallel", {"left": att, "right": mam})
+    lin = {"heads": h, "dim": 128, "vdim": 128}
+    kinds = [("hgrn2", lin), par, ("gla", dict(lin, tau=16.0, rank=16)), par]
+    im = (8 * width // 3) // 128 * 128
+    moe = {"kind": "moe", "expert": {"ff": (im // 4) // 64 * 64}, "router": {"experts": 8, "top": 2}, "shared": {"ff": (im // 2) // 64 * 64}}
+    k = 2 if layers >= 5 else 1                    # layers passed twice
+    n = layers - k
+    return {"architecture": "Dinatar", "vocab": vocab, "width": width, "max_positions": max_positions, "norm": {"eps": 1e-6},
+            "embedding": {"scale": 12.0}, "logit_scale": 0.5, "loop": {"start": 0, "stop": k, "times": 2},
+            "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1],
+                        "mlp": {"kind": "dense", "ff": 4 * width} if i % 3 == 0 else moe} for i in range(n)]}
+
+
 DESIGN_SIZES = {"1536": (1536, 12, 8), "4096": (4096, 32, 4)}      # width -> (width, heads, layers)
 DESIGNS = {"sukisun": lambda w, h, l: sukisun_config(w, h, l), "nadilorn": lambda w, h, l: nadilorn_config(w, h, l),
            "nadilorn-v64": lambda w, h, l: nadilorn_config(w, h, l, vdim=64), "sofudra": lambda w, h, l: sofudra_config(w, h, l),
-           "tuzupel": lambda w, h, l: tuzupel_config(w, h, l)}
+           "tuzupel": lambda w, h, l: tuzupel_config(w, h, l), "dinatar": lambda w, h, l: dinatar_config(w, h, l)}
 BESIDE = dict(DESIGNS, qwen2=lambda w, h, l: qwen2_like(w, h, l))
 
 
@@ -474,7 +499,8 @@ def design_point(cfg, pk, batch, context, steps, warmup, tokens):
     out["decode_ms"] = round(ms, 4)
     out["decode_launches_per_step"] = launches // max(1, steps)
     # (a layer with a window reads no more of a request's positions than the window holds)
-    windows = [l["mixer"].get("mask", {}).get("size") for l in cfg.get("layers", []) if isinstance(l.get("mixer"), dict)]
+    windows = [l["mixer"].get("left", l["mixer"]).get("mask", {}).get("size") for l in cfg.get("layers", [])
+               if isinstance(l.get("mixer"), dict) and l.get("type") not in ("hgrn2", "gla")]
     seen = min([context - steps / 2.0] + [w for w in windows if w]) if windows and all(windows) else context - steps / 2.0
     step_bytes = eng.model.weight_bytes() + batch * seen * out["cache_bytes_per_token"] + 2 * state_bytes
     out["decode_frac_of_hbm"] = round(step_bytes / (ms * 1e-3) / 1e9 / pk["hbm_gbs"], 4)
