@@ -6,7 +6,8 @@
 // token finds zeros there.  Four kernels: the convolution with SiLU, the update of its state, the scan, and the gate
 // with the grouped RMS norm.  Everything that enters the recurrence is float: step sizes, decays, B, C, x.
 //
-// Requests are given as a list of (request, first row, number of rows), one entry per request of the step.
+// Requests are given as a list of (request, first row, number of rows), one entry per request of the step (the scan's list
+// may leave out requests whose rows run in chunks: mamba2_chunked.cu).
 #include "common.cuh"
 
 namespace bg {
@@ -146,8 +147,8 @@ ssm_scan_kernel(const float* __restrict__ xbc, int channels, const TI* __restric
     float* y_s = sm + 2 * buf_floats;
     pdl_launch();
     pdl_wait();
-    const int h = blockIdx.x, req = blockIdx.y, p0 = blockIdx.z * PT;
-    const int row0 = reqs[req * 3 + 1], n = reqs[req * 3 + 2];
+    const int h = blockIdx.x, r = blockIdx.y, p0 = blockIdx.z * PT;
+    const int req = reqs[r * 3 + 0], row0 = reqs[r * 3 + 1], n = reqs[r * 3 + 2];   // (the list may leave requests out)
     if (n <= 0) return;
     const int tid = threadIdx.x;
     const int pl = tid / NS, ns = tid - pl * NS;

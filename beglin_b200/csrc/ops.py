@@ -144,6 +144,10 @@ _SIGNATURES = {
                      _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p],
     "bg_ssm_scan": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p,
                     _c_ll, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+    "bg_ssm_chunk_plan": [_c_int, _c_int, _c_int, _c_int, ctypes.POINTER(_c_int)],
+    "bg_ssm_chunked": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_ll,
+                       _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int,
+                       _c_int, _c_int, _c_void_p],
     "bg_gated_group_rmsnorm": [_c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_float, _c_void_p, _c_int,
                                _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "bg_gemm_f32_nt_batched": [_c_void_p, _c_int, _c_ll, _c_void_p, _c_int, _c_ll, _c_void_p, _c_int, _c_ll, _c_int, _c_int,
@@ -1250,14 +1254,24 @@ def conv_silu(src: torch.Tensor, col0: int, channels: int, weight: torch.Tensor,
         count_launches(1)
 
 
+def ssm_chunk(H: int, P: int, N: int, G: int) -> int:
+    """The number of tokens in a chunk of the chunked recurrence for these sizes, 0 when it does not take them."""
+    c = _c_int(0)
+    return c.value if lib().bg_ssm_chunk_plan(int(H), int(P), int(N), int(G), ctypes.byref(c)) == 0 else 0
+
+
 def ssm_scan(xbc: torch.Tensor, src: torch.Tensor, dt_col: int, dt_bias: torch.Tensor, A_log: torch.Tensor, D: torch.Tensor,
-             state: torch.Tensor, slots: torch.Tensor, reqs: torch.Tensor, n_req: int, y: torch.Tensor, H: int, P: int,
-             N: int, G: int) -> None:
+             state: torch.Tensor, slots: torch.Tensor, reqs: Optional[torch.Tensor], n_req: int, y: torch.Tensor, H: int, P: int,
+             N: int, G: int, chunks: Optional[torch.Tensor] = None, n_chunks: int = 0, longs: Optional[torch.Tensor] = None,
+             n_long: int = 0) -> None:
     """The recurrence over each request's rows, from and into the slots' state S [H, P, N] (float32, at the start of
     a slot): dt = softplus(src[t, dt_col + h] + dt_bias[h]); S = exp(-exp(A_log[h]) dt) S + dt B_t x_t^T;
-    y_t = S^T C_t + D[h] x_t.  xbc float32 [T, H P + 2 G N] = [x | B | C]; y float32 [T, H P]."""
-    _cuda(xbc, src, dt_bias, A_log, D, state, slots, reqs, y)
-    _i32(slots, "slots"); _i32(reqs, "reqs")
+    y_t = S^T C_t + D[h] x_t.  xbc float32 [T, H P + 2 G N] = [x | B | C]; y float32 [T, H P].  Requests of many rows may be
+    given apart, in chunks of `ssm_chunk(...)` rows (`chunks`, `longs` as in `decay_attention`)."""
+    _cuda(xbc, src, dt_bias, A_log, D, state, slots, reqs, y, chunks, longs)
+    _i32(slots, "slots")
+    if n_req:
+        _i32(reqs, "reqs")
     T = xbc.shape[0]
     if xbc.dtype != torch.float32 or not xbc.is_contiguous() or xbc.shape[1] != H * P + 2 * G * N:
         raise KernelError(f"ssm_scan: xbc is {tuple(xbc.shape)}")
@@ -1270,9 +1284,21 @@ def ssm_scan(xbc: torch.Tensor, src: torch.Tensor, dt_col: int, dt_bias: torch.T
     if y.dtype != torch.float32 or tuple(y.shape) != (T, H * P) or not y.is_contiguous():
         raise KernelError("ssm_scan: y is float32 [T, H P]")
     with phase("scan"):
-        _check(lib().bg_ssm_scan(_p(xbc), xbc.shape[1], _p(src), _dt(src), src.stride(0), dt_col, _p(dt_bias), _p(A_log), _p(D),
-                                 _dt(D), _p(state), state.stride(0), _p(slots), _p(reqs), n_req, _p(y), H, P, N, G, _stream()),
-               "ssm_scan")
+        if n_req:
+            _check(lib().bg_ssm_scan(_p(xbc), xbc.shape[1], _p(src), _dt(src), src.stride(0), dt_col, _p(dt_bias), _p(A_log), _p(D),
+                                     _dt(D), _p(state), state.stride(0), _p(slots), _p(reqs), n_req, _p(y), H, P, N, G, _stream()),
+                   "ssm_scan")
+        if n_chunks:
+            _i32(chunks, "chunks"); _i32(longs, "longs")
+            if chunks.shape[0] < n_chunks or longs.shape[0] < n_long or n_long < 1:
+                raise KernelError("ssm_scan: the lists of chunks and of long requests are shorter than their counts")
+            f32, size = dict(dtype=torch.float32, device=y.device), ssm_chunk(H, P, N, G)
+            scores, work = torch.empty((n_chunks, G, size * size), **f32), torch.empty((n_chunks, H, N * P), **f32)
+            decay = torch.empty((n_chunks, H), **f32)
+            _check(lib().bg_ssm_chunked(_p(xbc), xbc.shape[1], _p(src), _dt(src), src.stride(0), dt_col, _p(dt_bias), _p(A_log), _p(D),
+                                        _dt(D), _p(state), state.stride(0), _p(slots), _p(chunks), n_chunks, _p(longs), n_long,
+                                        _p(scores), _p(work), _p(decay), _p(y), H, P, N, G, _stream()), "ssm_chunked")
+            count_launches(3)
 
 
 def gated_group_rmsnorm(y: torch.Tensor, src: torch.Tensor, z_col: int, weight: torch.Tensor, eps: float, groups: int,

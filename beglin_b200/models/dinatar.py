@@ -287,7 +287,7 @@ def _parallel_spec(d: int, m: ParallelMixerConfig, eps: float, to: str):
                          position=PositionSpec(kind="none"), window=a.window, scale=a.scale, v_head_dim=a.vdim,
                          keep_first=a.keep_first if a.window is not None else 0, slopes=distance_slopes(a.heads))
     right = Mamba2Spec(hidden=d, n_heads=b.heads, vdim=b.vdim, state=b.state, groups=b.groups, conv=b.conv, norm_groups=b.norm_groups,
-                       eps=eps)
+                       eps=eps, chunked=True)
     names = {f"mixer.left.{x}_proj.{kind}": f"{to}left.{x}{end}" for x in "qkv" for kind, end in (("weight", ""), ("bias", ".b"))}
     names.update({"mixer.left.o_proj.weight": to + "left.o", "mixer.left.out_norm.weight": to + "left.out",
                   "mixer.right.in_proj.weight": to + "right.in", "mixer.right.conv.weight": to + "right.conv",

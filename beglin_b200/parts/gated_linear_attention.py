@@ -66,6 +66,9 @@ class GatedLinearAttention:
         self.r_col = sum(w.shape[0] for w in rows)
         if spec.write == "key":
             rows.append(tensors["decay_in.weight"])
+        pad = -sum(w.shape[0] for w in rows) % 8       # rows of zeros keep the product's rows 16 bytes apart
+        if pad:
+            rows.append(torch.zeros((pad, spec.hidden), dtype=rows[0].dtype, device=rows[0].device))
         self.in_proj = Linear(torch.cat(rows, dim=0), None, ctx, label="proj_qkv")
         self.o_proj = Linear(tensors["o_proj.weight"], None, ctx, label="proj_o")
         f32 = lambda t: t.to(device=ctx.device, dtype=torch.float32).contiguous()

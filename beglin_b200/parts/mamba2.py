@@ -10,6 +10,9 @@ The state S and the last conv - 1 inputs of the convolution are per-request stat
 the cache manager's slab, float32, zero when the request starts): a step continues each request from its
 slot, however the request's tokens are cut into steps and whatever else the step holds.  Everything that
 enters the recurrence is float in both number formats.
+
+With the spec's `chunked`, a request that brings `LONG_FROM` rows or more runs in chunks (the chunks' own sums and outputs side
+by side, a short pass over their states between), where the sizes allow it; fewer rows, and single tokens, are walked one by one.
 """
 from __future__ import annotations
 
@@ -62,14 +65,20 @@ class Mamba2:
             raise ValueError("the convolution has at least one tap")
         self.spec, self.ctx = spec, ctx
         self.inner, self.channels = inner, channels
-        self.in_proj = Linear(tensors["in_proj.weight"], None, ctx, label="proj_in")
+        w = tensors["in_proj.weight"]
+        pad = (-w.shape[0]) % 8            # rows of zeros behind the step sizes keep the product's rows 16 bytes apart
+        if pad:
+            w = torch.cat([w, torch.zeros((pad, w.shape[1]), dtype=w.dtype, device=w.device)], dim=0)
+        self.in_proj = Linear(w, None, ctx, label="proj_in")
         self.o_proj = Linear(tensors["o_proj.weight"], None, ctx, label="proj_o")
         same = lambda t: t.to(device=ctx.device, dtype=ctx.compute_dtype).contiguous()
         self.conv_w, self.conv_b = same(tensors["conv.weight"]), same(tensors["conv.bias"])
         self.dt_bias, self.A_log, self.D = same(tensors["dt_bias"]), same(tensors["A_log"]), same(tensors["D"])
         self.norm_w = ctx.vector(tensors["norm.weight"])
         self.conv_off = spec.n_heads * spec.state * spec.vdim
+        self.chunk = ops.ssm_chunk(spec.n_heads, spec.vdim, spec.state, spec.groups) if spec.chunked and ctx.device.type == "cuda" else 0
 
+    LONG_FROM = 64             # rows of a request in a step from which its tokens run in chunks
     takes_stream = True        # forward takes a NormedInput and may add its result to the stream itself
 
     def forward(self, h, batch, cache: FixedStateView, stream: Optional[ResidualStream] = None) -> Optional[torch.Tensor]:
@@ -85,8 +94,11 @@ class Mamba2:
         ops.conv_silu(proj, self.inner, self.channels, self.conv_w, self.conv_b, cache.state, self.conv_off, cache.slots,
                       batch.row_req, reqs, n_req, xbc)
         y = torch.empty((T, self.inner), dtype=torch.float32, device=h.device)
+        chunks, n_chunks, longs, n_long = None, 0, None, 0
+        if self.chunk and not batch.decode_only and hasattr(batch, "long_blocks"):
+            reqs, n_req, chunks, n_chunks, longs, n_long = batch.long_blocks(self.chunk, self.LONG_FROM)
         ops.ssm_scan(xbc, proj, self.inner + self.channels, self.dt_bias, self.A_log, self.D, cache.state, cache.slots,
-                     reqs, n_req, y, s.n_heads, s.vdim, s.state, s.groups)
+                     reqs, n_req, y, s.n_heads, s.vdim, s.state, s.groups, chunks, n_chunks, longs, n_long)
         out = torch.empty((T, self.inner), dtype=ctx.compute_dtype, device=h.device)
         ops.gated_group_rmsnorm(y, proj, 0, self.norm_w, s.eps, s.norm_groups, out)
         if stream is None:

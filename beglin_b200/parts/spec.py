@@ -180,7 +180,8 @@ class LatentAttentionSpec:
 class Mamba2Spec:
     """The Mamba-2 recurrence: `n_heads` heads of `vdim` features with a state of `state` x vdim each, B and C
     shared inside each of `groups` groups of heads, a causal convolution of `conv` taps over x, B and C, and
-    an RMS norm of the gated result in `norm_groups` equal parts."""
+    an RMS norm of the gated result in `norm_groups` equal parts.  `chunked`: portions of many rows may run in chunks, several
+    times faster; ways of cutting a prompt then agree up to rounding, where the walk row by row agrees bit for bit in float32."""
     hidden: int
     n_heads: int
     vdim: int
@@ -189,6 +190,7 @@ class Mamba2Spec:
     conv: int
     norm_groups: int
     eps: float
+    chunked: bool = False
     kind: str = "mamba2"
 
 

@@ -103,8 +103,9 @@ def test_linear_attention_token_by_token_in_chunks_over_steps_and_slots(H, n, nv
         out = torch.full((sum(lens), H * nv), NAN, device=DEV, dtype=dtype)
         L.run(rows, state, slots, out, reqs=up(short) if len(short) else None, chunks=up(chunks) if len(chunks) else None,
               longs=up(longs) if len(longs) else None)
-        assert rel_err(out, want) < (2e-5 if dtype == torch.float32 else 6e-3), lens
         for i in range(4):
+            sl = slice(starts[i], starts[i] + lens[i])
+            assert rel_err(out[sl], want[sl]) < (2e-5 if dtype == torch.float32 else 6e-3), (lens, i)
             assert rel_err(state[slot_of[i], :sz].view(H, n, nv), S[i]) < 5e-6, (lens, i)
     assert torch.isnan(state[[1, 3]]).all() and torch.isnan(state[:, sz:]).all()
 
@@ -136,6 +137,51 @@ def test_decays_of_nought_and_of_nearly_one():
         assert torch.isfinite(out).all() and rel_err(out, want) < 2e-4, way          # (900 products of decays, each rounded)
         assert rel_err(state.view(1, n, nv), S) < 2e-4
     assert float(S[0, 1].abs().max()) > 20.0
+
+
+# ---------------------------------------------------------------------------------------------- Mamba-2
+@pytest.mark.parametrize("H,P,N,G", [(1, 4, 4, 1), (6, 36, 20, 2), (2, 128, 128, 1), (4, 64, 64, 4), (3, 100, 200, 1), (2, 7, 9, 1)])
+@pytest.mark.parametrize("wdtype", [torch.float32, torch.bfloat16])
+def test_mamba2_in_chunks_and_row_by_row_over_steps_and_slots(H, P, N, G, wdtype):
+    """Three steps over four requests in shuffled slots with NaN in everything unwritten, portions of 64 rows and more in chunks
+    where the sizes allow it (multiples of 4): step sizes from nearly nought to ones that forget everything, against the
+    recurrence token by token."""
+    from beglin_b200.engine.batch import cut_long_requests
+    o = ops()
+    g = torch.Generator().manual_seed(H * P + N)
+    r = lambda *s: torch.randn(*s, generator=g)
+    A_log, dt_bias, D = (r(H) * 1.5).to(wdtype), r(H).to(wdtype), r(H).to(wdtype)
+    sz, width = H * N * P, H * P + 2 * G * N
+    state = torch.full((6, sz + 4), NAN, device=DEV)
+    slot_of = [4, 0, 5, 2]
+    state[slot_of, :sz] = 0.0
+    S = [torch.zeros(H, N, P, dtype=torch.float64) for _ in range(4)]
+    chunk = o.ssm_chunk(H, P, N, G)
+    assert bool(chunk) == (P % 4 == 0 and N % 4 == 0)
+    for lens in ([200, 1, 64, 3], [1, 70, 1, 129], [65, 17, 1, 63]):
+        T = sum(lens)
+        starts = [sum(lens[:i]) for i in range(4)]
+        xbc, raw = r(T, width), 3.0 * r(T, H + 2) - 2.0
+        raw[::13] = 60.0                                   # a step that forgets the state, between small ones
+        x, B, C = xbc[:, :H * P].double().view(T, H, P), xbc[:, H * P:H * P + G * N].double().view(T, G, N), xbc[:, H * P + G * N:].double().view(T, G, N)
+        dt = torch.nn.functional.softplus(raw[:, 2:].double() + dt_bias.double())
+        want = torch.zeros(T, H, P, dtype=torch.float64)
+        for i in range(4):
+            for t in range(starts[i], starts[i] + lens[i]):
+                for h in range(H):
+                    gg = h // (H // G)
+                    S[i][h] = torch.exp(-torch.exp(A_log[h].double()) * dt[t, h]) * S[i][h] + dt[t, h] * torch.outer(B[t, gg], x[t, h])
+                    want[t, h] = S[i][h].T @ C[t, gg] + D[h].double() * x[t, h]
+        short, chunks, longs = cut_long_requests(starts, lens, chunk or 64, 64 if chunk else 1 << 30)
+        up = lambda a: torch.from_numpy(a).to(DEV)
+        y = torch.full((T, H * P), NAN, device=DEV)
+        o.ssm_scan(dev(xbc), dev(raw), 2, dev(dt_bias), dev(A_log), dev(D), state, torch.tensor(slot_of, dtype=torch.int32, device=DEV),
+                   up(short), len(short), y, H, P, N, G, up(chunks), len(chunks), up(longs), len(longs))
+        for i in range(4):
+            sl = slice(starts[i], starts[i] + lens[i])
+            assert rel_err(y.view(T, H, P)[sl], want[sl]) < 5e-6, (lens, i)
+            assert rel_err(state[slot_of[i], :sz].view(H, P, N).transpose(1, 2), S[i]) < 5e-6, (lens, i)
+    assert torch.isnan(state[[1, 3]]).all() and torch.isnan(state[:, sz:]).all()
 
 
 # ---------------------------------------------------------------------------------------------- attention
