@@ -197,7 +197,13 @@ __global__ void __launch_bounds__(256) ssm_chunk_scan_kernel(SsmChunkParams p) {
     *st = S;
 }
 
-// acc[u][v] += sum over k of a[t0 + u][k] b[k][c0 + v], k in steps of 4 up to `k_end`
+// The token that a thread's row u (of eight) stands for: a warp holds sixteen tokens, a half of it four neighbours and the four
+// eight further on, so that the two halves' reads of a tile of rows fall on different banks.
+__device__ __forceinline__ int sc_token(int u) {
+    return ((int)threadIdx.x >> 5) * 16 + (((int)threadIdx.x >> 4) & 1) * 4 + (u & 3) + (u >> 2) * 8;
+}
+
+// acc[u][v] += sum over k of a[token of row u][k] b[k][v], k in steps of 4 up to `k_end`
 __device__ __forceinline__ void sc_product(float (&acc)[8][4], const float* a, int lda, const float* b, int k_end) {
 #pragma unroll 1
     for (int k = 0; k < k_end; k += 4) {
@@ -206,7 +212,7 @@ __device__ __forceinline__ void sc_product(float (&acc)[8][4], const float* a, i
         for (int i = 0; i < 4; ++i) bb[i] = *reinterpret_cast<const float4*>(b + (size_t)(k + i) * MPT);
 #pragma unroll
         for (int u = 0; u < 8; ++u) {
-            const float4 aa = *reinterpret_cast<const float4*>(a + (size_t)u * lda + k);
+            const float4 aa = *reinterpret_cast<const float4*>(a + sc_token(u) * lda + k);
             acc[u][0] = fmaf(aa.x, bb[0].x, acc[u][0]); acc[u][1] = fmaf(aa.x, bb[0].y, acc[u][1]);
             acc[u][2] = fmaf(aa.x, bb[0].z, acc[u][2]); acc[u][3] = fmaf(aa.x, bb[0].w, acc[u][3]);
             acc[u][0] = fmaf(aa.y, bb[1].x, acc[u][0]); acc[u][1] = fmaf(aa.y, bb[1].y, acc[u][1]);
@@ -267,24 +273,25 @@ __global__ void __launch_bounds__(128) ssm_chunk_out_kernel(SsmChunkParams p) {
         // (the first half's queries never read a key of the second)
     }
     __syncthreads();
-    const int t0 = (tid >> 4) * 8, c0 = (tid & 15) * 4;
+    const int t0 = (tid >> 5) * 16, c0 = (tid & 15) * 4;        // the warp's first token
     if (t0 >= rows || c0 >= pw) return;
     float acc[8][4] = {};
-    sc_product(acc, Cs + (size_t)t0 * ldc, ldc, Ss + c0, N);
+    sc_product(acc, Cs, ldc, Ss + c0, N);
     const float first = t0 >= MC / 2 ? pre[MC / 2 - 1] : 1.0f;
 #pragma unroll
     for (int u = 0; u < 8; ++u) {
-        const float f = first * pre[t0 + u];
+        const float f = first * pre[sc_token(u)];
 #pragma unroll
         for (int v = 0; v < 4; ++v) acc[u][v] *= f;
     }
-    sc_product(acc, Ws + (size_t)t0 * MCP, MCP, Xs + c0, t0 + 8);
+    sc_product(acc, Ws, MCP, Xs + c0, t0 + 16);
     const float Dh = to_float(((const TW*)p.D)[h]);
 #pragma unroll
     for (int u = 0; u < 8; ++u) {
-        if (t0 + u >= rows) break;
-        const float4 x = *reinterpret_cast<const float4*>(Xs + (t0 + u) * MPT + c0);
-        *reinterpret_cast<float4*>(p.y + (size_t)(row0 + t0 + u) * p.H * P + (size_t)h * P + p0 + c0) =
+        const int t = sc_token(u);
+        if (t >= rows) continue;
+        const float4 x = *reinterpret_cast<const float4*>(Xs + t * MPT + c0);
+        *reinterpret_cast<float4*>(p.y + (size_t)(row0 + t) * p.H * P + (size_t)h * P + p0 + c0) =
             make_float4(fmaf(Dh, x.x, acc[u][0]), fmaf(Dh, x.y, acc[u][1]), fmaf(Dh, x.z, acc[u][2]), fmaf(Dh, x.w, acc[u][3]));
     }
 }

@@ -87,7 +87,7 @@ _SIGNATURES = {
                           _c_void_p, _c_void_p, _c_void_p],
     "bg_gla_walk": [_c_void_p, _c_void_p, _c_int, _c_void_p],
     "bg_gla_chunk_plan": [_c_int, _c_int, ctypes.POINTER(_c_int)],
-    "bg_gla_chunked": [_c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p],
+    "bg_gla_chunked": [_c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_void_p],
     "bg_attention_mma_plan": [_c_int, _c_int, _c_int, ctypes.POINTER(_c_int)],
     "bg_attention_mma_partial": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p,
                                  _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
@@ -1575,11 +1575,13 @@ def gated_linear_attention(src: torch.Tensor, q_col: int, k_col: int, v_col: int
             if chunks.shape[0] < n_chunks or longs.shape[0] < n_long or n_long < 1:
                 raise KernelError("gated_linear_attention: the lists of chunks and of long requests are shorter than their counts")
             f32 = dict(dtype=torch.float32, device=out.device)
-            work, decay = torch.empty((n_chunks, H, n * nv), **f32), torch.empty((n_chunks, H, n), **f32)
-            alpha = torch.empty((T, H * n), **f32) if lower is None else None
-            _check(lib().bg_gla_chunked(ctypes.byref(a), T, _p(chunks), n_chunks, _p(longs), n_long, _p(work), _p(decay), _p(alpha),
-                                        _stream()), "gla_chunked")
-            count_launches(2 if lower is not None else 3)
+            np_, nvp, size = -(-n // 4) * 4, -(-nv // 4) * 4, gla_chunk(n, nv)
+            qkd = torch.empty((2, T, H * np_), **f32)
+            scores, work = torch.empty((n_chunks, H, size * size), **f32), torch.empty((n_chunks, H, np_ * nvp), **f32)
+            decay = torch.empty((n_chunks, H, n), **f32)
+            _check(lib().bg_gla_chunked(ctypes.byref(a), _p(chunks), n_chunks, _p(longs), n_long, _p(qkd[0]), _p(qkd[1]), _p(scores),
+                                        _p(work), _p(decay), _stream()), "gla_chunked")
+            count_launches(3)
 
 
 # ---------------------------------------------------------------------------------------------------- routed experts
