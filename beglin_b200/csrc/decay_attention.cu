@@ -503,6 +503,7 @@ __global__ void __launch_bounds__(256) add_terms_norm_kernel(TermsParams p) {
 // The sum of the partial sums of term i, four columns from element `at` on.
 __device__ __forceinline__ float4 term_value4(const TermsParams& p, int i, size_t at) {
     float4 v = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+#pragma unroll 4
     for (int q = 0; q < p.parts[i]; ++q) {
         float4 a;
         if (p.dtype[i] == BG_DTYPE_F32) {

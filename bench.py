@@ -450,7 +450,7 @@ def dinatar_config(width, heads, layers, vocab=32768, max_positions=32768):
     k = 2 if layers >= 5 else 1                    # layers passed twice
     n = layers - k
     return {"architecture": "Dinatar", "vocab": vocab, "width": width, "max_positions": max_positions, "norm": {"eps": 1e-6},
-            "embedding": {"scale": 12.0}, "logit_scale": 0.5, "loop": {"start": 0, "stop": k, "times": 2},
+            "embedding": {"scale": float(width) ** 0.5}, "logit_scale": 0.5, "loop": {"start": 0, "stop": k, "times": 2},
             "layers": [{"type": kinds[i % 4][0], "mixer": kinds[i % 4][1],
                         "mlp": {"kind": "dense", "ff": 4 * width} if i % 3 == 0 else moe} for i in range(n)]}
 
