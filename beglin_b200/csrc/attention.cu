@@ -234,7 +234,8 @@ __global__ void attention_merge_kernel(const float* __restrict__ part_o, const f
     const int lo = first_visible(pos, window);
     const int s_win = lo / split, s_hi = pos / split;
     const int s_lo = keep > 0 ? 0 : s_win;
-    auto seen = [&](int s) { return s <= s_hi && (s >= s_win || s * split < keep); };     // splits that the row has results of
+    const int s_kept = keep > 0 ? (keep - 1) / split : -1;
+    auto seen = [&](int s) { return s <= s_hi && (s >= s_win || s <= s_kept); };          // splits that the row has results of
     const size_t prow = (size_t)w * max_splits;
     // the maxima and sums of the first 32 * MERGE_GROUPS splits of the row: lane j holds split s_lo + 32 g + j
     float ms_r[MERGE_GROUPS], ls_r[MERGE_GROUPS];
@@ -382,6 +383,7 @@ __global__ void attention_merge_few_kernel(const float* __restrict__ part_o, con
     const int split = keys_per_split(split_arg, pos + 1, max_splits);
     const int lo = first_visible(pos, window);
     const int s_lo = lo / split, s_hi = pos / split;
+    const int s_kept = keep > 0 ? (keep - 1) / split : -1;       // (the last split with positions kept for good)
     pdl_wait();
     if (idle) return;                  // (not before the wait: with warps of a CTA gone before it, rows came out wrong)
     float ms[NS], ls[NS], v[NS][4];
@@ -400,7 +402,7 @@ __global__ void attention_merge_few_kernel(const float* __restrict__ part_o, con
     float m = sink ? sv : -INFINITY;
 #pragma unroll
     for (int s = 0; s < NS; ++s) {
-        if ((s < s_lo && s * split >= keep) || s > s_hi) ms[s] = -INFINITY;          // not written for this row: whatever was read is dropped
+        if ((s < s_lo && s > s_kept) || s > s_hi) ms[s] = -INFINITY;          // not written for this row: whatever was read is dropped
         m = fmaxf(m, ms[s]);
     }
     float acc[4] = {0.0f, 0.0f, 0.0f, 0.0f}, l = sink ? expf(sv - m) : 0.0f;
@@ -447,7 +449,7 @@ attention_merge_block_kernel(const float* __restrict__ part_o, const float* __re
     const int split = keys_per_split(split_arg, pos + 1, max_splits);
     const int lo = first_visible(pos, window);
     const int s_win = lo / split, s_hi = pos / split;
-    const int s_lo = keep > 0 ? 0 : s_win;
+    const int s_lo = keep > 0 ? 0 : s_win, s_kept = keep > 0 ? (keep - 1) / split : -1;
     pdl_wait();
     const size_t prow = (size_t)w * max_splits;
     const int d = lane * 4;
@@ -460,7 +462,7 @@ attention_merge_block_kernel(const float* __restrict__ part_o, const float* __re
 #pragma unroll
         for (int j = 0; j < 8; ++j) {
             const int sidx = g * 8 + j;
-            const bool have = sidx <= s_hi && (sidx >= s_win || sidx * split < keep);
+            const bool have = sidx <= s_hi && (sidx >= s_win || sidx <= s_kept);
             const float2 ml = have ? *reinterpret_cast<const float2*>(part_ml + (prow + sidx) * 2) : make_float2(-INFINITY, 0.0f);
             ms[j] = ml.x; ls[j] = ml.y;
             v[j] = (have && live) ? *reinterpret_cast<const float4*>(part_o + (prow + sidx) * hd + d)

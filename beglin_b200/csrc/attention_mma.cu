@@ -64,9 +64,20 @@ struct AttnMmaParams {
     int out_stride;         // the finished rows here (no partial results, no merge)
     int use_tma;            // pages are copied as TMA boxes (the page size divides 64)
     int whole_pages;        // a page is a stage (64 positions): keys and values of a stage come in ONE box
-    int keep;               // EXT: positions 0 .. keep - 1 stay visible behind a window
-    const float* slopes;    // EXT: [nh] or null
 };
+
+// What the EXT instances take besides.  (The plain ones are kept, expression by expression, as they were without EXT: with the
+// conditions of both written as one the compiler's other arrangement of them cost the decoding kernel 7 % of its time.)
+struct AttnMmaExtParams : AttnMmaParams {
+    int keep;               // positions 0 .. keep - 1 stay visible behind a window
+    const float* slopes;    // [nh] or null
+};
+template <bool EXT> struct AmParams { using type = AttnMmaParams; };
+template <> struct AmParams<true> { using type = AttnMmaExtParams; };
+__device__ __forceinline__ int am_keep(const AttnMmaParams&) { return 0; }
+__device__ __forceinline__ int am_keep(const AttnMmaExtParams& p) { return p.keep; }
+__device__ __forceinline__ const float* am_slopes(const AttnMmaParams&) { return nullptr; }
+__device__ __forceinline__ const float* am_slopes(const AttnMmaExtParams& p) { return p.slopes; }
 
 // A product q . k as the exponent of two that the softmax takes: scaled, squashed when the layer asks for it.
 __device__ __forceinline__ float am_score(float c, const AttnMmaParams& p) {
@@ -121,7 +132,8 @@ __device__ __forceinline__ int swz_kv(int row, int c) {
 
 template <int HD, bool BY_KEYS, int AM_STAGES, bool SWAP, bool EXT>
 __global__ void __launch_bounds__(AM_ALL)
-attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_constant__ CUtensorMap map_page, AttnMmaParams p) {
+attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_constant__ CUtensorMap map_page,
+                     typename AmParams<EXT>::type p) {
     constexpr int CH = HD / 8;                 // 16-byte columns per row
     constexpr int KSTEPS = HD / 16;            // k-steps of q.k
     constexpr int NT_O = HD / 8;               // 8-wide column tiles of the output
@@ -188,9 +200,9 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
 
     const int lo_first = first_visible(pos_first, p.window);
     const int k_first = direct ? 0 : sp * split;                  // this CTA's range of positions: [k_first, k_end)
-    const int k_begin = max(k_first, lo_first);                   // of which the window's keys are [k_begin, k_end)
+    const int k_begin = direct ? lo_first : max(k_first, lo_first);   // of which the window's keys are [k_begin, k_end)
     const int k_end = direct ? pos_last + 1 : min((sp + 1) * split, pos_last + 1);
-    const int keep = EXT ? p.keep : 0;
+    const int keep = am_keep(p);
     const int kept_end = min(keep, k_end);                        // and the kept ones [k_first, kept_end), possibly none
     const bool has_kept = EXT && k_first < kept_end;
     if (k_begin >= k_end && !has_kept) return;
@@ -202,7 +214,8 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
     const int n_kept = has_kept ? (kept_end - first_stage_key + AM_STAGE_KEYS - 1) / AM_STAGE_KEYS : 0;
     const int kept_stop = first_stage_key + n_kept * AM_STAGE_KEYS;
     const int skip = has_kept ? max((k_begin / AM_STAGE_KEYS) * AM_STAGE_KEYS - kept_stop, 0) : 0;
-    const int n_stage = n_kept + max((k_end - kept_stop - skip + AM_STAGE_KEYS - 1) / AM_STAGE_KEYS, 0);
+    const int n_stage = EXT ? n_kept + max((k_end - kept_stop - skip + AM_STAGE_KEYS - 1) / AM_STAGE_KEYS, 0)
+                            : (k_end - first_stage_key + AM_STAGE_KEYS - 1) / AM_STAGE_KEYS;
     auto stage_key = [&](int s) { return first_stage_key + s * AM_STAGE_KEYS + (EXT && s >= n_kept ? skip : 0); };
     const int last_page = (k_end - 1) / p.page_size;
     int table_group = (first_stage_key / p.page_size) / AM_TABLE;
@@ -226,8 +239,9 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
         const int* table = p.block_table + (size_t)req * p.max_pages;
         auto page_of = [&](int s, int o) {               // the page that box o of stage s comes from, or -1
             const int key_lo = stage_key(s) + (o / PER_PAGE) * ps;
-            if (s >= n_stage || o >= n_box || key_lo >= k_end || (key_lo >> shift) >= p.max_pages) return -1;
-            if (key_lo + ps <= k_begin && !(has_kept && key_lo < kept_end && key_lo + ps > k_first)) return -1;
+            if (!EXT && (s >= n_stage || o >= n_box || key_lo >= k_end || key_lo + ps <= k_begin || (key_lo >> shift) >= p.max_pages)) return -1;
+            if (EXT && (s >= n_stage || o >= n_box || key_lo >= k_end || (key_lo >> shift) >= p.max_pages ||
+                        (key_lo + ps <= k_begin && !(has_kept && key_lo < kept_end && key_lo + ps > k_first)))) return -1;
             return table[key_lo >> shift];
         };
         // stages of old keys only may be asked for before the kernel ahead has finished: all but the one that
@@ -300,7 +314,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
             for (int j = tid / CH; j < AM_STAGE_KEYS; j += ROWS_PER_PASS) {
                 const int key = stage_key0 + j;
                 const __nv_bfloat16* src = nullptr;
-                if (in_range(key)) {
+                if (EXT ? in_range(key) : (key >= k_begin && key < k_end)) {
                     const int pi = p.page_shift >= 0 ? key >> p.page_shift : key / p.page_size;
                     const int slot = p.page_shift >= 0 ? key & (p.page_size - 1) : key - pi * p.page_size;
                     const int page = table_s[pi - table_group * AM_TABLE];
@@ -348,11 +362,11 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
     }
     // what the scores of this thread's two rows (or two heads) fall by per position, in powers of two
     float slope_l2[2] = {0.0f, 0.0f};
-    if (EXT && p.slopes) {
+    if (EXT && am_slopes(p)) {
 #pragma unroll
         for (int h = 0; h < 2; ++h) {
             const int r = SWAP ? 2 * (lane & 3) + h : row_base + (lane >> 2) + h * 8;
-            if (r < n_rows) slope_l2[h] = p.slopes[kvh * group + r % group] * AM_LOG2E;
+            if (r < n_rows) slope_l2[h] = am_slopes(p)[kvh * group + r % group] * AM_LOG2E;
         }
     }
     // the span of keys that the rows of this warp can see at all, and the span that ALL its rows see
@@ -409,14 +423,13 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
             // A wait that runs out records it and goes on (with whatever the buffer holds; the host raises on
             // the status): every thread then still reaches the barriers below.
             if (!mbar_wait<4000>(&full_bar[buf], (s / AM_STAGES) & 1, &gave_up) && p.status) atomicOr(p.status, BG_STATUS_TIMEOUT);
-            const bool whole_stage = stage_key0 + AM_STAGE_KEYS <= k_end &&
-                (stage_key0 >= k_begin || (has_kept && stage_key0 >= k_first && stage_key0 + AM_STAGE_KEYS <= kept_end));
-            if (!whole_stage) {                                                    // uniform over the readers
+            const bool kept_stage = EXT && has_kept && stage_key0 >= k_first && stage_key0 + AM_STAGE_KEYS <= kept_end;
+            if ((stage_key0 < k_begin && !kept_stage) || stage_key0 + AM_STAGE_KEYS > k_end) {     // uniform over the readers
                 // whole pages were copied: rows outside the range of keys become zeros (a value row that no
                 // query sees must not hold garbage, since 0 * NaN is NaN)
                 for (int idx = t0; idx < AM_STAGE_KEYS * CH; idx += nt) {
                     const int j = idx / CH, c = idx - j * CH;
-                    if (!in_range(stage_key0 + j)) {
+                    if (EXT ? !in_range(stage_key0 + j) : (stage_key0 + j < k_begin || stage_key0 + j >= k_end)) {
                         *reinterpret_cast<uint4*>(kt + swz_kv(j, c)) = make_uint4(0, 0, 0, 0);
                         *reinterpret_cast<uint4*>(vt + swz_kv(j, c)) = make_uint4(0, 0, 0, 0);
                     }
@@ -429,7 +442,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
             for (int idx = lane; idx < AM_STAGE_KEYS * CH; idx += 32) {
                 const int j = idx / CH, c = idx - j * CH, key = stage_key0 + j;
                 const __nv_bfloat16* src = nullptr;
-                if (in_range(key)) {
+                if (EXT ? in_range(key) : (key >= k_begin && key < k_end)) {
                     const int pi = key / p.page_size, slot = key - pi * p.page_size;
                     const int page = pi < p.max_pages ? p.block_table[(size_t)req * p.max_pages + pi] : -1;
                     if (page < 0 || page >= p.num_pages) {
@@ -481,7 +494,8 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
 #pragma unroll
                 for (int e = 0; e < 4; ++e) {
                     const int key = w_key0 + kb * 16 + (lane >> 2) + 8 * (e >> 1);
-                    const bool ok = all_seen || (key <= pos && key_seen(key, lo, keep) && in_range(key));
+                    const bool ok = all_seen || (EXT ? (key <= pos && key_seen(key, lo, keep) && in_range(key))
+                                                     : (key <= pos && key >= lo && key >= k_begin && key < k_end));
                     float v = (ok && r0 + (e & 1) < n_rows) ? am_score(c[kb][e], p) : -INFINITY;
                     if (EXT) v = fmaf(slope_l2[e & 1], (float)(key - pos), v);
                     c[kb][e] = v;
@@ -566,7 +580,8 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
                     for (int e = 0; e < 4; ++e) {
                         const int key = w_key0 + j * 8 + (lane & 3) * 2 + (e & 1);
                         const int h = e >> 1;
-                        const bool ok = key <= pos_r[h] && key_seen(key, lo_r[h], keep) && in_range(key);
+                        const bool ok = EXT ? (key <= pos_r[h] && key_seen(key, lo_r[h], keep) && in_range(key))
+                                            : (key <= pos_r[h] && key >= lo_r[h] && key >= k_begin && key < k_end);
                         float v = ok ? am_score(sc[j][e], p) : -INFINITY;
                         if (EXT) v = fmaf(slope_l2[h], (float)(key - pos_r[h]), v);
                         sc[j][e] = v;
@@ -649,7 +664,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
         for (int h = 0; h < 2; ++h) {
             int r = row_base + (lane >> 2) + h * 8;
             if (r >= n_rows) continue;
-            if (pos_r[h] < sp * split || (lo_r[h] >= (sp + 1) * split && sp * split >= keep)) continue;
+            if (pos_r[h] < sp * split || (lo_r[h] >= (sp + 1) * split && !(EXT && sp * split < keep))) continue;
             int qi = r / group, g = r - qi * group;
             size_t prow = ((size_t)(row0 + qi) * p.nh + (size_t)kvh * group + g) * p.max_splits + sp;
             float* po = p.part_o + prow * HD;
@@ -693,7 +708,7 @@ attention_mma_kernel(const __grid_constant__ CUtensorMap map_kv, const __grid_co
         compute_sync();
         const int pos = pos_first;
         const int lo = first_visible(pos, p.window);
-        if (!(pos < sp * split || (lo >= (sp + 1) * split && sp * split >= keep))) {
+        if (!(pos < sp * split || (lo >= (sp + 1) * split && !(EXT && sp * split < keep)))) {
             // every thread takes one feature of all rows and works out the weights of the four warps' parts itself
             // (four exponentials a row: cheaper than a third barrier and a round through shared memory)
             if (tid < HD) {
@@ -729,25 +744,26 @@ static size_t am_smem_bytes() {
 }
 
 template <int HD, bool BY_KEYS, int STAGES, bool SWAP, bool EXT>
-static int am_launch_stages(const CUtensorMap& map, const CUtensorMap& map5, const AttnMmaParams& p, int n_qblk, int n_splits, cudaStream_t stream) {
+static int am_launch_stages(const CUtensorMap& map, const CUtensorMap& map5, const AttnMmaExtParams& p, int n_qblk, int n_splits, cudaStream_t stream) {
     auto kern = attention_mma_kernel<HD, BY_KEYS, STAGES, SWAP, EXT>;
     size_t smem = am_smem_bytes<HD, BY_KEYS, STAGES>();
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
     dim3 grid(n_qblk, p.nkv, n_splits);
-    e = launch(kern, grid, dim3(AM_ALL), smem, stream, map, map5, p);
+    e = launch(kern, grid, dim3(AM_ALL), smem, stream, map, map5,
+               static_cast<const typename AmParams<EXT>::type&>(p));
     if (e != cudaSuccess) return (int)e;
     return BG_OK;
 }
 
 template <int HD, bool BY_KEYS, bool EXT>
-static int am_launch_as(const CUtensorMap& map, const CUtensorMap& map5, const AttnMmaParams& p, int n_qblk, int n_splits, cudaStream_t stream) {
+static int am_launch_as(const CUtensorMap& map, const CUtensorMap& map5, const AttnMmaExtParams& p, int n_qblk, int n_splits, cudaStream_t stream) {
     if (BY_KEYS && p.group <= 8) return am_launch_stages<HD, BY_KEYS, AM_THREADS / 32, BY_KEYS, EXT>(map, map5, p, n_qblk, n_splits, stream);
     if (BY_KEYS) return am_launch_stages<HD, BY_KEYS, AM_THREADS / 32, false, EXT>(map, map5, p, n_qblk, n_splits, stream);   // a buffer per warp
     return am_launch_stages<HD, BY_KEYS, 3, false, EXT>(map, map5, p, n_qblk, n_splits, stream);
 }
 template <int HD, bool BY_KEYS>
-static int am_launch(const CUtensorMap& map, const CUtensorMap& map5, const AttnMmaParams& p, int n_qblk, int n_splits, cudaStream_t stream) {
+static int am_launch(const CUtensorMap& map, const CUtensorMap& map5, const AttnMmaExtParams& p, int n_qblk, int n_splits, cudaStream_t stream) {
     if (p.keep > 0 || p.slopes) return am_launch_as<HD, BY_KEYS, true>(map, map5, p, n_qblk, n_splits, stream);
     return am_launch_as<HD, BY_KEYS, false>(map, map5, p, n_qblk, n_splits, stream);
 }
@@ -781,7 +797,7 @@ extern "C" int bg_attention_mma_partial(const void* q, int q_stride, const void*
     if (nh % nkv != 0 || split % AM_STAGE_KEYS != 0 || (split <= 0 && !by_keys)) return BG_ERR_SHAPE;
     if (n_splits_launch > max_splits || n_splits_launch > 65535 || nkv > 65535) return BG_ERR_SHAPE;
     if ((q_stride % 8) != 0 || ((uintptr_t)q % 16) != 0 || ((uintptr_t)kv_pool % 16) != 0) return BG_ERR_ALIGN;
-    AttnMmaParams p;
+    AttnMmaExtParams p;
     p.q = (const __nv_bfloat16*)q; p.q_stride = q_stride; p.kv_pool = (const __nv_bfloat16*)kv_pool;
     p.num_pages = num_pages; p.page_size = page_size; p.block_table = block_table;
     p.page_shift = -1;

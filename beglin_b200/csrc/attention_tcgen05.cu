@@ -154,8 +154,8 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
     const int k_end = pos_last + 1;
     const int keep = EXT ? p.keep : 0;
     const int n_kept = EXT ? (min(keep, k_end) + AT_BK - 1) / AT_BK : 0;         // tiles with kept positions
-    const int tile0 = max(k_begin / AT_BK, n_kept);                              // the window's first tile behind those
-    const int n_tiles = n_kept + max((k_end + AT_BK - 1) / AT_BK - tile0, 0);
+    const int tile0 = EXT ? max(k_begin / AT_BK, n_kept) : k_begin / AT_BK;      // the window's first tile behind those
+    const int n_tiles = EXT ? n_kept + max((k_end + AT_BK - 1) / AT_BK - tile0, 0) : (k_end + AT_BK - 1) / AT_BK - tile0;
     auto tile_key = [&](int i) { return (EXT && i < n_kept ? i : tile0 + i - n_kept) * AT_BK; };
 
     // ---- Q into shared memory: row r, column block cb, 16-byte piece c at r*128 + ((c ^ (r & 7)) * 16)
@@ -305,7 +305,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
 #pragma unroll
                 for (int q = 0; q < GK; ++q) {
                     const int key = key0 + q;
-                    s[q] = (key <= pos && key_seen(key, lo, keep)) ? s[q] : -INFINITY;
+                    s[q] = (key <= pos && (EXT ? key_seen(key, lo, keep) : key >= lo)) ? s[q] : -INFINITY;
                     tm[q & 3] = fmaxf(tm[q & 3], s[q]);
                 }
             } else {
@@ -412,7 +412,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
                 const int k = h * 32 + lane;
                 const int pi = (key0 >> sh) + k;
                 pg[h] = -1;
-                if (i < n_tiles && k < n_pg && pi < p.max_pages && key0 + k * ps < k_end && (key0 + (k + 1) * ps > k_begin || key0 + k * ps < keep))
+                if (i < n_tiles && k < n_pg && pi < p.max_pages && key0 + k * ps < k_end && (key0 + (k + 1) * ps > k_begin || (EXT && key0 + k * ps < keep)))
                     pg[h] = p.block_table[(size_t)req * p.max_pages + pi];
             }
         };
@@ -442,7 +442,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
             // Key rows that no query may see need no care (their scores are masked, whatever they are); value rows
             // do: 0 * garbage can be NaN.  So a ragged tile of values lands on a barrier of its own, the rows
             // outside the range or in pages that are not held are zeroed, and only then is the tile released.
-            const bool direct = !which || (n_have == n_pg && (key0 >= k_begin || key0 + AT_BK <= keep) && key0 + AT_BK <= k_end);
+            const bool direct = !which || (n_have == n_pg && (key0 >= k_begin || (EXT && key0 + AT_BK <= keep)) && key0 + AT_BK <= k_end);
             unsigned long long* bar = direct ? &full[st] : &kv_landed[st];
             if (lane == 0) {
                 if (n_have > 0) mbar_expect_tx(bar, (unsigned)n_have * ps * HD * 2);
@@ -471,7 +471,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
 #pragma unroll
                     for (int h = 1; h < ROUNDS; ++h) mask = (k >> 5) == h ? have[h] : mask;
                     const int held = (mask >> (k & 31)) & 1;
-                    if (!held || !key_seen(key, k_begin, keep) || key >= k_end)
+                    if (!held || (EXT ? !key_seen(key, k_begin, keep) : key < k_begin) || key >= k_end)
                         *reinterpret_cast<uint4*>(dst + (c >> 3) * KV_BLOCK + jrow * 128 + (((c & 7) ^ (jrow & 7)) << 4)) = make_uint4(0, 0, 0, 0);
                 }
                 fence_proxy_async();
