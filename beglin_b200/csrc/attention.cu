@@ -53,6 +53,7 @@ struct AttnParams {
     float softcap;          // c > 0: scores pass c * tanh(s / c); 0: they stay as they are
     int keep;               // positions 0 .. keep - 1 stay visible behind a window
     const float* slopes;    // [nh] or null
+    int maps;               // a key row holds the keys of this many maps side by side; query head h meets those of map h % maps
     unsigned* status;
 };
 
@@ -61,10 +62,11 @@ __global__ void __launch_bounds__(ATT_THREADS)
 attention_partial_kernel(AttnParams p) {
     extern __shared__ float smem[];
     const int hd = p.hd, vd = p.vd, group = p.group;
+    const int qhd = hd / p.maps;                         // features of a query
     const int kstride = hd + 1;
     const int n_rows_max = p.bq * group;
-    float* q_s = smem;                                   // [n_rows_max][hd]
-    float* acc_s = q_s + (size_t)n_rows_max * hd;        // [n_rows_max][vd]
+    float* q_s = smem;                                   // [n_rows_max][qhd]
+    float* acc_s = q_s + (size_t)n_rows_max * qhd;       // [n_rows_max][vd]
     float* k_s = acc_s + (size_t)n_rows_max * vd;        // [tile][hd+1]
     float* v_s = k_s + (size_t)p.tile * kstride;         // [tile][vd]
     float* m_s = v_s + (size_t)p.tile * vd;              // [n_rows_max]
@@ -88,10 +90,10 @@ attention_partial_kernel(AttnParams p) {
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const int n_rows = nq * group;
     const TQ* q = (const TQ*)p.q;
-    for (int idx = tid; idx < n_rows * hd; idx += ATT_THREADS) {
-        int r = idx / hd, d = idx - r * hd;
+    for (int idx = tid; idx < n_rows * qhd; idx += ATT_THREADS) {
+        int r = idx / qhd, d = idx - r * qhd;
         int qi = r / group, g = r - qi * group;
-        q_s[idx] = to_float(q[(size_t)(row0 + qi) * p.q_stride + (size_t)(kvh * group + g) * hd + d]);
+        q_s[idx] = to_float(q[(size_t)(row0 + qi) * p.q_stride + (size_t)(kvh * group + g) * qhd + d]);
     }
     for (int idx = tid; idx < n_rows * vd; idx += ATT_THREADS) acc_s[idx] = 0.0f;
     for (int r = tid; r < n_rows; r += ATT_THREADS) { m_s[r] = -INFINITY; l_s[r] = 0.0f; }
@@ -137,7 +139,8 @@ attention_partial_kernel(AttnParams p) {
             const int qi = r / group;
             const int pos = p.positions[row0 + qi];
             const int lo = first_visible(pos, p.window);
-            const float* qr = q_s + (size_t)r * hd;
+            const float* qr = q_s + (size_t)r * qhd;
+            const int map_off = (r % group) % p.maps * qhd;
             float s[2];
             float tmax = -INFINITY;
 #pragma unroll
@@ -147,9 +150,9 @@ attention_partial_kernel(AttnParams p) {
                 if (j < tile) {
                     int key = t0 + j;
                     if (key_seen(key, lo, p.keep) && key <= pos && key < k_end && base_s[j] >= 0) {
-                        const float* kr = k_s + j * kstride;
+                        const float* kr = k_s + j * kstride + map_off;
                         float dot = 0.0f;
-                        for (int d = 0; d < hd; ++d) dot = fmaf(qr[d], kr[d], dot);
+                        for (int d = 0; d < qhd; ++d) dot = fmaf(qr[d], kr[d], dot);
                         s[c] = dot * p.scale;
                         if (p.softcap > 0.0f) s[c] = p.softcap * tanhf(s[c] / p.softcap);
                         if (p.slopes) s[c] -= p.slopes[kvh * group + r % group] * (float)(pos - key);
@@ -316,8 +319,9 @@ static size_t attention_smem_bytes(int bq, int group, int hd, int vd, int tile) 
 
 // Rows per query block and keys per tile that fit the shared memory of one CTA for these sizes.
 // Returns 0 and fills bq and tile, or BG_ERR_UNSUPPORTED.
-extern "C" int bg_attention_plan(int group, int hd, int vd, int* bq_out, int* tile_out) {
-    if (hd <= 0 || hd > 32 * ATT_MAX_DPL || vd <= 0 || vd > 32 * ATT_MAX_DPL || group <= 0) return BG_ERR_UNSUPPORTED;
+// (`hd` counts a whole key row; with two maps in it, it may be twice as wide)
+extern "C" int bg_attention_plan(int group, int hd, int vd, int maps, int* bq_out, int* tile_out) {
+    if (maps < 1 || hd <= 0 || hd > 32 * ATT_MAX_DPL * maps || vd <= 0 || vd > 32 * ATT_MAX_DPL || group <= 0) return BG_ERR_UNSUPPORTED;
     const size_t limit = 200 * 1024;
     for (int tile = 64; tile >= 32; tile >>= 1) {
         for (int bq = 16; bq >= 1; bq >>= 1) {
@@ -331,17 +335,18 @@ extern "C" int bg_attention_partial(const void* q, int q_dtype, int q_stride, co
                                     int num_pages, int page_size, const int* block_table, int max_pages,
                                     const int* positions, const int* qblk, int n_qblk, float* part_o, float* part_ml,
                                     int max_splits, int n_splits_launch, int nh, int nkv, int hd, int vd, int window, int split,
-                                    int tile, int bq, float scale, float softcap, int keep, const float* slopes, unsigned* status,
-                                    cudaStream_t stream) {
+                                    int tile, int bq, float scale, float softcap, int keep, const float* slopes, int maps,
+                                    unsigned* status, cudaStream_t stream) {
     if (n_qblk <= 0 || n_splits_launch <= 0) return BG_OK;
-    if (nh % nkv != 0 || hd > 32 * ATT_MAX_DPL || vd <= 0 || vd > 32 * ATT_MAX_DPL || (tile != 32 && tile != 64) || split % tile != 0) return BG_ERR_SHAPE;
+    if (maps < 1 || hd % maps || (nh / nkv) % maps) return BG_ERR_SHAPE;
+    if (nh % nkv != 0 || hd > 32 * ATT_MAX_DPL * maps || vd <= 0 || vd > 32 * ATT_MAX_DPL || (tile != 32 && tile != 64) || split % tile != 0) return BG_ERR_SHAPE;
     if (n_splits_launch > max_splits || n_splits_launch > 65535 || nkv > 65535 || keep < 0) return BG_ERR_SHAPE;
     AttnParams p;
     p.q = q; p.q_stride = q_stride; p.kv_pool = kv_pool; p.num_pages = num_pages; p.page_size = page_size;
     p.block_table = block_table; p.max_pages = max_pages; p.positions = positions; p.qblk = qblk;
     p.part_o = part_o; p.part_ml = part_ml; p.max_splits = max_splits; p.nh = nh; p.nkv = nkv; p.hd = hd; p.vd = vd;
     p.group = nh / nkv; p.window = window; p.split = split; p.tile = tile; p.bq = bq; p.scale = scale; p.softcap = softcap; p.status = status;
-    p.keep = keep; p.slopes = slopes;
+    p.keep = keep; p.slopes = slopes; p.maps = maps;
     size_t smem = attention_smem_bytes(bq, p.group, hd, vd, tile);
     if (smem > 227 * 1024) return BG_ERR_UNSUPPORTED;
     dim3 grid(n_qblk, nkv, n_splits_launch);

@@ -66,6 +66,14 @@ struct AttnTcParams {
     unsigned* status;
 };
 
+// What the DIFF instances take besides.
+struct AttnTcDiffParams : AttnTcParams {
+    int vd;                     // a head's own features of the HD that its values are stored in
+    float lambda, out_scale, eps;
+};
+template <bool DIFF> struct AtParams { using type = AttnTcParams; };
+template <> struct AtParams<true> { using type = AttnTcDiffParams; };
+
 __device__ __forceinline__ bool at_elect() {
     unsigned one;
     asm volatile("{\n .reg .pred p;\n elect.sync _|p, 0xffffffff;\n selp.u32 %0, 1, 0, p;\n}\n" : "=r"(one));
@@ -89,9 +97,17 @@ __device__ __forceinline__ float at_squash(float x, float cap_log2, float cap_k)
 // maximum and exp2(0 - maximum) into the sum; nothing else differs, and the plain instance is compiled as before.
 // EXT: scores fall with the distance by a slope of the head, and a window never loses the first `keep` positions: the
 // tiles are then those of the kept positions followed by those of the window, the tiles between passed over.
-template <int HD, int AT_BK, bool SINK = false, bool EXT = false>
+// DIFF: differential attention.  A query head is a pair of maps: a query row and a key row hold HD / 2 features of the first
+// map followed by those of the second, and both maps weigh the same values of HD features.  Here the two groups of softmax
+// warps are the two maps: every tile of 64 keys is taken twice, a turn for each (turn i is map i % 2 of tile i / 2: a score
+// product over the map's half of the features, then the product with the tile's values into the map's own O), so a tile of
+// keys and values is fetched once for both.  At the end the maps are not joined but subtracted, and the difference is normed:
+// out = o / sqrt(mean(o^2) + eps) * out_scale with o = O_0 / l_0 - lambda O_1 / l_1, the first `vd` of the HD features stored.
+// A stage of the rings serves two turns, so its release has barriers of its own (k_free, v_free).
+template <int HD, int AT_BK, bool SINK = false, bool EXT = false, bool DIFF = false>
 __global__ void __launch_bounds__(AT_THREADS)
-attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParams p) {
+attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, typename AtParams<DIFF>::type p) {
+    static_assert(!DIFF || (AT_BK == 64 && !SINK && !EXT), "the two maps take tiles of 64 keys in turns");
     constexpr int AT_HALF = AT_BK / 2, AT_STAGES = 256 / AT_BK;
     constexpr int NSB = AT_STAGES;                       // score buffers in tensor memory: tiles whose scores may be under way
     // How the two groups of softmax warps share the keys.  Tiles of 128 keys: every tile is cut in two halves, one for
@@ -122,6 +138,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
     // overwritten, the softmax warps that O may be rescaled, and the value loader that the stage is free.
     __shared__ __align__(8) unsigned long long k_full[AT_STAGES], v_full[AT_STAGES], kv_landed[AT_STAGES];
     __shared__ __align__(8) unsigned long long s_full[NSB], p_full[2 * NSB], pv_done[NSB], o_ready;    // p_full: [2 buffer + group]
+    __shared__ __align__(8) unsigned long long k_free[DIFF ? AT_STAGES : 1], v_free[DIFF ? AT_STAGES : 1];
     __shared__ float2 ml_other[AT_BM];                   // the second group's running maximum and sum of every row, for the join
     __shared__ unsigned tmem_sh;
     __shared__ int failed;
@@ -137,6 +154,9 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
         for (int b = 0; b < NSB; ++b) { mbar_init(&s_full[b], 1); mbar_init(&pv_done[b], 1); }
         for (int b = 0; b < 2 * NSB; ++b) mbar_init(&p_full[b], 4);       // one arrival per softmax warp of a group
         mbar_init(&o_ready, 1);
+        if constexpr (DIFF) {
+            for (int s = 0; s < AT_STAGES; ++s) { mbar_init(&k_free[s], 1); mbar_init(&v_free[s], 1); }
+        }
         failed = 0;
         mbar_init_fence();
     }
@@ -156,6 +176,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
     const int n_kept = EXT ? (min(keep, k_end) + AT_BK - 1) / AT_BK : 0;         // tiles with kept positions
     const int tile0 = EXT ? max(k_begin / AT_BK, n_kept) : k_begin / AT_BK;      // the window's first tile behind those
     const int n_tiles = EXT ? n_kept + max((k_end + AT_BK - 1) / AT_BK - tile0, 0) : (k_end + AT_BK - 1) / AT_BK - tile0;
+    const int n_turns = DIFF ? 2 * n_tiles : n_tiles;            // a turn: one score product and one softmax group's share of a tile
     auto tile_key = [&](int i) { return (EXT && i < n_kept ? i : tile0 + i - n_kept) * AT_BK; };
 
     // ---- Q into shared memory: row r, column block cb, 16-byte piece c at r*128 + ((c ^ (r & 7)) * 16)
@@ -195,14 +216,15 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
         if (warp == 0) {
             // scores: S[b] = Q K(i)^T as soon as the keys have landed and both groups' P of the buffer's last tile
             // have been used up
-            for (int i = 0; i < n_tiles && ok; ++i) {
-                const int st = i % AT_STAGES, b = i % NSB;
+            for (int i = 0; i < n_turns && ok; ++i) {
+                const int tile = DIFF ? i >> 1 : i, map = DIFF ? i & 1 : 0;
+                const int st = tile % AT_STAGES, b = i % NSB;
                 // (which of the two waits comes first is measured: with four score buffers the older event, the
                 // buffer's release, first: 234 -> 227 us at 8,192 tokens; with two buffers the keys first: 812
                 // against 864 us at 16,384 tokens)
                 if (ALT) {
                     if (i >= NSB) ok = wait_all(&pv_done[b], ((i / NSB) - 1) & 1);
-                    if (ok) ok = wait_all(&k_full[st], (i / AT_STAGES) & 1);
+                    if (ok && map == 0) ok = wait_all(&k_full[st], (tile / AT_STAGES) & 1);
                 } else {
                     ok = wait_all(&k_full[st], (i / AT_STAGES) & 1);
                     if (ok && i >= NSB) ok = wait_all(&pv_done[b], ((i / NSB) - 1) & 1);
@@ -211,21 +233,35 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
                 tc_fence_after();
                 const unsigned k_addr = smem_u32(k_s + st * KV_BYTES);
                 if (at_elect()) {
+                    if constexpr (DIFF) {                // the map's half of the features
+                        constexpr int HALF_STEPS = HD / 32;
 #pragma unroll
-                    for (int ks = 0; ks < HD / 16; ++ks) {
-                        const unsigned off = (ks & 3) * 32;
-                        tc_mma(tmem + (unsigned)b * AT_BK, smem_desc_sw128(q_addr + (ks >> 2) * (AT_BM * 128) + off),
-                               smem_desc_sw128(k_addr + (ks >> 2) * KV_BLOCK + off), idesc_qk, ks > 0 ? 1u : 0u);
+                        for (int kk = 0; kk < HALF_STEPS; ++kk) {
+                            const int ks = map * HALF_STEPS + kk;
+                            const unsigned off = (ks & 3) * 32;
+                            tc_mma(tmem + (unsigned)b * AT_BK, smem_desc_sw128(q_addr + (ks >> 2) * (AT_BM * 128) + off),
+                                   smem_desc_sw128(k_addr + (ks >> 2) * KV_BLOCK + off), idesc_qk, kk > 0 ? 1u : 0u);
+                        }
+                        tc_commit(&s_full[b]);
+                        if (map == 1) tc_commit(&k_free[st]);
+                    } else {
+#pragma unroll
+                        for (int ks = 0; ks < HD / 16; ++ks) {
+                            const unsigned off = (ks & 3) * 32;
+                            tc_mma(tmem + (unsigned)b * AT_BK, smem_desc_sw128(q_addr + (ks >> 2) * (AT_BM * 128) + off),
+                                   smem_desc_sw128(k_addr + (ks >> 2) * KV_BLOCK + off), idesc_qk, ks > 0 ? 1u : 0u);
+                        }
+                        tc_commit(&s_full[b]);
                     }
-                    tc_commit(&s_full[b]);
                 }
                 __syncwarp();
             }
         } else {
             // values: O[g] += P(i, g) V(i, g) once group g's softmax warps have written their half of P
-            for (int i = 0; i < n_tiles && ok; ++i) {
-                const int st = i % AT_STAGES, b = i % NSB;
-                ok = wait_all(&v_full[st], (i / AT_STAGES) & 1);
+            for (int i = 0; i < n_turns && ok; ++i) {
+                const int tile = DIFF ? i >> 1 : i;
+                const int st = tile % AT_STAGES, b = i % NSB;
+                if (!DIFF || (i & 1) == 0) ok = wait_all(&v_full[st], (tile / AT_STAGES) & 1);
                 const unsigned v_addr = smem_u32(v_s + st * KV_BYTES);
                 if constexpr (ALT) {
                     const int g = i & 1;
@@ -238,6 +274,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
                             tc_mma_ts(tmem + O_COL + 128u * (unsigned)g, tmem + (unsigned)b * AT_BK + (unsigned)ks * 8,
                                       smem_desc_sw128_nmajor(v_addr + ks * 2048, KV_BLOCK, 1024), idesc_pv, (i >= 2 || ks > 0) ? 1u : 0u);
                         tc_commit(&pv_done[b]);
+                        if (DIFF && g == 1) tc_commit(&v_free[st]);
                     }
                     __syncwarp();
                 } else {
@@ -280,10 +317,10 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
         const float sl2 = (capped || EXT) ? 1.0f : p.scale_log2;
         const float slope_l2 = (EXT && p.slopes && real) ? p.slopes[kvh * group + r % group] * AT_LOG2E : 0.0f;
         const int i_first = ALT ? grp : 0;                   // this group's first tile
-        for (int i = i_first; i < n_tiles && ok; i += (ALT ? 2 : 1)) {
+        for (int i = i_first; i < n_turns && ok; i += (ALT ? 2 : 1)) {
             const int b = i % NSB;
             const unsigned s_col = (unsigned)b * AT_BK + (ALT ? 0u : (unsigned)grp * AT_HALF);    // this group's scores of the tile, and its P
-            const int key0 = tile_key(i) + (ALT ? 0 : grp * AT_HALF);
+            const int key0 = tile_key(DIFF ? i >> 1 : i) + (ALT ? 0 : grp * AT_HALF);
             ok = mbar_wait(&s_full[b], (i / NSB) & 1);
             if (!ok) break;
             tc_fence_after();
@@ -360,7 +397,47 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
         // same row (the same lanes of tensor memory) reads both accumulators
         if (grp == 1) ml_other[r] = make_float2(m, l);
         asm volatile("bar.sync 1, 256;\n" ::: "memory");
-        if (grp == 0 && ok && n_tiles > 0) {
+        if constexpr (DIFF) {
+            if (grp == 0 && ok && n_tiles > 0) {
+                tc_fence_after();
+                const float l1 = ml_other[r].y;
+                const int qi = real ? r / group : 0, g = real ? r - qi * group : 0;
+                const float w0 = real ? 1.0f / l : 0.0f, w1 = real ? p.lambda / l1 : 0.0f;
+                float ss = 0.0f;
+#pragma unroll
+                for (int c0 = 0; c0 < HD; c0 += 32) {    // (features behind a head's own are zeros of the cache)
+                    float t[32], u[32];
+                    tc_ld32(tmem + lane_addr + O_COL + c0, t);
+                    tc_ld32(tmem + lane_addr + O_COL + 128u + c0, u);
+#pragma unroll
+                    for (int q = 0; q < 32; ++q) { const float v = t[q] * w0 - u[q] * w1; ss = fmaf(v, v, ss); }
+                }
+                const float mult = p.out_scale / sqrtf(ss / (float)p.vd + p.eps);
+                const float a0 = w0 * mult, a1 = w1 * mult;
+                __nv_bfloat16* o = p.out + (size_t)(row0 + qi) * p.out_stride + (size_t)(kvh * group + g) * p.vd;
+                const bool whole = (p.vd & 7) == 0;      // 16-byte stores
+#pragma unroll
+                for (int c0 = 0; c0 < HD; c0 += 32) {
+                    float t[32], u[32];
+                    tc_ld32(tmem + lane_addr + O_COL + c0, t);
+                    tc_ld32(tmem + lane_addr + O_COL + 128u + c0, u);
+                    if (!real) continue;
+#pragma unroll
+                    for (int q = 0; q < 32; q += 8) {
+                        float v8[8];
+#pragma unroll
+                        for (int k = 0; k < 8; ++k) v8[k] = t[q + k] * a0 - u[q + k] * a1;
+                        if (whole) {
+                            if (c0 + q < p.vd) store8(o + c0 + q, v8);
+                        } else {
+#pragma unroll
+                            for (int k = 0; k < 8; ++k)
+                                if (c0 + q + k < p.vd) o[c0 + q + k] = __float2bfloat16_rn(v8[k]);
+                        }
+                    }
+                }
+            }
+        } else if (grp == 0 && ok && n_tiles > 0) {
             tc_fence_after();
             const float2 other = ml_other[r];
             const float m_all = fmaxf(m, other.x);
@@ -399,7 +476,7 @@ attention_tcgen05_kernel(const __grid_constant__ CUtensorMap map_kv, AttnTcParam
         const int lsub = warp >= 12;
         unsigned char* ring = which ? v_s : k_s;
         unsigned long long* full = which ? v_full : k_full;
-        unsigned long long* empty = which ? pv_done : s_full;      // AT_STAGES == NSB: stage st is buffer st
+        unsigned long long* empty = DIFF ? (which ? v_free : k_free) : (which ? pv_done : s_full);      // AT_STAGES == NSB: stage st is buffer st
         const int ps = p.page_size, sh = p.page_shift;   // the page size is a power of two
         const int n_pg = AT_BK >> sh;                    // pages per tile (page_size divides 64)
         bool ok = true;
@@ -502,6 +579,18 @@ static int at_launch(const CUtensorMap& map, const AttnTcParams& p, int n_qblk, 
     return BG_OK;
 }
 
+// The same for differential attention (tiles of 64 keys).
+template <int HD>
+static int at_launch_difference(const CUtensorMap& map, const AttnTcDiffParams& p, int n_qblk, cudaStream_t stream) {
+    auto kern = attention_tcgen05_kernel<HD, 64, false, false, true>;
+    const size_t smem = (size_t)(HD / 64) * AT_BM * 128 + (size_t)2 * 256 * (HD / 64) * 128 + 1024;
+    cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+    if (e != cudaSuccess) return (int)e;
+    e = launch(kern, dim3(p.nkv, n_qblk), dim3(AT_THREADS), smem, stream, map, p);
+    if (e != cudaSuccess) return (int)e;
+    return BG_OK;
+}
+
 }  // namespace bg
 
 using namespace bg;
@@ -591,4 +680,32 @@ extern "C" int bg_attention_tc_ext(const void* q, int q_stride, const void* kv_p
     return attention_tc(q, q_stride, kv_pool, num_pages, page_size, block_table, max_pages, positions, qblk, n_qblk, out, out_stride,
                         nh, nkv, hd, window, scale, max_position, sink != 0 || sink_weight != nullptr, status, stream, sink_weight,
                         softcap, keep, slopes);
+}
+
+// Differential attention of prompt portions: q [T][nh][2][hd / 2], the pages' key rows [2][hd / 2] and values of hd features of
+// which a head's own are the first vd; out [T][nh * vd], the normed difference of the two maps (see the kernel).
+extern "C" int bg_attention_tc_difference(const void* q, int q_stride, const void* kv_pool, int num_pages, int page_size,
+                                          const int* block_table, int max_pages, const int* positions, const int* qblk, int n_qblk,
+                                          void* out, int out_stride, int nh, int nkv, int hd, int vd, int window, float scale,
+                                          float lambda, float out_scale, float eps, unsigned* status, cudaStream_t stream) {
+    if (n_qblk <= 0) return BG_OK;
+    if (nkv <= 0 || nh % nkv != 0 || (hd != 64 && hd != 128) || nh / nkv > 128 || !(scale > 0.0f)) return BG_ERR_UNSUPPORTED;
+    if (page_size < 1 || page_size > 64 || 64 % page_size != 0) return BG_ERR_UNSUPPORTED;
+    if (vd < 1 || vd > hd || n_qblk > 65535) return BG_ERR_SHAPE;
+    if ((q_stride % 8) || ((uintptr_t)q % 16) || ((uintptr_t)kv_pool % 16)) return BG_ERR_ALIGN;
+    if (vd % 8 == 0 && ((out_stride % 8) || ((uintptr_t)out % 16))) return BG_ERR_ALIGN;
+    AttnTcDiffParams p;
+    memset(&p, 0, sizeof(p));
+    p.q = (const __nv_bfloat16*)q; p.q_stride = q_stride; p.kv_pool = (const __nv_bfloat16*)kv_pool;
+    p.num_pages = num_pages; p.page_size = page_size; p.page_shift = -1;
+    for (int sh = 0; sh < 30; ++sh) if ((1 << sh) == page_size) p.page_shift = sh;
+    p.block_table = block_table; p.max_pages = max_pages; p.positions = positions; p.qblk = qblk;
+    p.out = (__nv_bfloat16*)out; p.out_stride = out_stride; p.nh = nh; p.nkv = nkv; p.group = nh / nkv;
+    p.window = window; p.scale_log2 = scale * AT_LOG2E; p.status = status;
+    p.vd = vd; p.lambda = lambda; p.out_scale = out_scale; p.eps = eps;
+    CUtensorMap map;
+    int rc = pt_pool_map(&map, kv_pool, num_pages, nkv, page_size, hd);
+    if (rc != BG_OK) return rc;
+    if (hd == 128) return at_launch_difference<128>(map, p, n_qblk, stream);
+    return at_launch_difference<64>(map, p, n_qblk, stream);
 }

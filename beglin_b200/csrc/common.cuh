@@ -210,6 +210,15 @@ __device__ __forceinline__ void store8(__nv_bfloat16* p, const float (&v)[8]) {
     *reinterpret_cast<uint4*>(p) = raw;
 }
 
+// g sigmoid(1.702 g) (u + 1) with g cut off above and u on both sides at `limit`.  FAST: the hardware's exponential and division
+// (for a result that is rounded to bfloat16); else expf and a division.
+template <bool FAST>
+__device__ __forceinline__ float glu_clamped_value(float gate, float up, float limit) {
+    const float g = fminf(gate, limit), u = fminf(fmaxf(up, -limit), limit);
+    if constexpr (FAST) return __fdividef(g, 1.0f + __expf(-1.702f * g)) * (u + 1.0f);
+    else return g / (1.0f + expf(-1.702f * g)) * (u + 1.0f);
+}
+
 // Sum of `parts` float4 values that lie `stride4` float4 apart, added in index order.  For up to sixteen parts the
 // count picks a branch with exactly that many loads and no condition among them, so that they all go out together
 // and the sum costs one round trip (with a condition on every load the compiler kept few of them in flight: the

@@ -329,8 +329,11 @@ __global__ void add_residual_kernel(float* __restrict__ x, const TD* __restrict_
 // instead of by these two functions; a float result is computed with expf and a division.
 // ACT 0: silu.  ACT 1: the tanh form of GELU, 0.5 g (1 + tanh(sqrt(2/pi) (g + 0.044715 g^3))), which is
 // g * sigmoid(2 sqrt(2/pi) (g + 0.044715 g^3)); a float result takes tanhf.  ACT 2: the square of relu.
-template <typename TO, int ACT> __device__ __forceinline__ float silu_mul(float g, float u) {
-    if constexpr (ACT == 0) {
+// ACT 3: the clamped form, glu_clamped_value with `limit`.
+template <typename TO, int ACT> __device__ __forceinline__ float silu_mul(float g, float u, float limit = 0.0f) {
+    if constexpr (ACT == 3) {
+        return glu_clamped_value<!std::is_same<TO, float>::value>(g, u, limit);
+    } else if constexpr (ACT == 0) {
         if constexpr (std::is_same<TO, float>::value) return (g / (1.0f + expf(-g))) * u;
         else return __fdividef(g, 1.0f + __expf(-g)) * u;
     } else if constexpr (ACT == 2) {
@@ -345,7 +348,7 @@ template <typename TO, int ACT> __device__ __forceinline__ float silu_mul(float 
 
 template <typename TI, typename TO, int ACT>
 __global__ void swiglu_kernel(const TI* __restrict__ gu, int parts, size_t part_stride, TO* __restrict__ out,
-                              int rows, int im, int block) {
+                              int rows, int im, int block, float limit) {
     pdl_launch();
     // where this thread's values lie is integer arithmetic (divisions) on the grid alone: done before the wait
     size_t idx = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -359,14 +362,14 @@ __global__ void swiglu_kernel(const TI* __restrict__ gu, int parts, size_t part_
     if (idle) return;
     float g = sum_parts(gp, parts, part_stride);
     float u = sum_parts(gp + (block > 0 ? block : im), parts, part_stride);
-    out[idx] = from_float<TO>(silu_mul<TO, ACT>(g, u));
+    out[idx] = from_float<TO>(silu_mul<TO, ACT>(g, u, limit));
 }
 
 // Float partial sums, im and block multiples of 4: four features per thread, 16-byte loads, the parts added in
 // index order as above.
 template <typename TO, int ACT>
 __global__ void swiglu_parts_vec4_kernel(const float* __restrict__ gu, int parts, size_t part_stride, TO* __restrict__ out,
-                                         int rows, int im, int block) {
+                                         int rows, int im, int block, float limit) {
     pdl_launch();
     const int im4 = im >> 2;
     const unsigned idx = blockIdx.x * blockDim.x + threadIdx.x;          // (the launcher keeps rows * im / 4 under 2^32)
@@ -379,7 +382,7 @@ __global__ void swiglu_parts_vec4_kernel(const float* __restrict__ gu, int parts
     if (idle) return;
     const float4 g = sum_parts4(gp, parts, part_stride / 4);
     const float4 u = sum_parts4(gp + (block > 0 ? block : im) / 4, parts, part_stride / 4);
-    const float r[4] = {silu_mul<TO, ACT>(g.x, u.x), silu_mul<TO, ACT>(g.y, u.y), silu_mul<TO, ACT>(g.z, u.z), silu_mul<TO, ACT>(g.w, u.w)};
+    const float r[4] = {silu_mul<TO, ACT>(g.x, u.x, limit), silu_mul<TO, ACT>(g.y, u.y, limit), silu_mul<TO, ACT>(g.z, u.z, limit), silu_mul<TO, ACT>(g.w, u.w, limit)};
     TO* o = out + (size_t)t * (size_t)im + i;
     if constexpr (std::is_same<TO, float>::value) {
         *reinterpret_cast<float4*>(o) = make_float4(r[0], r[1], r[2], r[3]);
@@ -394,7 +397,7 @@ __global__ void swiglu_parts_vec4_kernel(const float* __restrict__ gu, int parts
 
 // One tensor (no partial sums), im a multiple of 8: eight features per thread, 16-byte accesses.
 template <typename TI, typename TO, int ACT>
-__global__ void swiglu_vec8_kernel(const TI* __restrict__ gu, TO* __restrict__ out, int rows, int im, int block) {
+__global__ void swiglu_vec8_kernel(const TI* __restrict__ gu, TO* __restrict__ out, int rows, int im, int block, float limit) {
     pdl_launch();
     const int im8 = im >> 3;
     const unsigned idx = blockIdx.x * blockDim.x + threadIdx.x;          // (the launcher keeps rows * im / 8 under 2^32)
@@ -409,7 +412,7 @@ __global__ void swiglu_vec8_kernel(const TI* __restrict__ gu, TO* __restrict__ o
     load8(gu + t * 2 * (size_t)im + col, g);
     load8(gu + t * 2 * (size_t)im + col + (block > 0 ? block : im), u);
 #pragma unroll
-    for (int i = 0; i < 8; ++i) g[i] = silu_mul<TO, ACT>(g[i], u[i]);
+    for (int i = 0; i < 8; ++i) g[i] = silu_mul<TO, ACT>(g[i], u[i], limit);
     store8(out + t * (size_t)im + 8 * c, g);
 }
 
@@ -756,25 +759,25 @@ extern "C" int bg_add_residual(float* x, const void* delta, int delta_dtype, lon
 
 template <typename TI, int ACT>
 static int swiglu_in(const void* gu, int parts, size_t part_stride, void* out, int out_dtype, int rows, int im, int block,
-                     cudaStream_t stream) {
+                     float limit, cudaStream_t stream) {
     const bool small = (size_t)rows * (size_t)im < (1ull << 32);          // the vector kernels count their pieces in 32 bits
     const bool vec = small && parts == 1 && (im % 8 == 0) && (block % 8 == 0) && ((uintptr_t)gu % 16 == 0) && ((uintptr_t)out % 16 == 0);
     if (vec) {
         size_t total = (size_t)rows * (im / 8);
         unsigned blocks = (unsigned)((total + 255) / 256);
         BG_DISPATCH_DTYPE(out_dtype, TO, launch(swiglu_vec8_kernel<TI, TO, ACT>, dim3(blocks), dim3(256), 0, stream,
-            (const TI*)gu, (TO*)out, rows, im, block));
+            (const TI*)gu, (TO*)out, rows, im, block, limit));
     } else if (small && std::is_same<TI, float>::value && (im % 4 == 0) && (block % 4 == 0) && (part_stride % 4 == 0) &&
                ((uintptr_t)gu % 16 == 0) && ((uintptr_t)out % 16 == 0)) {
         size_t total = (size_t)rows * (im / 4);
         unsigned blocks = (unsigned)((total + 255) / 256);
         BG_DISPATCH_DTYPE(out_dtype, TO, launch(swiglu_parts_vec4_kernel<TO, ACT>, dim3(blocks), dim3(256), 0, stream,
-            (const float*)gu, parts, part_stride, (TO*)out, rows, im, block));
+            (const float*)gu, parts, part_stride, (TO*)out, rows, im, block, limit));
     } else {
         size_t total = (size_t)rows * im;
         unsigned blocks = (unsigned)((total + 255) / 256);
         BG_DISPATCH_DTYPE(out_dtype, TO, launch(swiglu_kernel<TI, TO, ACT>, dim3(blocks), dim3(256), 0, stream,
-            (const TI*)gu, parts, part_stride, (TO*)out, rows, im, block));
+            (const TI*)gu, parts, part_stride, (TO*)out, rows, im, block, limit));
     }
     BG_LAUNCH_CHECK();
     return BG_OK;
@@ -837,11 +840,12 @@ extern "C" int bg_activation(const void* z, int in_dtype, int parts, long long p
 }
 
 extern "C" int bg_swiglu(const void* gu, int in_dtype, int parts, long long part_stride, void* out, int out_dtype,
-                         int rows, int im, int block, int act, cudaStream_t stream) {
+                         int rows, int im, int block, int act, float limit, cudaStream_t stream) {
     if (rows <= 0) return BG_OK;
-    if (parts < 1 || block < 0 || (block > 0 && im % block != 0) || act < 0 || act > 1) return BG_ERR_SHAPE;
-    if (act == 0) BG_DISPATCH_DTYPE(in_dtype, TI, return (swiglu_in<TI, 0>(gu, parts, (size_t)part_stride, out, out_dtype, rows, im, block, stream)));
-    else BG_DISPATCH_DTYPE(in_dtype, TI, return (swiglu_in<TI, 1>(gu, parts, (size_t)part_stride, out, out_dtype, rows, im, block, stream)));
+    if (parts < 1 || block < 0 || (block > 0 && im % block != 0) || act < 0 || act > 3 || act == 2 || (act == 3 && !(limit > 0.0f))) return BG_ERR_SHAPE;
+    if (act == 3) BG_DISPATCH_DTYPE(in_dtype, TI, return (swiglu_in<TI, 3>(gu, parts, (size_t)part_stride, out, out_dtype, rows, im, block, limit, stream)));
+    if (act == 0) BG_DISPATCH_DTYPE(in_dtype, TI, return (swiglu_in<TI, 0>(gu, parts, (size_t)part_stride, out, out_dtype, rows, im, block, limit, stream)));
+    else BG_DISPATCH_DTYPE(in_dtype, TI, return (swiglu_in<TI, 1>(gu, parts, (size_t)part_stride, out, out_dtype, rows, im, block, limit, stream)));
     return BG_OK;
 }
 

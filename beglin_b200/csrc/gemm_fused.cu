@@ -69,7 +69,14 @@ struct RopeParams {
     __nv_bfloat16* kv_pool;         // [num_pages][2][nkv][page_size][hd]
     int max_pages, num_pages, page_size, nh, nkv;
 };
+// What the clamped form of the gated mode needs beside: where its two branches are cut off.
+struct LimitParams { float limit; };
 struct NoRope {};
+// The kinds of instances: 0 every mode but those of the other two, 1 the rope mode, 2 the clamped gated mode.
+constexpr int GF_KIND_BASE = 0, GF_KIND_ROPE = 1, GF_KIND_CLAMPED = 2;
+template <int KIND> struct GfExtra { using type = NoRope; };
+template <> struct GfExtra<GF_KIND_ROPE> { using type = RopeParams; };
+template <> struct GfExtra<GF_KIND_CLAMPED> { using type = LimitParams; };
 
 // Pair j of a tile is rows row_of_pair(j) and row_of_pair(j) + (1 << pair_log).
 __device__ __forceinline__ int pair_of_row(int m, int pair_log) { return ((m >> (pair_log + 1)) << pair_log) | (m & ((1 << pair_log) - 1)); }
@@ -99,12 +106,13 @@ __device__ __forceinline__ float ranks_sum(const float* rp, int part, int S) {
 
 __device__ __forceinline__ void epilogue_sync() { asm volatile("bar.sync 1, 128;\n" ::: "memory"); }   // warps 2..5
 
-// ROPE: the kernel of the rope mode is an instance of its own, so that the other modes' code (and what the compiler
-// makes of it) does not change with it.
-template <int BN, int STAGES, bool ROPE>
+// KIND: the kernels of the rope mode and of the clamped gated mode are instances of their own, so that the other modes' code
+// (and what the compiler makes of it) does not change with them.
+template <int BN, int STAGES, int KIND>
 __global__ void __launch_bounds__(TC_THREADS)
 gemm_fused_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_x, FusedParams p,
-                  typename std::conditional<ROPE, RopeParams, NoRope>::type r) {
+                  typename GfExtra<KIND>::type r) {
+    constexpr bool ROPE = KIND == GF_KIND_ROPE;
     constexpr unsigned A_BYTES = TC_BM * TC_BK * 2;
     constexpr unsigned B_BYTES = BN * TC_BK * 2;
     constexpr unsigned STAGE_BYTES = A_BYTES + B_BYTES;
@@ -483,8 +491,10 @@ gemm_fused_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_consta
             for (int c = te >> (6 - p.log_splits); c < t_real; c += 2 << p.log_splits) {
                 const float g = ranks_sum(recv + c * rows_per + i, part, S) + bias_g;
                 const float u = ranks_sum(recv + c * rows_per + half + i, part, S) + bias_u;
-                ((__nv_bfloat16*)p.out)[(size_t)(tile_n * BN + c) * p.ldo + tile_m * 64 + rank * half + i] =
-                    __float2bfloat16_rn(__fdividef(g, 1.0f + __expf(-g)) * u);   // as the SwiGLU kernel does for a bfloat16 result
+                float v;
+                if constexpr (KIND == GF_KIND_CLAMPED) v = glu_clamped_value<true>(g, u, r.limit);
+                else v = __fdividef(g, 1.0f + __expf(-g)) * u;                 // as the SwiGLU kernel does for a bfloat16 result
+                ((__nv_bfloat16*)p.out)[(size_t)(tile_n * BN + c) * p.ldo + tile_m * 64 + rank * half + i] = __float2bfloat16_rn(v);
             }
         }
     }
@@ -496,10 +506,10 @@ gemm_fused_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_consta
     if (threadIdx.x == 0 && failed && p.status) atomicOr(p.status, BG_STATUS_TIMEOUT);
 }
 
-template <int BN, int STAGES, bool ROPE>
-static int gf_launch_stages(const CUtensorMap& mw, const CUtensorMap& mx, const FusedParams& p, const RopeParams* rope,
+template <int BN, int STAGES, int KIND>
+static int gf_launch_stages(const CUtensorMap& mw, const CUtensorMap& mx, const FusedParams& p, const typename GfExtra<KIND>::type& extra,
                             cudaStream_t stream) {
-    auto kern = gemm_fused_kernel<BN, STAGES, ROPE>;
+    auto kern = gemm_fused_kernel<BN, STAGES, KIND>;
     size_t smem = (size_t)STAGES * (TC_BM * TC_BK * 2 + BN * TC_BK * 2) + (size_t)BN * TC_BM * 4 + 1024;
     static bool set = false;
     if (!set) {
@@ -510,9 +520,7 @@ static int gf_launch_stages(const CUtensorMap& mw, const CUtensorMap& mx, const 
         set = true;
     }
     dim3 grid((p.n_out + TC_BM - 1) / TC_BM, (p.T + BN - 1) / BN, p.splits);
-    cudaError_t e;
-    if constexpr (ROPE) e = launch_cluster(kern, grid, dim3(TC_THREADS), smem, stream, p.splits, mw, mx, p, *rope);
-    else e = launch_cluster(kern, grid, dim3(TC_THREADS), smem, stream, p.splits, mw, mx, p, NoRope());
+    cudaError_t e = launch_cluster(kern, grid, dim3(TC_THREADS), smem, stream, p.splits, mw, mx, p, extra);
     if (e != cudaSuccess) return (int)e;
     BG_LAUNCH_CHECK();
     return BG_OK;
@@ -520,16 +528,19 @@ static int gf_launch_stages(const CUtensorMap& mw, const CUtensorMap& mx, const 
 
 // A grid that leaves SMs to spare has a CTA alone on its SM: eight stages then keep enough bytes on their way
 // from HBM (the stream of a few CTAs is bound by what they have in flight); else four, so that two CTAs share an SM.
-template <int BN>
-static int gf_launch(const CUtensorMap& mw, const CUtensorMap& mx, const FusedParams& p, const RopeParams* rope,
-                     cudaStream_t stream) {
+template <int BN, int KIND>
+static int gf_launch_kind(const CUtensorMap& mw, const CUtensorMap& mx, const FusedParams& p, const typename GfExtra<KIND>::type& extra,
+                          cudaStream_t stream) {
     const long long ctas = (long long)((p.n_out + TC_BM - 1) / TC_BM) * ((p.T + BN - 1) / BN) * p.splits;
-    if (p.mode == GF_ROPE) {
-        if (BN <= 32 && ctas <= sm_count() && p.kb_per_split > 4) return gf_launch_stages<BN, 8, true>(mw, mx, p, rope, stream);
-        return gf_launch_stages<BN, 4, true>(mw, mx, p, rope, stream);
-    }
-    if (BN <= 32 && ctas <= sm_count() && p.kb_per_split > 4) return gf_launch_stages<BN, 8, false>(mw, mx, p, rope, stream);
-    return gf_launch_stages<BN, 4, false>(mw, mx, p, rope, stream);
+    if (BN <= 32 && ctas <= sm_count() && p.kb_per_split > 4) return gf_launch_stages<BN, 8, KIND>(mw, mx, p, extra, stream);
+    return gf_launch_stages<BN, 4, KIND>(mw, mx, p, extra, stream);
+}
+template <int BN>
+static int gf_launch(const CUtensorMap& mw, const CUtensorMap& mx, const FusedParams& p, const RopeParams& rope, float limit,
+                     cudaStream_t stream) {
+    if (p.mode == GF_ROPE) return gf_launch_kind<BN, GF_KIND_ROPE>(mw, mx, p, rope, stream);
+    if (p.mode == GF_SWIGLU && limit > 0.0f) return gf_launch_kind<BN, GF_KIND_CLAMPED>(mw, mx, p, LimitParams{limit}, stream);
+    return gf_launch_kind<BN, GF_KIND_BASE>(mw, mx, p, NoRope(), stream);
 }
 
 }  // namespace bg
@@ -546,7 +557,7 @@ struct RopeArgs {
 static int gemm_fused_run(const void* W, int n_out, int K, int ldw, const void* X, int ldx, const float* xf, int ldxf,
                           const float* ssq_in, int n_ssq_in, int ssq_in_stride, const void* norm_w, float eps, int T,
                           const float* bias, int mode, void* out, int out_dtype, int ldo, float* ssq_out,
-                          int ssq_out_stride, int splits, const RopeArgs* rope, unsigned* status, cudaStream_t stream) {
+                          int ssq_out_stride, int splits, const RopeArgs* rope, float limit, unsigned* status, cudaStream_t stream) {
     if (T <= 0 || n_out <= 0) return BG_OK;
     if (K <= 0 || T > 64) return BG_ERR_SHAPE;
     if (splits != 1 && splits != 2 && splits != 4 && splits != 8 && splits != 16) return BG_ERR_SHAPE;
@@ -602,21 +613,22 @@ static int gemm_fused_run(const void* W, int n_out, int K, int ldw, const void* 
         memset(&mx, 0, sizeof(mx));
     }
     switch (bn) {
-        case 16: return gf_launch<16>(mw, mx, p, &rp, stream);
-        case 32: return gf_launch<32>(mw, mx, p, &rp, stream);
-        default: return gf_launch<64>(mw, mx, p, &rp, stream);
+        case 16: return gf_launch<16>(mw, mx, p, rp, limit, stream);
+        case 32: return gf_launch<32>(mw, mx, p, rp, limit, stream);
+        default: return gf_launch<64>(mw, mx, p, rp, limit, stream);
     }
 }
 
 // See the head of the file.  X (bfloat16 [T, K], row stride ldx) or xf (float [T, K], row stride ldxf, with
-// ssq_in, norm_w and eps) is the left operand; splits is 1, 2, 4, 8 or 16.
+// ssq_in, norm_w and eps) is the left operand; splits is 1, 2, 4, 8 or 16.  `limit` > 0 in the gated mode: the clamped form,
+// g sigmoid(1.702 g) (u + 1) with both branches cut off at the limit, in silu's place.
 extern "C" int bg_gemm_fused(const void* W, int n_out, int K, int ldw, const void* X, int ldx, const float* xf, int ldxf,
                              const float* ssq_in, int n_ssq_in, int ssq_in_stride, const void* norm_w, float eps, int T,
                              const float* bias, int mode, void* out, int out_dtype, int ldo, float* ssq_out,
-                             int ssq_out_stride, int splits, unsigned* status, cudaStream_t stream) {
-    if (mode == GF_ROPE) return BG_ERR_SHAPE;
+                             int ssq_out_stride, int splits, float limit, unsigned* status, cudaStream_t stream) {
+    if (mode == GF_ROPE || limit < 0.0f || (limit > 0.0f && mode != GF_SWIGLU)) return BG_ERR_SHAPE;
     return gemm_fused_run(W, n_out, K, ldw, X, ldx, xf, ldxf, ssq_in, n_ssq_in, ssq_in_stride, norm_w, eps, T, bias, mode,
-                          out, out_dtype, ldo, ssq_out, ssq_out_stride, splits, nullptr, status, stream);
+                          out, out_dtype, ldo, ssq_out, ssq_out_stride, splits, nullptr, limit, status, stream);
 }
 
 // The q/k/v product of a step of few tokens with rotation and cache append behind it: W [(nh + 2 nkv) hd, K], the
@@ -633,5 +645,5 @@ extern "C" int bg_gemm_fused_rope(const void* W, int K, int ldw, const void* X, 
     r.max_pages = max_pages; r.num_pages = num_pages; r.page_size = page_size; r.nh = nh; r.nkv = nkv; r.hd = hd;
     if (nh < 1 || nkv < 1 || hd < 1) return BG_ERR_SHAPE;
     return gemm_fused_run(W, (nh + 2 * nkv) * hd, K, ldw, X, ldx, xf, ldxf, ssq_in, n_ssq_in, ssq_in_stride, norm_w, eps, T,
-                          bias, GF_ROPE, q_out, BG_DTYPE_BF16, q_stride, nullptr, 0, splits, &r, status, stream);
+                          bias, GF_ROPE, q_out, BG_DTYPE_BF16, q_stride, nullptr, 0, splits, &r, 0.0f, status, stream);
 }

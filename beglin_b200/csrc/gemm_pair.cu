@@ -37,7 +37,8 @@ constexpr int GP_MODE_SWIGLU = 1;          // out[t, j] = silu(gate) * up, the w
 constexpr int GP_MODE_RESIDUAL = 2;        // out (float, the residual stream) [t, n] += product (+ bias[n])
 constexpr int GP_MODE_GEGLU = 3;           // as GP_MODE_SWIGLU with the tanh form of GELU in silu's place
 // (a template instance of its own: the other modes' code is compiled as if it did not exist)
-__host__ __device__ constexpr bool gp_glu(int mode) { return mode == GP_MODE_SWIGLU || mode == GP_MODE_GEGLU; }
+constexpr int GP_MODE_GLU_CLAMPED = 4;     // the same with g sigmoid(1.702 g) (u + 1), both branches cut off at a limit
+__host__ __device__ constexpr bool gp_glu(int mode) { return mode == GP_MODE_SWIGLU || mode == GP_MODE_GEGLU || mode == GP_MODE_GLU_CLAMPED; }
 // A tile is 256 tokens x BN output features, BN = 256, 192 or 128: a CTA loads BN / 2 rows of the weight.  The widest
 // tile that keeps the pairs of the device busy is chosen on the host: a narrow matrix has too few tiles of 256.
 template <int BN> struct GpTile {
@@ -52,6 +53,11 @@ struct PairParams {
     int tiles_m, tiles_n;   // tiles of 256 tokens and of BN features
     unsigned* status;
 };
+
+// (the limit of the clamped form: a parameter that the instances of the other modes do not carry)
+struct PairLimitParams : PairParams { float limit; };
+template <int MODE> struct GpParams { using type = PairParams; };
+template <> struct GpParams<GP_MODE_GLU_CLAMPED> { using type = PairLimitParams; };
 
 __device__ __forceinline__ unsigned cluster_rank() {
     unsigned r;
@@ -89,7 +95,7 @@ __device__ __forceinline__ void stage_store16(unsigned char* buf, int row, int c
 template <int STAGES, int MODE, int BN>
 __global__ void __launch_bounds__(GP_THREADS)
 gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constant__ CUtensorMap map_w,
-                 const __grid_constant__ CUtensorMap map_out, PairParams p) {
+                 const __grid_constant__ CUtensorMap map_out, typename GpParams<MODE>::type p) {
     extern __shared__ unsigned char gp_smem_raw[];
     constexpr unsigned GP_STAGE_BYTES = GpTile<BN>::STAGE_BYTES;
     constexpr int GP_HALF_N = BN / 2;
@@ -245,7 +251,9 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
 #pragma unroll
                         for (int j = 0; j < 32; ++j) {
                             const float gv = __uint_as_float(g[j]), uv = __uint_as_float(u[j]);
-                            if (MODE == GP_MODE_GEGLU)       // 0.5 g (1 + tanh(z)) = g sigmoid(2 z), z = sqrt(2/pi) (g + 0.044715 g^3)
+                            if constexpr (MODE == GP_MODE_GLU_CLAMPED)
+                                o[j] = glu_clamped_value<true>(gv, uv, p.limit);
+                            else if (MODE == GP_MODE_GEGLU)  // 0.5 g (1 + tanh(z)) = g sigmoid(2 z), z = sqrt(2/pi) (g + 0.044715 g^3)
                                 o[j] = __fdividef(gv, 1.0f + __expf(-1.5957691216057308f * (gv + 0.044715f * gv * gv * gv))) * uv;
                             else
                                 o[j] = __fdividef(gv, 1.0f + __expf(-gv)) * uv;
@@ -293,7 +301,7 @@ gemm_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_constan
 }
 
 template <int STAGES, int MODE, int BN>
-static int gp_launch(const CUtensorMap& mx, const CUtensorMap& mw, const CUtensorMap& mo, const PairParams& p, cudaStream_t stream) {
+static int gp_launch(const CUtensorMap& mx, const CUtensorMap& mw, const CUtensorMap& mo, const typename GpParams<MODE>::type& p, cudaStream_t stream) {
     auto kern = gemm_pair_kernel<STAGES, MODE, BN>;
     const size_t smem = (size_t)STAGES * GpTile<BN>::STAGE_BYTES + 2 * GP_OUT_BYTES + 1024;
     static bool set = false;
@@ -356,19 +364,22 @@ using namespace bg;
 //   mode 0: out[t, n] = sum_k X[t, k] W[n, k] (+ bias[n]) as bfloat16 [T, ldo];
 //   mode 1: the rows of W are gate and up features interleaved in blocks of 64 (n_out = 2 * inner, a multiple of
 //           128): out[t, j] = silu(gate_j) * up_j as bfloat16 [T, ldo] with n_out / 2 columns; no bias;
+//   mode 3, mode 4: as mode 1 with another activation (the tanh form of GELU; the clamped form, cut off at `limit`);
 //   mode 2: out is the float residual stream [T, ldo]: out[t, n] += sum_k X[t, k] W[n, k] (+ bias[n]).
 //   W: [n_out, K] bfloat16, row stride ldw; X: [T, K] bfloat16, row stride ldx; strides multiples of 8 elements
 //   (ldo of mode 2: of 4), bases 16-byte aligned.
 extern "C" int bg_gemm_pair(const void* W, int n_out, int K, int ldw, const void* X, int T, int ldx, const float* bias,
-                            void* out, int ldo, int mode, unsigned* status, cudaStream_t stream) {
+                            void* out, int ldo, int mode, float limit, unsigned* status, cudaStream_t stream) {
     if (T <= 0 || n_out <= 0) return BG_OK;
     if (K <= 0) return BG_ERR_SHAPE;
-    if (mode != GP_MODE_PLAIN && mode != GP_MODE_SWIGLU && mode != GP_MODE_RESIDUAL && mode != GP_MODE_GEGLU) return BG_ERR_UNSUPPORTED;
+    if (mode != GP_MODE_PLAIN && mode != GP_MODE_SWIGLU && mode != GP_MODE_RESIDUAL && mode != GP_MODE_GEGLU && mode != GP_MODE_GLU_CLAMPED) return BG_ERR_UNSUPPORTED;
+    if (mode == GP_MODE_GLU_CLAMPED && !(limit > 0.0f)) return BG_ERR_SHAPE;
     if ((ldw % 8) || (ldx % 8) || ((uintptr_t)W % 16) || ((uintptr_t)X % 16) || ((uintptr_t)out % 16)) return BG_ERR_ALIGN;
     if (mode == GP_MODE_RESIDUAL ? (ldo % 4) : (ldo % 8)) return BG_ERR_ALIGN;
     if (gp_glu(mode) && (n_out % 128 || bias)) return BG_ERR_SHAPE;
     const int bn = gp_tile_width(T, n_out, mode);
-    PairParams p;
+    PairLimitParams p;
+    p.limit = limit;
     p.bias = bias; p.n_out = n_out; p.T = T; p.K = K; p.status = status;
     p.tiles_m = (T + 2 * GP_BM - 1) / (2 * GP_BM);
     p.tiles_n = (n_out + bn - 1) / bn;
@@ -384,6 +395,8 @@ extern "C" int bg_gemm_pair(const void* W, int n_out, int K, int ldw, const void
         return bn == 256 ? gp_launch<6, GP_MODE_SWIGLU, 256>(mx, mw, mo, p, stream) : gp_launch<8, GP_MODE_SWIGLU, 128>(mx, mw, mo, p, stream);
     if (mode == GP_MODE_GEGLU)
         return bn == 256 ? gp_launch<6, GP_MODE_GEGLU, 256>(mx, mw, mo, p, stream) : gp_launch<8, GP_MODE_GEGLU, 128>(mx, mw, mo, p, stream);
+    if (mode == GP_MODE_GLU_CLAMPED)
+        return bn == 256 ? gp_launch<6, GP_MODE_GLU_CLAMPED, 256>(mx, mw, mo, p, stream) : gp_launch<8, GP_MODE_GLU_CLAMPED, 128>(mx, mw, mo, p, stream);
     if (mode == GP_MODE_PLAIN)
         return bn == 256 ? gp_launch<6, GP_MODE_PLAIN, 256>(mx, mw, mo, p, stream)
              : bn == 192 ? gp_launch<6, GP_MODE_PLAIN, 192>(mx, mw, mo, p, stream) : gp_launch<8, GP_MODE_PLAIN, 128>(mx, mw, mo, p, stream);

@@ -273,7 +273,7 @@ latent_attention_partial_kernel(LatentParams p) {
 }
 
 // out[h][t][:] = sum_s o_s e^(m_s - m) / sum_s l_s e^(m_s - m) over the splits that hold a key the row sees, in split
-// order.  One block of 128 threads per (row, head): the splits' weights are worked out once, by the first warp, and
+// order; with `sink_w` the denominator also holds exp of the head's number sink_w[h], which counts once and has no value.  One block of 128 threads per (row, head): the splits' weights are worked out once, by the first warp, and
 // every thread then sums its features over the splits with all its loads independent of one another (a warp per
 // (row, head) that recomputed the weights for every 32 features took 32 us for 96 rows of 17 splits).
 constexpr int LAT_MERGE_THREADS = 128;
@@ -281,7 +281,8 @@ template <typename TO>
 __global__ void __launch_bounds__(LAT_MERGE_THREADS)
 latent_attention_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                               const int* __restrict__ positions, TO* __restrict__ out, long long out_head,
-                              int out_row, int T, int H, int rank, int max_splits, int split, int window) {
+                              int out_row, int T, int H, int rank, int max_splits, int split, int window,
+                              const float* __restrict__ sink_w) {
     extern __shared__ float f_s[];                 // [max_splits] weights e^(m_s - m) / l
     pdl_launch();
     pdl_wait();
@@ -295,7 +296,8 @@ latent_attention_merge_kernel(const float* __restrict__ part_o, const float* __r
         float m = -INFINITY;
         for (int s = s_lo + lane; s <= s_hi; s += 32) m = fmaxf(m, part_ml[(prow + s) * 2]);
         m = warp_max(m);
-        float l = 0.0f;
+        if (sink_w) m = fmaxf(m, sink_w[h]);
+        float l = sink_w ? expf(sink_w[h] - m) : 0.0f;
         for (int s = s_lo; s <= s_hi; ++s) l = fmaf(part_ml[(prow + s) * 2 + 1], expf(part_ml[(prow + s) * 2] - m), l);
         const float inv = 1.0f / l;
         for (int s = s_lo + lane; s <= s_hi; s += 32) f_s[s] = expf(part_ml[(prow + s) * 2] - m) * inv;
@@ -470,13 +472,13 @@ extern "C" int bg_latent_attention_partial(const void* q_lat, int ql_dtype, long
 
 extern "C" int bg_latent_attention_merge(const float* part_o, const float* part_ml, const int* positions, void* out,
                                          int out_dtype, long long out_head, int out_row, int T, int H, int rank,
-                                         int max_splits, int split, int window, cudaStream_t stream) {
+                                         int max_splits, int split, int window, const float* sink_w, cudaStream_t stream) {
     const long long blocks = (long long)T * H;
     if (blocks <= 0) return BG_OK;
     if (blocks > 0x7fffffffLL || max_splits > 8192) return BG_ERR_SHAPE;
     BG_DISPATCH_DTYPE(out_dtype, TO,
         launch(latent_attention_merge_kernel<TO>, dim3((unsigned)blocks), dim3(LAT_MERGE_THREADS), (size_t)max_splits * sizeof(float),
-               stream, part_o, part_ml, positions, (TO*)out, out_head, out_row, T, H, rank, max_splits, split, window));
+               stream, part_o, part_ml, positions, (TO*)out, out_head, out_row, T, H, rank, max_splits, split, window, sink_w));
     BG_LAUNCH_CHECK();
     return BG_OK;
 }

@@ -27,28 +27,32 @@ _SIGNATURES = {
     "bg_add_rmsnorm": [_c_void_p, _c_void_p, _c_int, _c_int, _c_ll, _c_void_p, _c_int, _c_float, _c_void_p, _c_int,
                        _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
     "bg_add_residual": [_c_void_p, _c_void_p, _c_int, _c_ll, _c_void_p],
-    "bg_swiglu": [_c_void_p, _c_int, _c_int, _c_ll, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p],
+    "bg_swiglu": [_c_void_p, _c_int, _c_int, _c_ll, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_void_p],
     "bg_activation": [_c_void_p, _c_int, _c_int, _c_ll, _c_void_p, _c_int, _c_ll, _c_int, _c_void_p],
     "bg_rope_table": [_c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_float, _c_void_p],
     "bg_rope_kv_append": [_c_void_p, _c_int, _c_int, _c_int, _c_ll, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p,
                           _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                           _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
-    "bg_attention_plan": [_c_int, _c_int, _c_int, ctypes.POINTER(_c_int), ctypes.POINTER(_c_int)],
+    "bg_attention_plan": [_c_int, _c_int, _c_int, _c_int, ctypes.POINTER(_c_int), ctypes.POINTER(_c_int)],
     "bg_attention_partial": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int,
                              _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int,
-                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_void_p, _c_void_p,
-                             _c_void_p],
+                             _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_int, _c_void_p, _c_int,
+                             _c_void_p, _c_void_p],
+    "bg_difference_merge": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+                            _c_int, _c_int, _c_float, _c_float, _c_float, _c_void_p],
     "bg_attention_merge": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int,
                            _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p],
     "bg_rmsnorm_add": [_c_void_p, _c_void_p, _c_int, _c_int, _c_ll, _c_void_p, _c_int, _c_float, _c_void_p, _c_int, _c_int,
                        _c_int, _c_void_p],
+    "bg_norm_step": [_c_void_p, _c_void_p, _c_int, _c_int, _c_ll, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_void_p, _c_int,
+                     _c_float, _c_void_p, _c_int, _c_int, _c_int, _c_void_p],
     "bg_rmsnorm_add_routed": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_float, _c_void_p,
                               _c_int, _c_int, _c_int, _c_void_p],
     "bg_cast_rows": [_c_void_p, _c_void_p, _c_int, _c_ll, _c_void_p],
     "bg_qk_norm_rope_append": [_c_void_p, _c_int, _c_int, _c_int, _c_ll, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p,
                                _c_float, _c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int,
-                               _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p,
-                               _c_void_p],
+                               _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
+                               _c_int, _c_void_p, _c_void_p],
     "bg_route_logits": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p],
     "bg_route_topk": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_float, _c_void_p, _c_void_p, _c_void_p,
                       _c_void_p],
@@ -95,6 +99,9 @@ _SIGNATURES = {
     "bg_attention_tc_plan": [_c_int, _c_int, _c_int, ctypes.POINTER(_c_int)],
     "bg_attention_tc": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int,
                         _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_void_p, _c_void_p],
+    "bg_attention_tc_difference": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int,
+                                   _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_float, _c_float, _c_float,
+                                   _c_void_p, _c_void_p],
     "bg_attention_tc_ext": [_c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int,
                             _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_float, _c_int, _c_int, _c_void_p, _c_float,
                             _c_int, _c_void_p, _c_void_p, _c_void_p],
@@ -105,10 +112,10 @@ _SIGNATURES = {
     "bg_gemm_bf16_tn": [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int,
                         _c_int, _c_int, _c_void_p, _c_void_p],
     "bg_gemm_pair": [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_void_p, _c_int, _c_int,
-                     _c_void_p, _c_void_p],
+                     _c_float, _c_void_p, _c_void_p],
     "bg_gemm_fused": [_c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int,
                       _c_void_p, _c_float, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_int,
-                      _c_void_p, _c_void_p],
+                      _c_float, _c_void_p, _c_void_p],
     "bg_gemm_fused_rope": [_c_void_p, _c_int, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_void_p, _c_int, _c_int,
                            _c_void_p, _c_float, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_void_p,
                            _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p,
@@ -120,7 +127,7 @@ _SIGNATURES = {
     "bg_rmsnorm_slice": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_float, _c_void_p, _c_int, _c_int,
                          _c_int, _c_void_p],
     "bg_gate_heads": [_c_void_p, _c_int, _c_ll, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_int, _c_int,
-                      _c_int, _c_void_p],
+                      _c_int, _c_int, _c_void_p],
     "bg_latent_attention_plan": [_c_int, _c_int, ctypes.POINTER(_c_int), ctypes.POINTER(_c_int)],
     "bg_latent_append": [_c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_void_p, _c_int, _c_float, _c_void_p,
                          _c_void_p, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_void_p,
@@ -130,7 +137,7 @@ _SIGNATURES = {
                                     _c_void_p, _c_void_p, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int, _c_int,
                                     _c_int, _c_int, _c_int, _c_float, _c_void_p, _c_void_p],
     "bg_latent_attention_merge": [_c_void_p, _c_void_p, _c_void_p, _c_void_p, _c_int, _c_ll, _c_int, _c_int, _c_int, _c_int,
-                                  _c_int, _c_int, _c_int, _c_void_p],
+                                  _c_int, _c_int, _c_int, _c_void_p, _c_void_p],
     "bg_latent_attention_mma_plan": [_c_int, _c_int, ctypes.POINTER(_c_int), ctypes.POINTER(_c_int)],
     "bg_latent_attention_mma_partial": [_c_void_p, _c_ll, _c_int, _c_void_p, _c_int, _c_int, _c_int, _c_void_p, _c_void_p, _c_int,
                                         _c_int, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int, _c_void_p, _c_void_p, _c_int,
@@ -424,13 +431,13 @@ def add_residual(x: torch.Tensor, delta: torch.Tensor) -> None:
         _check(lib().bg_add_residual(_p(x), _p(delta), _dt(delta), x.numel(), _stream()), "add_residual")
 
 
-GLU_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}
-ACTIVATIONS = dict(GLU_ACTIVATIONS, relu2=2)          # of a feed-forward without a gate branch
+GLU_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "glu_clamped": 3}
+ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "relu2": 2}          # of a feed-forward without a gate branch
 
 
-def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0, activation: str = "silu") -> None:
+def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0, activation: str = "silu", limit: float = 0.0) -> None:
     """out[t, i] = act(g[t, i]) * g[t, im + i], g = gate_up or the sum of its partial sums; act is silu or the tanh form
-    of GELU.  With `block` > 0 the columns of g are interleaved in blocks of that many: gate, up, gate, up, ..."""
+    of GELU; "glu_clamped": out = a sigmoid(1.702 a) (b + 1), a = min(g[t, i], limit), b = clamp(g[t, im + i], -limit, limit).  With `block` > 0 the columns of g are interleaved in blocks of that many: gate, up, gate, up, ..."""
     if activation not in GLU_ACTIVATIONS:
         raise KernelError(f"swiglu: unknown activation '{activation}' ({', '.join(GLU_ACTIVATIONS)})")
     _cuda(gate_up, out)
@@ -443,9 +450,11 @@ def swiglu(gate_up: torch.Tensor, out: torch.Tensor, block: int = 0, activation:
         raise KernelError("swiglu: tensors must be contiguous")
     if block < 0 or (block > 0 and im % block):
         raise KernelError(f"swiglu: blocks of {block} do not divide {im} features")
+    if activation == "glu_clamped" and not limit > 0.0:
+        raise KernelError("swiglu: the clamped form wants a positive limit")
     with phase("swiglu"):
         _check(lib().bg_swiglu(_p(gate_up), _dt(gate_up), parts, stride, _p(out), _dt(out), rows, im, block,
-                               GLU_ACTIVATIONS[activation], _stream()), "swiglu")
+                               GLU_ACTIVATIONS[activation], float(limit), _stream()), "swiglu")
 
 
 def activation(z: torch.Tensor, out: torch.Tensor, activation: str = "silu") -> None:
@@ -554,7 +563,7 @@ def attention_plan(group: int, hd: int, dtype: torch.dtype = torch.float32, deco
             raise KernelError(f"the tensor-core attention kernel does not take head_dim {hd} with {group} query "
                               "heads per kv head (head_dim 64 or 128; at most 64 heads per kv head)")
     bq, tile = _c_int(0), _c_int(0)
-    rc = L.bg_attention_plan(group, hd, vd, ctypes.byref(bq), ctypes.byref(tile))
+    rc = L.bg_attention_plan(group, hd, vd, 1, ctypes.byref(bq), ctypes.byref(tile))
     if rc != 0:
         raise KernelError(f"attention: head_dim {hd} (values of {vd}) with {group} query heads per kv head is not "
                           "supported (both sizes must be at most 256)")
@@ -694,7 +703,7 @@ def _attention(q: torch.Tensor, q_stride: int, kv_pool: torch.Tensor, block_tabl
         _check(L.bg_attention_partial(_p(q), _dt(q), q_stride, _p(kv_pool), _dt(kv_pool), num_pages, page_size,
                                       _p(block_table), block_table.shape[1], _p(positions), _p(qblk), n_qblk,
                                       _p(part_o), _p(part_ml), n_splits, n_splits, nh, nkv, hd, vd, window, split, tile,
-                                      bq, float(scale), float(softcap), int(keep), _p(slopes), _p(status), _stream()),
+                                      bq, float(scale), float(softcap), int(keep), _p(slopes), 1, _p(status), _stream()),
                "attention_partial")
     elif kernel in ("mma_keys", "mma_rows"):
         # (the kernels that write finished rows know the plain softmax only: with the enlarged denominator their rows
@@ -712,6 +721,88 @@ def _attention(q: torch.Tensor, q_stride: int, kv_pool: torch.Tensor, block_tabl
         raise KernelError(f"unknown attention kernel '{kernel}'")
     _check(L.bg_attention_merge(_p(part_o), _p(part_ml), _p(positions), _p(out), _dt(out), out.stride(0), n_rows, nh,
                                 vd, n_splits, split, window, 1 if sink else 0, _p(sink_weight), int(keep), _stream()), "attention_merge")
+
+
+# ------------------------------------------------------------------------------------------------
+# Differential attention: heads that are pairs of maps over the same values
+def difference_plan(group: int, kw: int, vw: int, dtype: torch.dtype, decode_only: bool, prefer: str = "auto",
+                    page_size: int = 64) -> Tuple[str, int, int]:
+    """(kernel, rows per query block, keys per tile) for `group` query heads per kv head, maps stored `kw` features wide and values
+    `vw`: "tc_rows" (portions on tcgen05, the difference inside the kernel), "mma_keys" (decoding on the tensor cores) or "generic"
+    (CUDA cores, every size)."""
+    L = lib()
+    bq, tile = _c_int(0), _c_int(0)
+    if dtype == torch.bfloat16 and prefer != "generic" and 2 * kw == vw:
+        if decode_only:
+            if L.bg_attention_mma_plan(2 * group, vw, 1, ctypes.byref(bq)) == 0:
+                return "mma_keys", bq.value, 64
+        elif prefer in TC_ROWS_FOR and L.bg_attention_tc_plan(group, vw, page_size, ctypes.byref(bq)) == 0:
+            return "tc_rows", bq.value, 64
+    if L.bg_attention_plan(2 * group, 2 * kw, vw, 2, ctypes.byref(bq), ctypes.byref(tile)) != 0:
+        raise KernelError(f"differential attention: maps of {kw} features (values of {vw}) with {group} query heads per kv head are not "
+                          "supported (both sizes must be at most 256)")
+    return "generic", bq.value, tile.value
+
+
+def difference_attention(*args, **kwargs) -> None:
+    """`_difference_attention` under the phase timer of its kernel class (the partial kernel and its merge together)."""
+    with phase("attn"):
+        _difference_attention(*args, **kwargs)
+
+
+def _difference_attention(q: torch.Tensor, kv_pool: torch.Tensor, block_table: torch.Tensor, positions: torch.Tensor,
+                          qblk: Optional[torch.Tensor], n_qblk: int, max_position: int, n_rows: int, nh: int, nkv: int, kw: int,
+                          vw: int, vd: int, window: int, split: int, tile: int, bq: int, scale: float, lam: float, out_scale: float,
+                          eps: float, out: torch.Tensor, status: Optional[torch.Tensor], kernel: str) -> None:
+    """Paged differential attention of a step's rows.  Per head the maps' results a1, a2 (softmax over the same positions, the
+    same values) give o = a1 - lam a2, and out[t, h] = o / sqrt(mean(o^2) + eps) * out_scale over the head's `vd` features;
+    out [T, nh * vd].  `kernel`, `bq` and `tile` come from `difference_plan`, the queries and pages from `qk_norm_rope_append`
+    with two maps (queries padded for "mma_keys", alone for the others)."""
+    _cuda(q, kv_pool, block_table, positions, qblk, out, status)
+    _i32(positions, "positions"); _i32(block_table, "block_table")
+    if qblk is not None:
+        _i32(qblk, "qblk")
+    elif kernel != "mma_keys" or n_qblk != n_rows:
+        raise KernelError("differential attention: only the decoding kernel runs without a list of query blocks (block i = row i)")
+    q_width = 2 * nh * kw * (2 if kernel == "mma_keys" else 1)
+    if q.dim() != 2 or q.stride(1) != 1 or q.shape[0] < n_rows or q.shape[1] != q_width:
+        raise KernelError(f"differential attention: q is {tuple(q.shape)}, expected rows of {q_width} features")
+    if not kv_pool.is_contiguous() or kv_pool[0].numel() % (nkv * (2 * kw + vw)):
+        raise KernelError(f"differential attention: pages of {tuple(kv_pool.shape)} for {nkv} kv heads of 2 x {kw} + {vw} features")
+    num_pages, page_size = kv_pool.shape[0], kv_pool[0].numel() // (nkv * (2 * kw + vw))
+    if out.stride(1) != 1 or tuple(out.shape) != (n_rows, nh * vd) or nh % nkv or not 0 < vd <= vw:
+        raise KernelError("differential attention: out is [T, nh * vd] with unit inner stride")
+    L = lib()
+    if kernel == "tc_rows":
+        if q.dtype != torch.bfloat16 or kv_pool.dtype != torch.bfloat16 or out.dtype != torch.bfloat16 or status is None:
+            raise KernelError("differential attention: the tcgen05 kernel takes bfloat16 queries, caches and outputs, and a status word")
+        _check(L.bg_attention_tc_difference(
+            _p(q), q.stride(0), _p(kv_pool), num_pages, page_size, _p(block_table), block_table.shape[1], _p(positions), _p(qblk),
+            n_qblk, _p(out), out.stride(0), nh, nkv, vw, vd, int(window), float(scale), float(lam), float(out_scale), float(eps),
+            _p(status), _stream()), "attention_tcgen05_difference")
+        return
+    if kernel == "mma_keys":
+        split, n_splits = 0, decode_splits(n_qblk * nkv, max_position + 1)
+    else:
+        n_splits = max_position // split + 1
+    part_o = torch.empty((n_rows * 2 * nh * n_splits, vw), dtype=torch.float32, device=q.device)
+    part_ml = torch.empty((n_rows * 2 * nh * n_splits, 2), dtype=torch.float32, device=q.device)
+    if kernel == "generic":
+        _check(L.bg_attention_partial(_p(q), _dt(q), q.stride(0), _p(kv_pool), _dt(kv_pool), num_pages, page_size, _p(block_table),
+                                      block_table.shape[1], _p(positions), _p(qblk), n_qblk, _p(part_o), _p(part_ml), n_splits,
+                                      n_splits, 2 * nh, nkv, 2 * kw, vw, int(window), split, tile, bq, float(scale), 0.0, 0, None, 2,
+                                      _p(status), _stream()), "attention_partial")
+    elif kernel == "mma_keys":
+        if q.dtype != torch.bfloat16 or kv_pool.dtype != torch.bfloat16:
+            raise KernelError("differential attention: the tensor-core kernel takes bfloat16 queries and caches")
+        _check(L.bg_attention_mma_partial(_p(q), q.stride(0), _p(kv_pool), num_pages, page_size, _p(block_table),
+                                          block_table.shape[1], _p(positions), _p(qblk), n_qblk, _p(part_o), _p(part_ml), n_splits,
+                                          n_splits, 2 * nh, nkv, vw, int(window), split, 1, float(scale), 0.0, None, 0, 0, None,
+                                          _p(status), _stream()), "attention_mma_partial")
+    else:
+        raise KernelError(f"unknown differential attention kernel '{kernel}'")
+    _check(L.bg_difference_merge(_p(part_o), _p(part_ml), _p(positions), _p(out), _dt(out), out.stride(0), n_rows, nh, vw, vd,
+                                 n_splits, split, int(window), float(lam), float(out_scale), float(eps), _stream()), "difference_merge")
 
 
 def gemm_f32_nt(a: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor], out: torch.Tensor,
@@ -769,19 +860,21 @@ def gemm_bf16_tn_unchecked(x: torch.Tensor, w_ptr: int, n_out: int, k: int, ldw:
 
 
 PAIR_PLAIN, PAIR_SWIGLU, PAIR_RESIDUAL, PAIR_GEGLU = 0, 1, 2, 3       # PAIR_GEGLU: as PAIR_SWIGLU with the tanh form of GELU
-PAIR_GLU = {"silu": PAIR_SWIGLU, "gelu_tanh": PAIR_GEGLU}
+PAIR_GLU_CLAMPED = 4                                                  # the clamped form, with a limit
+PAIR_GLU = {"silu": PAIR_SWIGLU, "gelu_tanh": PAIR_GEGLU, "glu_clamped": PAIR_GLU_CLAMPED}
 
 
 def gemm_pair(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int = PAIR_PLAIN,
-              bias: Optional[torch.Tensor] = None, status: Optional[torch.Tensor] = None) -> None:
+              bias: Optional[torch.Tensor] = None, status: Optional[torch.Tensor] = None, limit: float = 0.0) -> None:
     """The product of many rows (prompt portions) with w[N, K]^T by pairs of CTAs on the tcgen05 tensor cores.
     mode PAIR_PLAIN: out bfloat16 [T, N] = product (+ bias).  mode PAIR_SWIGLU: w's rows are interleaved (64 of
     gate, then their 64 of up); out bfloat16 [T, N / 2] = silu(gate) * up.  mode PAIR_RESIDUAL: out is the float32
-    residual stream [T, N]: out += product (+ bias)."""
+    residual stream [T, N]: out += product (+ bias).  PAIR_GEGLU and PAIR_GLU_CLAMPED are PAIR_SWIGLU with another activation
+    (`swiglu`'s; the clamped form wants `limit`)."""
     _cuda(x, w, out, bias, status)
     N, K = w.shape
     T = x.shape[0]
-    cols = N // 2 if mode in (PAIR_SWIGLU, PAIR_GEGLU) else N
+    cols = N // 2 if mode in PAIR_GLU.values() else N
     if x.dtype != torch.bfloat16 or w.dtype != torch.bfloat16 or \
             out.dtype != (torch.float32 if mode == PAIR_RESIDUAL else torch.bfloat16):
         raise KernelError("gemm_pair takes bfloat16 operands and gives a bfloat16 result (adds to a float32 stream)")
@@ -792,17 +885,17 @@ def gemm_pair(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: int = P
     if bias is not None and (bias.dtype != torch.float32 or bias.numel() != N or not bias.is_contiguous()):
         raise KernelError("gemm_pair: bias must be float32 with one value per output feature")
     _check(lib().bg_gemm_pair(_p(w), N, K, w.stride(0), _p(x), T, x.stride(0), _p(bias), _p(out), out.stride(0), mode,
-                              _p(status), _stream()), "gemm_pair")
+                              float(limit), _p(status), _stream()), "gemm_pair")
 
 
 def gemm_pair_unchecked(x: torch.Tensor, w_ptr: int, n_out: int, k: int, ldw: int, out: torch.Tensor, mode: int,
-                        status_ptr, bias_ptr=None) -> None:
+                        status_ptr, bias_ptr=None, limit: float = 0.0) -> None:
     """gemm_pair for a caller that has checked the weight once (Linear): x bfloat16 [T, k] with contiguous rows,
     out bfloat16 [T, n_out], with PAIR_SWIGLU [T, n_out / 2], with PAIR_RESIDUAL the float32 stream [T, n_out]."""
     if status_ptr is None:
         raise KernelError("gemm_pair wants a status word (its waits are bounded)")
     _check(_lib.bg_gemm_pair(w_ptr, n_out, k, ldw, x.data_ptr(), x.shape[0], x.stride(0), bias_ptr, out.data_ptr(),
-                             out.stride(0), mode, status_ptr, _stream()), "gemm_pair")
+                             out.stride(0), mode, limit, status_ptr, _stream()), "gemm_pair")
 
 
 FUSED_PLAIN, FUSED_RESIDUAL, FUSED_SWIGLU = 0, 1, 2
@@ -811,7 +904,8 @@ FUSED_PLAIN, FUSED_RESIDUAL, FUSED_SWIGLU = 0, 1, 2
 def gemm_fused(w: torch.Tensor, out: torch.Tensor, mode: int = FUSED_PLAIN, *, x: Optional[torch.Tensor] = None,
                xf: Optional[torch.Tensor] = None, ssq_in: Optional[torch.Tensor] = None,
                norm_weight: Optional[torch.Tensor] = None, eps: float = 0.0, bias: Optional[torch.Tensor] = None,
-               ssq_out: Optional[torch.Tensor] = None, splits: int = 1, status: Optional[torch.Tensor] = None) -> None:
+               ssq_out: Optional[torch.Tensor] = None, splits: int = 1, status: Optional[torch.Tensor] = None,
+               limit: float = 0.0) -> None:
     """The product of up to 64 rows with w[N, K]^T on the tcgen05 tensor cores, with its neighbours fused in.
 
     Left operand: `x` (bfloat16 [T, K]), or the float32 residual stream `xf` [T, K] normalised on the fly:
@@ -821,7 +915,7 @@ def gemm_fused(w: torch.Tensor, out: torch.Tensor, mode: int = FUSED_PLAIN, *, x
     mode FUSED_RESIDUAL: out (float32 [T, N], the residual stream) += product (+ bias); ssq_out
       [ceil(N / 128) * splits, >= T] receives partial sums of squares of the new rows.
     mode FUSED_SWIGLU: w's rows are interleaved (64 of gate, then their 64 of up); out bfloat16 [T, N / 2] =
-      silu(gate) * up."""
+      silu(gate) * up, or, with `limit` > 0, the clamped form of `swiglu`."""
     _cuda(w, out, x, xf, ssq_in, norm_weight, bias, ssq_out, status)
     N, K = w.shape
     if w.dtype != torch.bfloat16 or w.stride(1) != 1:
@@ -855,12 +949,12 @@ def gemm_fused(w: torch.Tensor, out: torch.Tensor, mode: int = FUSED_PLAIN, *, x
                                xf.stride(0) if xf is not None else 0, _p(ssq_in),
                                ssq_in.shape[0] if ssq_in is not None else 0, ssq_in.stride(0) if ssq_in is not None else 0,
                                _p(norm_weight), float(eps), T, _p(bias), mode, _p(out), _dt(out), out.stride(0),
-                               _p(ssq_out), ssq_out.stride(0) if ssq_out is not None else 0, splits, _p(status),
+                               _p(ssq_out), ssq_out.stride(0) if ssq_out is not None else 0, splits, float(limit), _p(status),
                                _stream()), "gemm_fused")
 
 
 def gemm_fused_unchecked(w_ptr: int, n_out: int, k: int, ldw: int, T: int, out: torch.Tensor, mode: int, x, xf, ssq_in,
-                         norm_w_ptr, eps: float, bias_ptr, ssq_out, splits: int, status_ptr) -> None:
+                         norm_w_ptr, eps: float, bias_ptr, ssq_out, splits: int, status_ptr, limit: float = 0.0) -> None:
     """gemm_fused for a caller that has checked the shapes once (Linear)."""
     _check(_lib.bg_gemm_fused(w_ptr, n_out, k, ldw, None if x is None else x.data_ptr(), 0 if x is None else x.stride(0),
                               None if xf is None else xf.data_ptr(), 0 if xf is None else xf.stride(0),
@@ -868,7 +962,7 @@ def gemm_fused_unchecked(w_ptr: int, n_out: int, k: int, ldw: int, T: int, out: 
                               0 if ssq_in is None else ssq_in.stride(0), norm_w_ptr, eps, T, bias_ptr, mode, out.data_ptr(),
                               F32 if out.dtype == torch.float32 else BF16, out.stride(0),
                               None if ssq_out is None else ssq_out.data_ptr(), 0 if ssq_out is None else ssq_out.stride(0),
-                              splits, status_ptr, _stream()), "gemm_fused")
+                              splits, limit, status_ptr, _stream()), "gemm_fused")
 
 
 def gemm_fused_rope(w: torch.Tensor, x: Optional[torch.Tensor], bias: Optional[torch.Tensor], q_out: torch.Tensor,
@@ -1035,18 +1129,20 @@ def rmsnorm_slice(src: torch.Tensor, col0: int, n: int, weight: torch.Tensor, ep
                                       _dt(out), out.stride(0), src.shape[0], _stream()), "rmsnorm_slice")
 
 
-def gate_heads(src: torch.Tensor, gate: Optional[torch.Tensor], gate_col0: int, out: torch.Tensor) -> None:
+def gate_heads(src: torch.Tensor, gate: Optional[torch.Tensor], gate_col0: int, out: torch.Tensor, per_feature: bool = False) -> None:
     """out[t, h * vd + j] = src[h, t, j] * sigmoid(gate[t, gate_col0 + h]); src is [H, T, vd].  Without `gate` the heads
-    are put row by row as they are."""
+    are put row by row as they are; `per_feature`: every feature has a gate, gate[t, gate_col0 + h * vd + j]."""
     _cuda(src, gate, out)
     H, T, vd = src.shape
-    if src.stride(2) != 1 or (gate is not None and (gate.stride(1) != 1 or gate_col0 + H > gate.shape[1] or gate.shape[0] < T)):
-        raise KernelError("gate_heads: src [H, T, vd] with unit inner stride, gate rows that hold H values from gate_col0")
+    n_gates = H * vd if per_feature else H
+    if src.stride(2) != 1 or (gate is not None and (gate.stride(1) != 1 or gate_col0 + n_gates > gate.shape[1] or gate.shape[0] < T)):
+        raise KernelError("gate_heads: src [H, T, vd] with unit inner stride, gate rows that hold the gates from gate_col0")
     if tuple(out.shape) != (T, H * vd) or not out.is_contiguous():
         raise KernelError(f"gate_heads: out is {tuple(out.shape)}, expected {(T, H * vd)}")
     with phase("activation"):
         _check(lib().bg_gate_heads(_p(src), _dt(src), src.stride(0), src.stride(1), _p(gate), _dt(gate) if gate is not None else F32,
-                                   gate.stride(0) if gate is not None else 0, gate_col0, _p(out), _dt(out), T, H, vd, _stream()),
+                                   gate.stride(0) if gate is not None else 0, gate_col0, _p(out), _dt(out), T, H, vd,
+                                   1 if per_feature else 0, _stream()),
                "gate_heads")
 
 
@@ -1125,14 +1221,17 @@ def latent_attention(q_lat: torch.Tensor, q_raw: torch.Tensor, dim: int, rot: in
                      cos_sin: Optional[torch.Tensor], pool: torch.Tensor, block_table: torch.Tensor,
                      positions: torch.Tensor, qblk: torch.Tensor, n_qblk: int, max_position: int, bq: int, hc: int,
                      tile: int, split: int, scale: float, out: torch.Tensor, status: Optional[torch.Tensor],
-                     mma_stages: int = 0, window: int = 0) -> None:
+                     mma_stages: int = 0, window: int = 0, sink_weight: Optional[torch.Tensor] = None) -> None:
     """Causal attention of a step's rows over the latent cache.  q_lat float32 [H, T, rank]: the queries carried into
     the latent space; q_raw [T, H * (dim + rot)]: the query product's rows, whose rot part is rotated here; pool
     [pages, page_size, rank + rot]; out [H, T, rank] receives, per head, the softmax-weighted sum of the cached
     latents.  `qblk` is cut for `bq` rows; a CTA takes `hc` heads; keys are cut into splits of `split` positions.
     With `mma_stages` 1 or 2 the products run on the tensor cores (bfloat16 q_raw and pool, bq * hc at most 64, sizes as
     `latent_attention_mma_plan` says); else on the CUDA cores in float, for every size and type.  `window` w > 0: a row
-    sees itself and the w - 1 positions before it."""
+    sees itself and the w - 1 positions before it.  `sink_weight` (float32 [H]): the softmax's denominator also holds exp of the
+    head's number."""
+    if sink_weight is not None and (sink_weight.dtype != torch.float32 or sink_weight.numel() != q_lat.shape[0] or not sink_weight.is_contiguous()):
+        raise KernelError("latent_attention: the sink's scores are contiguous float32, one per head")
     _cuda(q_lat, q_raw, cos_sin, pool, block_table, positions, qblk, out, status)
     _i32(positions, "positions"); _i32(block_table, "block_table"); _i32(qblk, "qblk")
     H, T, rank = q_lat.shape
@@ -1166,7 +1265,7 @@ def latent_attention(q_lat: torch.Tensor, q_raw: torch.Tensor, dim: int, rot: in
                                                  n_qblk, _p(part_o), _p(part_ml), n_splits, n_splits, H, hc, rank, rot, rot_dims,
                                                  split, tile, bq, int(window), float(scale), _p(status), _stream()), "latent_attention_partial")
         _check(L.bg_latent_attention_merge(_p(part_o), _p(part_ml), _p(positions), _p(out), _dt(out), out.stride(0),
-                                           out.stride(1), T, H, rank, n_splits, split, int(window), _stream()), "latent_attention_merge")
+                                           out.stride(1), T, H, rank, n_splits, split, int(window), _p(sink_weight), _stream()), "latent_attention_merge")
 
 
 def latent_gather(pool: torch.Tensor, block_table: torch.Tensor, req: int, rank: int, lat: torch.Tensor, kr: torch.Tensor,
@@ -1337,6 +1436,40 @@ def rmsnorm_add(x: torch.Tensor, y: torch.Tensor, weight: torch.Tensor, eps: flo
                                     _dt(lowp) if lowp is not None else F32, T, d, _stream()), "rmsnorm_add")
 
 
+def norm_step(x: torch.Tensor, y: Optional[torch.Tensor] = None, y_weight: Optional[torch.Tensor] = None, y_eps: float = 0.0,
+              rows: Optional[torch.Tensor] = None, vector: Optional[torch.Tensor] = None, weight: Optional[torch.Tensor] = None,
+              eps: float = 0.0, out: Optional[torch.Tensor] = None) -> None:
+    """What stands between two sublayers that have a norm in front and a norm behind, in one pass over the rows:
+    x += rmsnorm(y) * y_weight (y [T, d], or its float partial sums [parts, T, d]), x += rows (float32 [T, d]), x += vector
+    (float32 [d], the same for every row), each where given, then out = rmsnorm(x) * weight where asked for.  The weights have one
+    type.  Statistics and sums in float."""
+    _cuda(x, y, y_weight, rows, vector, weight, out)
+    T, d = x.shape
+    if x.dtype != torch.float32 or not x.is_contiguous():
+        raise KernelError("norm_step: x is contiguous float32 [T, d]")
+    parts, stride = 1, 0
+    if y is not None:
+        parts, stride = _parts(y, "norm_step: y")
+        if tuple(y.shape[-2:]) != (T, d) or not y.is_contiguous() or y_weight is None or (parts > 1 and y.dtype != torch.float32):
+            raise KernelError("norm_step: y is contiguous and shaped like x (or its float partial sums), with a weight")
+    for w in (y_weight, weight):
+        if w is not None and (w.numel() != d or not w.is_contiguous()):
+            raise KernelError(f"norm_step: a weight of {w.numel()} for rows of {d}")
+    if y_weight is not None and weight is not None and y_weight.dtype != weight.dtype:
+        raise KernelError("norm_step: the two weights are of one type")
+    if rows is not None and (rows.dtype != torch.float32 or rows.shape != x.shape or not rows.is_contiguous()):
+        raise KernelError("norm_step: rows to add are contiguous float32 and shaped like x")
+    if vector is not None and (vector.dtype != torch.float32 or vector.numel() != d or not vector.is_contiguous()):
+        raise KernelError("norm_step: a vector to add is contiguous float32 [d]")
+    if (out is None) != (weight is None) or (out is not None and (tuple(out.shape) != (T, d) or not out.is_contiguous())):
+        raise KernelError("norm_step: the normed rows are contiguous [T, d] and have a weight")
+    w_any = y_weight if y_weight is not None else weight
+    with phase("rmsnorm" if out is not None else "residuals"):
+        _check(lib().bg_norm_step(_p(x), _p(y), _dt(y) if y is not None else F32, parts, stride, _p(y_weight), float(y_eps), _p(rows),
+                                  _p(vector), _p(weight), _dt(w_any) if w_any is not None else F32, float(eps), _p(out),
+                                  _dt(out) if out is not None else F32, T, d, _stream()), "norm_step")
+
+
 def rmsnorm_add_routed(x: torch.Tensor, yp: torch.Tensor, row_of: torch.Tensor, weights: torch.Tensor, top: int, scale: bool,
                        weight: torch.Tensor, eps: float, lowp: Optional[torch.Tensor] = None) -> None:
     """`route_combine` and `rmsnorm_add` as one kernel: x += rmsnorm(y) * weight with y[t] the sum over j < top of
@@ -1370,22 +1503,29 @@ def qk_norm_rope_append(src: torch.Tensor, q_out: torch.Tensor, n_rows: int, nh:
                         interleaved: bool, q_weight: Optional[torch.Tensor], k_weight: Optional[torch.Tensor], eps: float,
                         cos_sin: Optional[torch.Tensor], positions: torch.Tensor, row_req: torch.Tensor,
                         block_table: torch.Tensor, kv_pool: Optional[torch.Tensor], page_size: int,
-                        status: Optional[torch.Tensor], stored: Optional[int] = None, per_head: bool = False) -> None:
+                        status: Optional[torch.Tensor], stored=None, per_head: bool = False, maps: int = 1,
+                        padded: bool = False) -> None:
     """Rows [q | k | v | ...] of `src` ([T, W], or float partial sums [parts, T, W]): RMS norm of the whole q row and of
     the whole k row with the float weights given (None: no norm; with `per_head` every head is normed by itself and the
     weights have hd values, shared by the heads), rotation of the first `rot` features of every head,
     q into q_out [T, nh*hd], k and v into the paged cache (a page: keys [nkv, page, hd], then values [nkv, page, vd]).
-    With `stored` = D every head of q, k and v is stored D features wide, zeros behind its own."""
-    qs, ks, vs = (hd, hd, vd) if stored is None else (stored, stored, stored)
+    With `stored` = D every head of q, k and v is stored D features wide, zeros behind its own; a pair gives the width of keys
+    and that of values.
+
+    `maps` 2: a head is a pair of maps over one value.  `nh` counts the query maps (two per query head), a kv head has two keys
+    of `hd` features and one value, a page's key row holds both keys side by side, and `stored[0]` is the width of one map.  A
+    query map is stored alone, or, `padded`, at its own keys' place in a row as wide as a key row, zeros beside it."""
+    kw, vs = (hd, vd) if stored is None else ((stored, stored) if isinstance(stored, int) else stored)
+    ks, qs, q_shift = maps * kw, (maps * kw if padded else kw), (kw if padded else 0)
     _cuda(src, q_out, q_weight, k_weight, cos_sin, positions, row_req, block_table, kv_pool)
     _i32(positions, "positions"); _i32(row_req, "row_req"); _i32(block_table, "block_table")
     parts, stride = _parts(src, "qk_norm_rope_append: src")
-    need = nh * hd + (nkv * (hd + vd) if kv_pool is not None else 0)
+    need = nh * hd + (nkv * (maps * hd + vd) if kv_pool is not None else 0)
     if src.stride(-1) != 1 or src.shape[-1] < need or src.shape[-2] < n_rows:
         raise KernelError(f"qk_norm_rope_append: rows of {src.shape[-1]} features cannot hold q, k, v ({need})")
     if q_out.stride(1) != 1 or q_out.shape[1] < nh * qs or q_out.shape[0] < n_rows:
         raise KernelError("qk_norm_rope_append: q_out must be [T, nh*hd]")
-    for w, n in ((q_weight, hd if per_head else nh * hd), (k_weight, hd if per_head else nkv * hd)):
+    for w, n in ((q_weight, hd if per_head else nh * hd), (k_weight, hd if per_head else nkv * maps * hd)):
         if w is not None and (w.dtype != torch.float32 or w.numel() != n or not w.is_contiguous()):
             raise KernelError("qk_norm_rope_append: norm weights are contiguous float32 of the projection's width")
     num_pages = 0
@@ -1400,7 +1540,8 @@ def qk_norm_rope_append(src: torch.Tensor, q_out: torch.Tensor, n_rows: int, nh:
                                             _p(q_weight), _p(k_weight), float(eps), _p(cos_sin), _p(positions), _p(row_req),
                                             _p(block_table), block_table.shape[1], _p(kv_pool),
                                             _dt(kv_pool) if kv_pool is not None else _dt(q_out), num_pages, page_size, n_rows, nh,
-                                            nkv, hd, vd, rot, 1 if interleaved else 0, qs, ks, vs, 1 if per_head else 0, _p(status), _stream()),
+                                            nkv, hd, vd, rot, 1 if interleaved else 0, qs, ks, vs, 1 if per_head else 0, maps, q_shift,
+                                            _p(status), _stream()),
                "qk_norm_rope_append")
 
 

@@ -178,6 +178,140 @@ __global__ void cast_rows_kernel(const float* __restrict__ x, TO* __restrict__ o
     if (i < n) out[i] = from_float<TO>(x[i]);
 }
 
+// What stands between two sublayers of a layer with a norm in front of each and another on its result, in one pass:
+//   x[t] += rmsnorm(y[t]) * wy    (y: the sublayer's product, or its split-K partial sums)
+//   x[t] += rows[t] + vec         (where a pass of a repeated run of layers begins: the embedded rows, a learned row)
+//   out[t] = rmsnorm(x[t]) * w    (what the next sublayer reads)
+// each where its pointer is given.  A row's sums are added up in an order fixed by the width alone.
+struct NormStepParams {
+    float* x;
+    const void* y; int parts; size_t part_stride;
+    const void* wy; float y_eps;
+    const float* rows; const float* vec;
+    const void* w; float eps;
+    void* out;
+    int n_rows, d;
+};
+
+template <typename TY, typename TW, typename TO>
+__global__ void __launch_bounds__(256) norm_step_kernel(NormStepParams p) {
+    extern __shared__ float row_buf[];
+    __shared__ float red[32];
+    pdl_launch();
+    pdl_wait();
+    const size_t base = (size_t)blockIdx.x * p.d;
+    float inv = 0.0f;
+    if (p.y) {
+        float ss = 0.0f;
+        for (int i = threadIdx.x; i < p.d; i += blockDim.x) {
+            const float v = sum_parts((const TY*)p.y + base + i, p.parts, p.part_stride);
+            row_buf[i] = v;
+            ss += v * v;
+        }
+        ss = block_sum(ss, red);
+        inv = 1.0f / sqrtf(ss / (float)p.d + p.y_eps);
+    }
+    float ss = 0.0f;
+    for (int i = threadIdx.x; i < p.d; i += blockDim.x) {
+        float v = p.x[base + i];
+        if (p.y) v += row_buf[i] * inv * to_float(((const TW*)p.wy)[i]);
+        if (p.rows) v += p.rows[base + i];
+        if (p.vec) v += p.vec[i];
+        p.x[base + i] = v;
+        row_buf[i] = v;
+        ss += v * v;
+    }
+    if (!p.out) return;
+    ss = block_sum(ss, red);
+    inv = 1.0f / sqrtf(ss / (float)p.d + p.eps);
+    for (int i = threadIdx.x; i < p.d; i += blockDim.x)
+        ((TO*)p.out)[base + i] = from_float<TO>(row_buf[i] * inv * to_float(((const TW*)p.w)[i]));
+}
+
+__device__ __forceinline__ float4 step_load4(const float* p) { return *reinterpret_cast<const float4*>(p); }
+__device__ __forceinline__ float4 step_load4(const __nv_bfloat16* p) {
+    const uint2 raw = *reinterpret_cast<const uint2*>(p);
+    const float2 lo = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.x));
+    const float2 hi = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&raw.y));
+    return make_float4(lo.x, lo.y, hi.x, hi.y);
+}
+__device__ __forceinline__ void step_store4(float* p, float4 v) { *reinterpret_cast<float4*>(p) = v; }
+__device__ __forceinline__ void step_store4(__nv_bfloat16* p, float4 v) {
+    uint2 raw;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
+    h[0] = __floats2bfloat162_rn(v.x, v.y);
+    h[1] = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(p) = raw;
+}
+
+// Four columns a thread (d a multiple of 4, everything 16-byte aligned), the row in registers: ITER groups of four a thread.
+template <typename TY, typename TW, typename TO, int ITER>
+__global__ void __launch_bounds__(1024) norm_step_vec4_kernel(NormStepParams p) {
+    __shared__ float red[32];
+    pdl_launch();
+    const int d4 = p.d >> 2;
+    const size_t base = (size_t)blockIdx.x * p.d;
+    pdl_wait();
+    float4 xv[ITER];
+    float inv = 0.0f;
+    {
+        float4 yv[ITER];
+        float ss = 0.0f;
+#pragma unroll
+        for (int it = 0; it < ITER; ++it) {                      // the residual and the addend are asked for together
+            const int c = threadIdx.x + it * blockDim.x;
+            if (c >= d4) continue;
+            xv[it] = step_load4(p.x + base + 4 * c);
+            if (p.y) {
+                if constexpr (std::is_same<TY, float>::value)
+                    yv[it] = sum_parts4(reinterpret_cast<const float4*>((const float*)p.y + base) + c, p.parts, p.part_stride / 4);
+                else yv[it] = step_load4((const TY*)p.y + base + 4 * c);
+                ss += yv[it].x * yv[it].x + yv[it].y * yv[it].y + yv[it].z * yv[it].z + yv[it].w * yv[it].w;
+            }
+        }
+        if (p.y) {
+            ss = block_sum(ss, red);
+            inv = 1.0f / sqrtf(ss / (float)p.d + p.y_eps);
+        }
+#pragma unroll
+        for (int it = 0; it < ITER; ++it) {
+            const int c = threadIdx.x + it * blockDim.x;
+            if (c >= d4) continue;
+            float4 v = xv[it];
+            if (p.y) {
+                const float4 w = step_load4((const TW*)p.wy + 4 * c);
+                v.x += yv[it].x * inv * w.x; v.y += yv[it].y * inv * w.y; v.z += yv[it].z * inv * w.z; v.w += yv[it].w * inv * w.w;
+            }
+            if (p.rows) {
+                const float4 a = step_load4(p.rows + base + 4 * c);
+                v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+            }
+            if (p.vec) {
+                const float4 a = step_load4(p.vec + 4 * c);
+                v.x += a.x; v.y += a.y; v.z += a.z; v.w += a.w;
+            }
+            xv[it] = v;
+            step_store4(p.x + base + 4 * c, v);
+        }
+    }
+    if (!p.out) return;
+    float ss = 0.0f;
+#pragma unroll
+    for (int it = 0; it < ITER; ++it) {
+        const int c = threadIdx.x + it * blockDim.x;
+        if (c < d4) ss += xv[it].x * xv[it].x + xv[it].y * xv[it].y + xv[it].z * xv[it].z + xv[it].w * xv[it].w;
+    }
+    ss = block_sum(ss, red);
+    inv = 1.0f / sqrtf(ss / (float)p.d + p.eps);
+#pragma unroll
+    for (int it = 0; it < ITER; ++it) {
+        const int c = threadIdx.x + it * blockDim.x;
+        if (c >= d4) continue;
+        const float4 w = step_load4((const TW*)p.w + 4 * c), v = xv[it];
+        step_store4((TO*)p.out + base + 4 * c, make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w));
+    }
+}
+
 }  // namespace bg
 
 using namespace bg;
@@ -259,5 +393,50 @@ extern "C" int bg_cast_rows(const float* x, void* out, int out_dtype, long long 
     const unsigned blocks = (unsigned)((n + 255) / 256);
     BG_DISPATCH_DTYPE(out_dtype, TO, launch(cast_rows_kernel<TO>, dim3(blocks), dim3(256), 0, stream, x, (TO*)out, n));
     BG_LAUNCH_CHECK();
+    return BG_OK;
+}
+
+template <typename TY, typename TW, typename TO>
+static int norm_step_launch(const NormStepParams& p, bool vec, cudaStream_t stream) {
+    const int d4 = p.d / 4;
+    if (vec && d4 <= 4096) {
+        // (the number of threads depends on the width alone: it decides the order in which a row is added up)
+        int threads = (d4 + 31) / 32 * 32;
+        if (threads > 1024) threads = 1024;
+        if (threads > 512 && (d4 + 1) / 2 <= 512) threads = ((d4 + 1) / 2 + 31) / 32 * 32;
+        const int iter = (d4 + threads - 1) / threads;
+        if (iter <= 1) launch(norm_step_vec4_kernel<TY, TW, TO, 1>, dim3(p.n_rows), dim3(threads), 0, stream, p);
+        else if (iter <= 2) launch(norm_step_vec4_kernel<TY, TW, TO, 2>, dim3(p.n_rows), dim3(threads), 0, stream, p);
+        else launch(norm_step_vec4_kernel<TY, TW, TO, 4>, dim3(p.n_rows), dim3(threads), 0, stream, p);
+        BG_LAUNCH_CHECK();
+        return BG_OK;
+    }
+    const size_t smem = (size_t)p.d * sizeof(float);
+    if (smem > 200 * 1024) return BG_ERR_SHAPE;
+    auto kern = norm_step_kernel<TY, TW, TO>;
+    if (smem > BG_SMEM_OPT_IN) {
+        cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
+        if (e != cudaSuccess) return (int)e;
+    }
+    launch(kern, dim3(p.n_rows), dim3(256), smem, stream, p);
+    BG_LAUNCH_CHECK();
+    return BG_OK;
+}
+
+// See NormStepParams.  y, rows, vec and out may be null; wy and w are of one type (w_dtype).
+extern "C" int bg_norm_step(float* x, const void* y, int y_dtype, int parts, long long part_stride, const void* wy, float y_eps,
+                            const float* rows, const float* vec, const void* w, int w_dtype, float eps, void* out, int out_dtype,
+                            int n_rows, int d, cudaStream_t stream) {
+    if (n_rows <= 0 || d <= 0) return BG_OK;
+    if (parts < 1 || (y && !wy) || (out && !w)) return BG_ERR_SHAPE;
+    NormStepParams p;
+    p.x = x; p.y = y; p.parts = parts; p.part_stride = (size_t)part_stride; p.wy = wy; p.y_eps = y_eps; p.rows = rows; p.vec = vec;
+    p.w = w; p.eps = eps; p.out = out; p.n_rows = n_rows; p.d = d;
+    if (!y) y_dtype = BG_DTYPE_F32;
+    if (!out) out_dtype = BG_DTYPE_F32;
+    const uintptr_t all = (uintptr_t)x | (uintptr_t)y | (uintptr_t)wy | (uintptr_t)rows | (uintptr_t)vec | (uintptr_t)w | (uintptr_t)out;
+    const bool vec4 = d % 4 == 0 && all % 16 == 0 && part_stride % 4 == 0 && (y_dtype == BG_DTYPE_F32 || parts == 1);
+    BG_DISPATCH_DTYPE(y_dtype, TY, BG_DISPATCH_DTYPE(w_dtype, TW, BG_DISPATCH_DTYPE(out_dtype, TO,
+        return (norm_step_launch<TY, TW, TO>(p, vec4, stream)))));
     return BG_OK;
 }

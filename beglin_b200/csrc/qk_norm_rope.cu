@@ -31,6 +31,20 @@ struct QkNormRopeParams {
     unsigned* status;
 };
 
+// A query head may be made of MAPS maps, each with a query of its own, and a kv head of as many keys (and ONE value): `nh`
+// counts maps, a page's key row holds the maps of a kv head side by side, and a query is stored alone or, where a kernel
+// multiplies whole key rows, at its map's place in a row of zeros.
+struct QkMapsParams : QkNormRopeParams {
+    int kw;                                                  // features of one map in a stored key row (ks = MAPS * kw)
+    int q_shift;                                             // where map m's features begin in a stored query: m * q_shift
+};
+template <int MAPS> struct QkParamsOf { using type = QkMapsParams; };
+template <> struct QkParamsOf<1> { using type = QkNormRopeParams; };
+__device__ __forceinline__ int map_width(const QkNormRopeParams& p) { return p.ks; }
+__device__ __forceinline__ int map_width(const QkMapsParams& p) { return p.kw; }
+__device__ __forceinline__ int map_shift(const QkNormRopeParams&) { return 0; }
+__device__ __forceinline__ int map_shift(const QkMapsParams& p) { return p.q_shift; }
+
 // Every head of the staged queries and keys divided by its own root mean square and multiplied by the weights of its
 // kind (one vector of hd weights for all query heads, one for all key heads).  A warp per head.
 __device__ __forceinline__ void norm_heads_in_place(float* qk_s, const QkNormRopeParams& p, int n_heads) {
@@ -46,13 +60,13 @@ __device__ __forceinline__ void norm_heads_in_place(float* qk_s, const QkNormRop
     }
 }
 
-template <typename TS, typename TQ, typename TC>
-__global__ void __launch_bounds__(256) qk_norm_rope_append_kernel(QkNormRopeParams p) {
+template <typename TS, typename TQ, typename TC, int MAPS>
+__global__ void __launch_bounds__(256) qk_norm_rope_append_kernel(typename QkParamsOf<MAPS>::type p) {
     extern __shared__ float qk_s[];                          // [nh*hd] queries, then [nkv*hd] keys
     __shared__ float red[32];
     pdl_launch();
     const int t = blockIdx.x;
-    const int qd = p.nh * p.hd, kd = p.pool ? p.nkv * p.hd : 0, vdd = p.pool ? p.nkv * p.vd : 0;
+    const int qd = p.nh * p.hd, kd = p.pool ? p.nkv * MAPS * p.hd : 0, vdd = p.pool ? p.nkv * p.vd : 0;
     const int half = p.rot / 2;
     const TS* row = (const TS*)p.src + (size_t)t * p.src_stride;
     // the token's place depends on no kernel of the step
@@ -79,7 +93,7 @@ __global__ void __launch_bounds__(256) qk_norm_rope_append_kernel(QkNormRopePara
     }
     if (p.wq && p.per_head) {
         __syncthreads();
-        norm_heads_in_place(qk_s, p, p.nh + (p.pool ? p.nkv : 0));
+        norm_heads_in_place(qk_s, p, p.nh + (p.pool ? p.nkv * MAPS : 0));
     } else if (p.wq) {
         ssq = block_sum(ssq, red);
         ssk = block_sum(ssk, red);
@@ -105,8 +119,8 @@ __global__ void __launch_bounds__(256) qk_norm_rope_append_kernel(QkNormRopePara
             const float c = cs[2 * pair], s = cs[2 * pair + 1], o = qk_s[partner];
             v = low ? v * c - o * s : v * c + o * s;
         }
-        if (i < qd) qo[(size_t)h * p.qs + f] = from_float<TQ>(v);
-        else if (k_base >= 0) pool[k_base + (size_t)h * p.page_size * p.ks + f] = from_float<TC>(v);
+        if (i < qd) qo[(size_t)h * p.qs + (h % MAPS) * map_shift(p) + f] = from_float<TQ>(v);
+        else if (k_base >= 0) pool[k_base + (size_t)(h / MAPS) * p.page_size * p.ks + (h % MAPS) * map_width(p) + f] = from_float<TC>(v);
     }
     if (v_base >= 0) {
         for (int i = threadIdx.x; i < vdd; i += blockDim.x) {
@@ -115,11 +129,16 @@ __global__ void __launch_bounds__(256) qk_norm_rope_append_kernel(QkNormRopePara
         }
     }
     // heads stored wider than they are: zeros behind every head
-    const int qpad = p.qs - p.hd, kpad = p.ks - p.hd, vpad = p.vs - p.vd;
-    for (int i = threadIdx.x; i < p.nh * qpad; i += blockDim.x) qo[(size_t)(i / qpad) * p.qs + p.hd + i % qpad] = from_float<TQ>(0.0f);
+    const int qpad = p.qs - p.hd, kpad = map_width(p) - p.hd, vpad = p.vs - p.vd;
+    for (int i = threadIdx.x; i < p.nh * qpad; i += blockDim.x) {
+        const int h = i / qpad, r = i - h * qpad;
+        qo[(size_t)h * p.qs + (r < (h % MAPS) * map_shift(p) ? r : r + p.hd)] = from_float<TQ>(0.0f);
+    }
     if (k_base >= 0)
-        for (int i = threadIdx.x; i < p.nkv * kpad; i += blockDim.x)
-            pool[k_base + (size_t)(i / kpad) * p.page_size * p.ks + p.hd + i % kpad] = from_float<TC>(0.0f);
+        for (int i = threadIdx.x; i < p.nkv * MAPS * kpad; i += blockDim.x) {
+            const int h = i / kpad;
+            pool[k_base + (size_t)(h / MAPS) * p.page_size * p.ks + (h % MAPS) * map_width(p) + p.hd + i % kpad] = from_float<TC>(0.0f);
+        }
     if (v_base >= 0)
         for (int i = threadIdx.x; i < p.nkv * vpad; i += blockDim.x)
             pool[v_base + (size_t)(i / vpad) * p.page_size * p.vs + p.vd + i % vpad] = from_float<TC>(0.0f);
@@ -129,13 +148,13 @@ __global__ void __launch_bounds__(256) qk_norm_rope_append_kernel(QkNormRopePara
 // rotation in halves or in neighbouring pairs: every access moves eight values, 16 bytes of bfloat16.  A thread's eight
 // features lie in one head and, in halves, on one side of the rotated part, so their partners are eight consecutive
 // features too; in neighbouring pairs they are four pairs of the thread's own.
-template <typename TS, typename TQ, typename TC>
-__global__ void __launch_bounds__(256) qk_norm_rope_append_vec8_kernel(QkNormRopeParams p) {
+template <typename TS, typename TQ, typename TC, int MAPS>
+__global__ void __launch_bounds__(256) qk_norm_rope_append_vec8_kernel(typename QkParamsOf<MAPS>::type p) {
     extern __shared__ float qk_s[];
     __shared__ float red[32];
     pdl_launch();
     const int t = blockIdx.x;
-    const int qd = p.nh * p.hd, kd = p.pool ? p.nkv * p.hd : 0, vdd = p.pool ? p.nkv * p.vd : 0;
+    const int qd = p.nh * p.hd, kd = p.pool ? p.nkv * MAPS * p.hd : 0, vdd = p.pool ? p.nkv * p.vd : 0;
     const int half = p.rot / 2;
     const TS* row = (const TS*)p.src + (size_t)t * p.src_stride;
     const int pos = p.positions[t];
@@ -172,7 +191,7 @@ __global__ void __launch_bounds__(256) qk_norm_rope_append_vec8_kernel(QkNormRop
     const bool whole = p.wq && !p.per_head;                  // the norm over the whole row is applied on the way out
     if (p.wq && p.per_head) {
         __syncthreads();
-        norm_heads_in_place(qk_s, p, p.nh + (p.pool ? p.nkv : 0));
+        norm_heads_in_place(qk_s, p, p.nh + (p.pool ? p.nkv * MAPS : 0));
     } else if (p.wq) {
         ssq = block_sum(ssq, red);
         ssk = block_sum(ssk, red);
@@ -212,8 +231,8 @@ __global__ void __launch_bounds__(256) qk_norm_rope_append_vec8_kernel(QkNormRop
                 v[e] = low ? v[e] * c - o * sn : v[e] * c + o * sn;
             }
         }
-        if (is_q) store8(qo + (size_t)h * p.qs + f, v);
-        else if (k_base >= 0) store8(pool + k_base + (size_t)h * p.page_size * p.ks + f, v);
+        if (is_q) store8(qo + (size_t)h * p.qs + (h % MAPS) * map_shift(p) + f, v);
+        else if (k_base >= 0) store8(pool + k_base + (size_t)(h / MAPS) * p.page_size * p.ks + (h % MAPS) * map_width(p) + f, v);
     }
     if (v_base >= 0) {
         for (int i = threadIdx.x * 8; i < vdd; i += blockDim.x * 8) {
@@ -230,11 +249,16 @@ __global__ void __launch_bounds__(256) qk_norm_rope_append_vec8_kernel(QkNormRop
         }
     }
     const float zero[8] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
-    const int qpad = (p.qs - p.hd) / 8, kpad = (p.ks - p.hd) / 8, vpad = (p.vs - p.vd) / 8;
-    for (int i = threadIdx.x; i < p.nh * qpad; i += blockDim.x) store8(qo + (size_t)(i / qpad) * p.qs + p.hd + 8 * (i % qpad), zero);
+    const int qpad = (p.qs - p.hd) / 8, kpad = (map_width(p) - p.hd) / 8, vpad = (p.vs - p.vd) / 8;
+    for (int i = threadIdx.x; i < p.nh * qpad; i += blockDim.x) {
+        const int h = i / qpad, r = 8 * (i - h * qpad);
+        store8(qo + (size_t)h * p.qs + (r < (h % MAPS) * map_shift(p) ? r : r + p.hd), zero);
+    }
     if (k_base >= 0)
-        for (int i = threadIdx.x; i < p.nkv * kpad; i += blockDim.x)
-            store8(pool + k_base + (size_t)(i / kpad) * p.page_size * p.ks + p.hd + 8 * (i % kpad), zero);
+        for (int i = threadIdx.x; i < p.nkv * MAPS * kpad; i += blockDim.x) {
+            const int h = i / kpad;
+            store8(pool + k_base + (size_t)(h / MAPS) * p.page_size * p.ks + (h % MAPS) * map_width(p) + p.hd + 8 * (i % kpad), zero);
+        }
     if (v_base >= 0)
         for (int i = threadIdx.x; i < p.nkv * vpad; i += blockDim.x)
             store8(pool + v_base + (size_t)(i / vpad) * p.page_size * p.vs + p.vd + 8 * (i % vpad), zero);
@@ -296,36 +320,46 @@ __global__ void sigmoid_gate_vec8_kernel(TO* __restrict__ out, int out_stride, c
 
 using namespace bg;
 
-template <typename TS, typename TQ, typename TC>
-static int qk_norm_rope_launch(const QkNormRopeParams& p, int T, cudaStream_t stream) {
-    const int width = p.nh * p.hd + (p.pool ? p.nkv * (p.hd + p.vd) : 0);
+template <typename TS, typename TQ, typename TC, int MAPS>
+static int qk_norm_rope_launch_maps(const QkMapsParams& p, int T, cudaStream_t stream) {
+    const int width = p.nh * p.hd + (p.pool ? p.nkv * (MAPS * p.hd + p.vd) : 0);
     const bool vec = !std::is_same<TQ, float>::value && p.hd % 8 == 0 && p.vd % 8 == 0 && p.rot % (p.interleaved ? 8 : 16) == 0 &&
-                     p.qs % 8 == 0 && p.ks % 8 == 0 && p.vs % 8 == 0 && p.src_stride % 8 == 0 && p.part_stride % 8 == 0 &&
+                     p.qs % 8 == 0 && p.ks % 8 == 0 && p.kw % 8 == 0 && p.q_shift % 8 == 0 && p.vs % 8 == 0 && p.src_stride % 8 == 0 && p.part_stride % 8 == 0 &&
                      p.q_stride % 8 == 0 && (uintptr_t)p.src % 16 == 0 && (uintptr_t)p.q_out % 16 == 0 && (uintptr_t)p.pool % 16 == 0 &&
                      (!p.wq || ((uintptr_t)p.wq % 16 == 0 && (uintptr_t)p.wk % 16 == 0)) && width > 0;
-    auto kern = vec ? qk_norm_rope_append_vec8_kernel<TS, TQ, TC> : qk_norm_rope_append_kernel<TS, TQ, TC>;
-    const size_t smem = (size_t)(p.nh * p.hd + (p.pool ? p.nkv * p.hd : 0)) * sizeof(float);
+    auto kern = vec ? qk_norm_rope_append_vec8_kernel<TS, TQ, TC, MAPS> : qk_norm_rope_append_kernel<TS, TQ, TC, MAPS>;
+    const size_t smem = (size_t)(p.nh * p.hd + (p.pool ? p.nkv * MAPS * p.hd : 0)) * sizeof(float);
     if (smem > 200 * 1024) return BG_ERR_SHAPE;
     if (smem > BG_SMEM_OPT_IN) {
         cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
         if (e != cudaSuccess) return (int)e;
     }
-    launch(kern, dim3(T), dim3(256), smem, stream, p);
+    launch(kern, dim3(T), dim3(256), smem, stream, static_cast<const typename QkParamsOf<MAPS>::type&>(p));
     BG_LAUNCH_CHECK();
     return BG_OK;
 }
 
+template <typename TS, typename TQ, typename TC>
+static int qk_norm_rope_launch(const QkMapsParams& p, int maps, int T, cudaStream_t stream) {
+    if (maps == 2) return qk_norm_rope_launch_maps<TS, TQ, TC, 2>(p, T, stream);
+    return qk_norm_rope_launch_maps<TS, TQ, TC, 1>(p, T, stream);
+}
+
+// `maps` 1 or 2: with 2, `nh` counts maps (two per query head), `qs` and `ks` are the stored widths of a map's query and of a kv
+// head's key row, and map m's features begin at m * q_shift of its stored query and at m * ks / 2 of the key row.
 extern "C" int bg_qk_norm_rope_append(const void* src, int src_dtype, int src_stride, int parts, long long part_stride,
                                       void* q_out, int q_dtype, int q_stride, const float* wq, const float* wk, float eps,
                                       const float* cos_sin, const int* positions, const int* row_req, const int* block_table,
                                       int max_pages, void* pool, int cache_dtype, int num_pages, int page_size, int T, int nh,
-                                      int nkv, int hd, int vd, int rot, int interleaved, int qs, int ks, int vs, int per_head,
+                                      int nkv, int hd, int vd, int rot, int interleaved, int qs, int ks, int vs, int per_head, int maps, int q_shift,
                                       unsigned* status, cudaStream_t stream) {
     if (T <= 0) return BG_OK;
     if (rot < 0 || rot > hd || rot % 2 || parts < 1 || (rot > 0 && !cos_sin) || ((wq == nullptr) != (wk == nullptr))) return BG_ERR_SHAPE;
-    if (qs < hd || ks < hd || vs < vd) return BG_ERR_SHAPE;
+    if (maps < 1 || maps > 2 || nh % maps || ks % maps || q_shift < 0) return BG_ERR_SHAPE;
+    if (qs < (maps - 1) * q_shift + hd || ks / maps < hd || vs < vd) return BG_ERR_SHAPE;
     if (src_dtype != q_dtype && src_dtype != BG_DTYPE_F32) return BG_ERR_DTYPE;
-    QkNormRopeParams p;
+    QkMapsParams p;
+    p.kw = ks / maps; p.q_shift = q_shift;
     p.src = src; p.src_stride = src_stride; p.parts = parts; p.part_stride = (size_t)part_stride; p.q_out = q_out;
     p.q_stride = q_stride; p.wq = wq; p.wk = wk; p.eps = eps; p.cos_sin = cos_sin; p.positions = positions; p.row_req = row_req;
     p.block_table = block_table; p.max_pages = max_pages; p.pool = pool; p.num_pages = num_pages; p.page_size = page_size;
@@ -334,10 +368,10 @@ extern "C" int bg_qk_norm_rope_append(const void* src, int src_dtype, int src_st
     if (cache_dtype != q_dtype) return BG_ERR_DTYPE;            // queries and cache are both of the compute type
     if (q_dtype == BG_DTYPE_F32) {
         if (src_dtype != BG_DTYPE_F32) return BG_ERR_DTYPE;
-        return qk_norm_rope_launch<float, float, float>(p, T, stream);
+        return qk_norm_rope_launch<float, float, float>(p, maps, T, stream);
     }
-    if (src_dtype == BG_DTYPE_F32) return qk_norm_rope_launch<float, __nv_bfloat16, __nv_bfloat16>(p, T, stream);
-    return qk_norm_rope_launch<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>(p, T, stream);
+    if (src_dtype == BG_DTYPE_F32) return qk_norm_rope_launch<float, __nv_bfloat16, __nv_bfloat16>(p, maps, T, stream);
+    return qk_norm_rope_launch<__nv_bfloat16, __nv_bfloat16, __nv_bfloat16>(p, maps, T, stream);
 }
 
 extern "C" int bg_sigmoid_gate(void* out, int out_dtype, int out_stride, const void* src, int src_stride, int vd, int head_stride,

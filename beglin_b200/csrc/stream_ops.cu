@@ -224,11 +224,12 @@ __global__ void rmsnorm_slice_kernel(const TI* __restrict__ src, int src_stride,
 }
 
 // out[t, h * vd + j] = src[h][t][j] * sigmoid(gate[t, gate_col0 + h]): head-major results put row by row,
-// each head scaled by its gate (without `gate`: put row by row as they are).
+// each head scaled by its gate (without `gate`: put row by row as they are).  `per_feature`: a gate for every feature,
+// gate[t, gate_col0 + h * vd + j].
 template <typename TI, typename TG, typename TO>
 __global__ void gate_heads_kernel(const TI* __restrict__ src, size_t src_head_stride, int src_row_stride,
                                   const TG* __restrict__ gate, int gate_stride, int gate_col0, TO* __restrict__ out,
-                                  int T, int H, int vd) {
+                                  int T, int H, int vd, int per_feature) {
     pdl_launch();
     pdl_wait();
     const size_t i = (size_t)blockIdx.x * blockDim.x + threadIdx.x;
@@ -237,7 +238,8 @@ __global__ void gate_heads_kernel(const TI* __restrict__ src, size_t src_head_st
     const int j = (int)(i % vd);
     const int h = (int)((i / vd) % H);
     const int t = (int)(i / ((size_t)vd * H));
-    const float s = gate ? 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * gate_stride + gate_col0 + h]))) : 1.0f;
+    const int gi = per_feature ? h * vd + j : h;
+    const float s = gate ? 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * gate_stride + gate_col0 + gi]))) : 1.0f;
     out[i] = from_float<TO>(to_float(src[(size_t)h * src_head_stride + (size_t)t * src_row_stride + j]) * s);
 }
 
@@ -245,7 +247,7 @@ __global__ void gate_heads_kernel(const TI* __restrict__ src, size_t src_head_st
 template <typename TI, typename TG, typename TO>
 __global__ void gate_heads_vec8_kernel(const TI* __restrict__ src, size_t src_head_stride, int src_row_stride,
                                        const TG* __restrict__ gate, int gate_stride, int gate_col0, TO* __restrict__ out,
-                                       int T, int H, int vd) {
+                                       int T, int H, int vd, int per_feature) {
     pdl_launch();
     pdl_wait();
     const int v8 = vd / 8;
@@ -255,11 +257,18 @@ __global__ void gate_heads_vec8_kernel(const TI* __restrict__ src, size_t src_he
     const int j = (int)(i % v8);
     const int h = (int)((i / v8) % H);
     const int t = (int)(i / ((size_t)v8 * H));
-    const float sg = gate ? 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * gate_stride + gate_col0 + h]))) : 1.0f;
     float v[8];
     load8(src + (size_t)h * src_head_stride + (size_t)t * src_row_stride + j * 8, v);
+    if (per_feature) {                       // (the gate's columns then lie on 16-byte boundaries)
+        float g[8];
+        load8(gate + (size_t)t * gate_stride + gate_col0 + h * vd + j * 8, g);
 #pragma unroll
-    for (int k = 0; k < 8; ++k) v[k] *= sg;
+        for (int k = 0; k < 8; ++k) v[k] /= 1.0f + expf(-g[k]);
+    } else {
+        const float sg = gate ? 1.0f / (1.0f + expf(-to_float(gate[(size_t)t * gate_stride + gate_col0 + h]))) : 1.0f;
+#pragma unroll
+        for (int k = 0; k < 8; ++k) v[k] *= sg;
+    }
     store8(out + ((size_t)t * H + h) * vd + j * 8, v);
 }
 
@@ -367,21 +376,23 @@ extern "C" int bg_rmsnorm_slice(const void* src, int src_dtype, int src_stride, 
 
 extern "C" int bg_gate_heads(const void* src, int src_dtype, long long src_head_stride, int src_row_stride, const void* gate,
                              int gate_dtype, int gate_stride, int gate_col0, void* out, int out_dtype, int T, int H, int vd,
-                             cudaStream_t stream) {
+                             int per_feature, cudaStream_t stream) {
     const long long n = (long long)T * H * vd;
     if (n <= 0) return BG_OK;
-    if (vd % 8 == 0 && src_head_stride % 8 == 0 && src_row_stride % 8 == 0 && (uintptr_t)src % 16 == 0 && (uintptr_t)out % 16 == 0) {
+    const bool gate_vec = !per_feature || (gate_stride % 8 == 0 && gate_col0 % 8 == 0 && (uintptr_t)gate % 16 == 0);
+    if (per_feature && !gate) return BG_ERR_SHAPE;
+    if (vd % 8 == 0 && src_head_stride % 8 == 0 && src_row_stride % 8 == 0 && (uintptr_t)src % 16 == 0 && (uintptr_t)out % 16 == 0 && gate_vec) {
         const size_t n8 = (size_t)n / 8;
         BG_DISPATCH_DTYPE(src_dtype, TI, BG_DISPATCH_DTYPE(gate_dtype, TG, BG_DISPATCH_DTYPE(out_dtype, TO,
             launch(gate_heads_vec8_kernel<TI, TG, TO>, dim3((unsigned)((n8 + 255) / 256)), dim3(256), 0, stream, (const TI*)src,
-                   (size_t)src_head_stride, src_row_stride, (const TG*)gate, gate_stride, gate_col0, (TO*)out, T, H, vd))));
+                   (size_t)src_head_stride, src_row_stride, (const TG*)gate, gate_stride, gate_col0, (TO*)out, T, H, vd, per_feature))));
         BG_LAUNCH_CHECK();
         return BG_OK;
     }
     const unsigned blocks = (unsigned)((n + 255) / 256);
     BG_DISPATCH_DTYPE(src_dtype, TI, BG_DISPATCH_DTYPE(gate_dtype, TG, BG_DISPATCH_DTYPE(out_dtype, TO,
         launch(gate_heads_kernel<TI, TG, TO>, dim3(blocks), dim3(256), 0, stream, (const TI*)src, (size_t)src_head_stride,
-               src_row_stride, (const TG*)gate, gate_stride, gate_col0, (TO*)out, T, H, vd))));
+               src_row_stride, (const TG*)gate, gate_stride, gate_col0, (TO*)out, T, H, vd, per_feature))));
     BG_LAUNCH_CHECK();
     return BG_OK;
 }

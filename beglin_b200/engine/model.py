@@ -134,6 +134,8 @@ class DecoderModel:
                 rows = stream.x.clone()
                 if stream.pending is not None:
                     rows += stream.pending.float().reshape(-1, *rows.shape).sum(0)
+                if stream.step is not None:
+                    rows += stream.step.float(rows)
                 if stream.terms is not None:
                     for t, c in stream.terms.items:
                         rows += c * t.float().reshape(-1, *rows.shape).sum(0)      # (a normed term's float() is its normed rows)

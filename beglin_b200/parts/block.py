@@ -11,7 +11,7 @@ import torch
 
 from ..csrc import ops
 from .registry import register_block
-from .stream import NormedInput, ResidualStream, Terms
+from .stream import NormedInput, NormedStep, ResidualStream, Terms
 
 
 @register_block("prenorm")
@@ -175,3 +175,50 @@ class ParallelMixerBlock(ParallelBlock):
 class ParallelSharedBlock(ParallelBlock):
     """The parallel layer with ONE norm, whose rows both sublayers read: h = norm(x), x <- x + m (mixer(h) + feed_forward(h))."""
     SLOTS = (("mixer_norm", "norm"), ("mixer", "mixer"), ("feed_forward", "feed_forward"))
+
+
+@register_block("sandwich")
+class SandwichBlock:
+    """Every sublayer has a norm in front of it and another on its result: x <- x + norm2(mixer(norm1(x))), then
+    x <- x + norm4(feed_forward(norm3(x))), all RMS norms.  A sublayer's result stays owed to the stream until the next norm
+    reads it: ONE kernel norms the result, adds it to the float stream and norms the new rows for the next sublayer."""
+    SLOTS = (("mixer_norm", "norm"), ("mixer", "mixer"), ("mixer_out_norm", "norm"),
+             ("feed_forward_norm", "norm"), ("feed_forward", "feed_forward"), ("feed_forward_out_norm", "norm"))
+
+    def __init__(self, mixer_norm, mixer, mixer_out_norm, feed_forward_norm=None, feed_forward=None, feed_forward_out_norm=None):
+        for norm in (mixer_norm, mixer_out_norm, feed_forward_norm, feed_forward_out_norm):
+            if norm is not None and getattr(norm, "kind", None) != "rmsnorm":
+                raise ValueError("a block with norms in front of and behind its sublayers takes RMS norms")
+        self.mixer_norm, self.mixer, self.mixer_out_norm = mixer_norm, mixer, mixer_out_norm
+        self.feed_forward_norm, self.feed_forward, self.feed_forward_out_norm = feed_forward_norm, feed_forward, feed_forward_out_norm
+
+    @staticmethod
+    def read(stream: ResidualStream, norm) -> torch.Tensor:
+        """The normed rows of the stream with everything it is owed added."""
+        if stream.terms is not None or stream.pending is not None:      # something an earlier block of another kind still owes
+            stream.settle()
+            if stream.pending is not None:
+                ops.add_residual(stream.x, stream.pending)
+                stream.updated(None)
+        return stream.normed_step(norm, norm.ctx.compute_dtype)
+
+    def forward(self, stream: ResidualStream, batch, cache) -> None:
+        h = self.read(stream, self.mixer_norm)
+        if getattr(self.mixer, "takes_stream", False):
+            y = self.mixer.forward(h, batch, cache, None)
+        else:
+            y = self.mixer.forward(h, batch, cache)
+        stream.step = NormedStep(y, self.mixer_out_norm)
+        if self.feed_forward is not None:
+            h = self.read(stream, self.feed_forward_norm)
+            if getattr(self.feed_forward, "takes_stream", False):
+                y = self.feed_forward.forward(h, batch, None)
+            else:
+                y = self.feed_forward.forward(h, batch)
+            stream.step = NormedStep(y, self.feed_forward_out_norm)
+
+
+@register_block("sandwich_mixer")
+class SandwichMixerBlock(SandwichBlock):
+    """The same layer without a feed-forward."""
+    SLOTS = (("mixer_norm", "norm"), ("mixer", "mixer"), ("mixer_out_norm", "norm"))

@@ -4,6 +4,10 @@
 meets the stream.  It stands in front of every pass of a run of layers that is repeated with the same weights.  The
 product is split in its halves, W [x; e] = W_x x + W_e e: the second term is the same for every pass of a step and is
 computed once; the sum of the two is float and becomes the new stream.
+
+"pass_step": x <- x (+ e) + P[t], a learned row for pass t of a repeated run of layers, and, in front of every pass but the
+first, the embedded rows once more.  Both stay owed to the stream and are added by the kernel that norms it for the pass's
+first sublayer.
 """
 from __future__ import annotations
 
@@ -15,8 +19,8 @@ from ..csrc import ops
 from .context import BuildContext
 from .linear import Linear
 from .registry import register_entry
-from .spec import InputMixSpec, TensorRole
-from .stream import ResidualStream
+from .spec import InputMixSpec, PassStepSpec, TensorRole
+from .stream import NormedStep, ResidualStream
 
 
 @register_entry("input_mix")
@@ -52,3 +56,25 @@ class InputMix:
         moving = self.of_stream.partial(stream.lowp if stream.lowp is not None else self._rows(stream.x))
         ops.add_terms_norm(stream.x, [(moving, 1.0), (fixed, 1.0)], assign=True)
         stream.updated(None)
+
+
+@register_entry("pass_step")
+class PassStep:
+    @staticmethod
+    def expected_tensors(spec: PassStepSpec) -> List[TensorRole]:
+        return [TensorRole("step", (spec.passes, spec.hidden))]
+
+    def __init__(self, spec: PassStepSpec, tensors: Dict[str, torch.Tensor], ctx: BuildContext):
+        if not 0 <= spec.index < spec.passes:
+            raise ValueError(f"pass {spec.index} of {spec.passes}")
+        self.spec, self.ctx = spec, ctx
+        self.needs_origin = spec.again
+        self.vector = tensors["step"][spec.index].to(device=ctx.device, dtype=torch.float32).contiguous()
+
+    def forward(self, stream: ResidualStream, batch) -> None:
+        step = stream.step if stream.step is not None else NormedStep()
+        if step.again is not None or step.vector is not None:           # (two entries in front of one stage)
+            stream.settle()
+            step = NormedStep()
+        step.again, step.vector = (stream.origin if self.spec.again else None), self.vector
+        stream.step, stream.ssq, stream.lowp = step, None, None

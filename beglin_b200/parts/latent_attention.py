@@ -1,4 +1,4 @@
-"""Attention through a low-rank latent, with an output gate per head.
+"""Attention through a low-rank latent, with an output gate per head or per feature.
 
 Of every position only ONE row is cached for all heads: the RMS-normed latent c (kv_rank features) and the
 rotated key part k_r (rot_dim features) that the heads share.  A head's keys W_uk c and values W_uv c are
@@ -15,7 +15,9 @@ query product; queries into the latent space; attention (the queries' rotated pa
 and the merge of its splits; values out of the latent space; gates; the output product, which in steps of
 few rows adds into the residual stream itself.  A mixer with `own_kv` False has no key/value projection and
 reads the cache of the stage it is told to.  Options of the spec: queries that are one product of the input (no query
-latent), no rotated part, no gates, a sliding window.
+latent), no rotated part, no gates or a gate per feature, a sliding window, a learned sink per head (which the kernel that
+merges the ranges of keys takes into the denominator).  Gates per feature are as many as the joined heads' features: in steps of
+many rows they are a product of their own, in the compute type.
 
 Long prompt portions in bfloat16 go the other way round where the sizes allow it (dim + rot_dim = vdim = 64 or
 128): the keys and values of all heads are made once per step from the request's cached rows, by ONE product
@@ -58,7 +60,9 @@ class LatentAttention:
             roles += [TensorRole("kv_down.weight", (spec.kv_rank + spec.rot_dim, spec.hidden), True, True),
                       TensorRole("kv_down.norm", (spec.kv_rank,), role="scale")]
         if spec.gated:
-            roles.append(TensorRole("gate.weight", (H, spec.hidden), True, True))
+            roles.append(TensorRole("gate.weight", (H * spec.vdim if spec.gate_features else H, spec.hidden), True, True))
+        if spec.sink:
+            roles.append(TensorRole("sink", (H,)))
         return roles
 
     @staticmethod
@@ -83,13 +87,24 @@ class LatentAttention:
         self.window = int(spec.window) if spec.window else 0
         names = ([] if self.direct_q else ["q_down.weight"]) + (["kv_down.weight"] if spec.own_kv else []) \
             + (["gate.weight"] if spec.gated else [])
-        w_down = torch.cat([tensors[n] for n in names], dim=0)
+        rows = [tensors[n] for n in names]
+        self.wide_gate = spec.gated and spec.gate_features
+        latent_rows = sum(w.shape[0] for w in rows[:-1]) if self.wide_gate else 0
+        gate_pad = -latent_rows % 16                # (the gates begin on a multiple of 16 columns)
+        if gate_pad:
+            rows.insert(-1, torch.zeros((gate_pad, spec.hidden), dtype=rows[0].dtype, device=rows[0].device))
+        w_down = torch.cat(rows, dim=0)
         if w_down.shape[0] % 16:                    # rows of zeros up to a multiple of 16 outputs: a width that is no multiple
             pad = 16 - w_down.shape[0] % 16         # of 8 takes the library's product of many rows off its fast kernels
             w_down = torch.cat([w_down, torch.zeros((pad, w_down.shape[1]), dtype=w_down.dtype, device=w_down.device)], dim=0)
         self.down = Linear(w_down, None, ctx, label="proj_qkv")
         self.kv_col = self.q_rank
-        self.gate_col = self.q_rank + (spec.kv_rank + spec.rot_dim if spec.own_kv else 0)
+        self.gate_col = self.q_rank + (spec.kv_rank + spec.rot_dim if spec.own_kv else 0) + gate_pad
+        self.down_parts = {}                        # the two parts of the same matrix (views of it), for steps of many rows
+        if self.wide_gate:
+            self.down_parts = {"latent": Linear(self.down.weight[:self.gate_col], None, ctx, label="proj_qkv"),
+                               "gate": Linear(self.down.weight[self.gate_col:], None, ctx, label="proj_gate")}
+        self.sink_weight = tensors["sink"].to(device=ctx.device, dtype=torch.float32).contiguous() if spec.sink else None
         self.q_norm = None if self.direct_q else ctx.vector(tensors["q_down.norm"])
         self.kv_norm = ctx.vector(tensors["kv_down.norm"]) if spec.own_kv else None
         self.q_up = Linear(tensors["q_proj.weight" if self.direct_q else "q_up.weight"], None, ctx, label="proj_q")
@@ -123,6 +138,7 @@ class LatentAttention:
                 self.expand = (bq, tile)
                 self.kv_up = ctx.matrix(torch.cat([tensors["k_up.weight"], tensors["v_up.weight"]], dim=0))
 
+    WIDE_ROWS = 17             # from this many rows on gates per feature are a product of their own
     EXPAND_ROWS = 128          # portions of one request of at least this many rows make per-head keys and values
 
     def _per_head(self, x: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
@@ -137,7 +153,7 @@ class LatentAttention:
                 return torch.bmm(x, w.transpose(1, 2))
             return torch.bmm(x, w.transpose(1, 2), out_dtype=out_dtype)
 
-    def _per_head_keys(self, q: torch.Tensor, down: torch.Tensor, cos_sin, batch, cache: PagedKVView) -> torch.Tensor:
+    def _per_head_keys(self, q: torch.Tensor, gate: Optional[torch.Tensor], gate_col: int, cos_sin, batch, cache: PagedKVView) -> torch.Tensor:
         """The gated heads [T, H vdim] of a portion of ONE request, through keys and values made per head."""
         s, ctx = self.spec, self.ctx
         T, H, hd = batch.n_rows, s.n_heads, s.dim + s.rot_dim
@@ -161,11 +177,14 @@ class LatentAttention:
         qblk, n_qblk = batch.query_blocks(bq)
         att = torch.empty((T, H * hd), dtype=torch.bfloat16, device=q.device)
         ops.attention(q, q.stride(0), pages, table, batch.positions, qblk, n_qblk, batch.max_position, T, H, H, hd, self.window,
-                      ctx.kv_split, tile, bq, self.scale, att, ctx.status, "tc_rows")
+                      ctx.kv_split, tile, bq, self.scale, att, ctx.status, "tc_rows", sink_weight=self.sink_weight)
         if not s.gated:
             return att
+        if s.gate_features:
+            ops.sigmoid_gate(att, gate, gate_col, H * hd)
+            return att
         out = torch.empty((T, H * hd), dtype=torch.bfloat16, device=q.device)
-        ops.gate_heads(att.view(T, H, hd).transpose(0, 1), down, self.gate_col, out)
+        ops.gate_heads(att.view(T, H, hd).transpose(0, 1), gate, gate_col, out)
         return out
 
     takes_stream = True        # forward takes a NormedInput and may add its result to the stream itself
@@ -177,7 +196,11 @@ class LatentAttention:
             h = h.tensor()
         s, ctx = self.spec, self.ctx
         T, H = batch.n_rows, s.n_heads
-        down = self.down.full_f32(h)                                    # [T, q_rank (+ kv_rank + rot) (+ H)]
+        if self.wide_gate and T >= self.WIDE_ROWS:
+            down, gate, gate_col = self.down_parts["latent"].full_f32(h), self.down_parts["gate"](h), 0
+        else:
+            down = self.down.full_f32(h)                                # [T, q_rank (+ kv_rank + rot) (+ gates)]
+            gate, gate_col = down, self.gate_col
         cos_sin = self.position.table(batch) if self.rot_dims else None
         if self.direct_q:
             ops.latent_append(down, self.kv_col, s.kv_rank, s.rot_dim, self.rot_dims, self.kv_norm, s.eps, cos_sin,
@@ -193,7 +216,7 @@ class LatentAttention:
                 ops.rmsnorm_slice(down, 0, s.q_rank, self.q_norm, s.eps, cq)
             q = self.q_up(cq)                                           # [T, H (dim + rot)]
         if self.expand is not None and batch.n_req == 1 and T >= self.EXPAND_ROWS:
-            return self._result(self._per_head_keys(q, down, cos_sin, batch, cache), stream)
+            return self._result(self._per_head_keys(q, gate, gate_col, cos_sin, batch, cache), stream)
         q_plain = q.view(T, H, s.dim + s.rot_dim)[:, :, :s.dim].transpose(0, 1)          # [H, T, dim]
         q_lat = self._per_head(q_plain, self.k_up_t, torch.float32)    # [H, T, kv_rank] float
         hc, bq, stages = (self.hc, self.bq, 0) if self.mma is None else self.mma
@@ -207,10 +230,10 @@ class LatentAttention:
         o_lat = torch.empty((H, T, s.kv_rank), dtype=ctx.compute_dtype, device=h.device)
         ops.latent_attention(q_lat, q, s.dim, s.rot_dim, self.rot_dims, cos_sin, cache.pool, cache.block_table,
                              batch.positions, qblk, n_qblk, batch.max_position, bq, hc, self.tile, split,
-                             self.scale, o_lat, ctx.status, mma_stages=stages, window=self.window)
+                             self.scale, o_lat, ctx.status, mma_stages=stages, window=self.window, sink_weight=self.sink_weight)
         v = self._per_head(o_lat, self.v_up, ctx.compute_dtype)        # [H, T, vdim]
         out = torch.empty((T, H * s.vdim), dtype=ctx.compute_dtype, device=h.device)
-        ops.gate_heads(v, down if s.gated else None, self.gate_col, out)      # (without gates: the heads row by row)
+        ops.gate_heads(v, gate if s.gated else None, gate_col, out, per_feature=self.wide_gate)      # (without gates: the heads row by row)
         return self._result(out, stream)
 
     def _result(self, heads: torch.Tensor, stream: Optional[ResidualStream]) -> Optional[torch.Tensor]:

@@ -86,14 +86,15 @@ class Linear:
         """Whether a step of T rows runs the gated product of many rows on pairs of CTAs (and not the fused one of few)."""
         return self._tc is not None and not self.fuses(T) and self._tc.pairs(T)
 
-    def of(self, inp, swiglu: bool = False, activation: str = "silu") -> torch.Tensor:
+    def of(self, inp, swiglu: bool = False, activation: str = "silu", limit: float = 0.0) -> torch.Tensor:
         """The product of `inp`, a tensor [T, in] or a NormedInput (a norm of the residual stream that has
         not been computed).  Where the fused product runs, the norm is applied to the operand inside it;
         the result is then complete ([T, out], float).  Else as `partial`.  With `swiglu` (the weight's
         rows interleaved in blocks of 64, gate then up) the result is silu(gate) * up, [T, out / 2] in the
         compute type (from the fused product of few rows or from the product of many rows on pairs of CTAs), or
-        None when this step runs neither.  `activation` other than silu is known to the product of many rows only."""
-        if swiglu and activation != "silu" and not self.pairs(inp.rows if isinstance(inp, NormedInput) else inp.shape[0]):
+        None when this step runs neither.  `activation` "glu_clamped" (with its `limit`) is known to both, any other than silu
+        to the product of many rows only."""
+        if swiglu and activation not in ("silu", "glu_clamped") and not self.pairs(inp.rows if isinstance(inp, NormedInput) else inp.shape[0]):
             return None
         lazy = isinstance(inp, NormedInput)
         T = inp.rows if lazy else inp.shape[0]
@@ -102,7 +103,7 @@ class Linear:
                 if self._tc is None or not self._tc.pairs(T):
                     return None
                 with ops.phase(self.label):
-                    return self._tc.pair_swiglu(inp.tensor() if lazy else inp, activation)
+                    return self._tc.pair_swiglu(inp.tensor() if lazy else inp, activation, limit)
             return self.partial(inp.tensor() if lazy else inp)
         fusion = inp.fusable() if lazy else None
         n = self.out_features // 2 if swiglu else self.out_features
@@ -112,12 +113,12 @@ class Linear:
             weight, eps = fusion
             with ops.phase(self.label):
                 self._tc.fused(T, out, mode, xf=inp.stream.x, ssq_in=inp.stream.ssq, norm_weight=weight, eps=eps,
-                               bias=self.bias_f32)
+                               bias=self.bias_f32, limit=limit if swiglu else 0.0)
         else:
             x = inp.tensor() if lazy else inp
             self._check_rows(x)
             with ops.phase(self.label):
-                self._tc.fused(T, out, mode, x=x, bias=self.bias_f32)
+                self._tc.fused(T, out, mode, x=x, bias=self.bias_f32, limit=limit if swiglu else 0.0)
         return out
 
     def rope_fuses(self, T: int, hd: int) -> bool:

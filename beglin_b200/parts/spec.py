@@ -107,11 +107,34 @@ class AttentionSpec:
 
 
 @dataclass(frozen=True)
+class DifferentialAttentionSpec:
+    """Grouped-query attention whose heads are pairs of maps: a query head has two queries and a kv head two keys of `dim`
+    features each (stored head by head, first map then second), and ONE value of `vdim` features that both maps weigh.  With a1,
+    a2 the maps' results and lambda = exp(lq1 . lk1) - exp(lq2 . lk2) + `diff` (four learned vectors of `dim` values, one number
+    per layer) a head's result is a1 - lambda a2, divided by its root mean square (`eps`), times 1 - `diff`.  q, k and v have
+    biases; `position.rotary_dim` leading features of every map turn.  `window` as in AttentionSpec."""
+    hidden: int
+    n_heads: int
+    n_kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    diff: float
+    eps: float
+    position: PositionSpec
+    qkv_bias: bool = True
+    window: Optional[int] = None
+    kind: str = "differential_attention"
+
+
+@dataclass(frozen=True)
 class SwiGLUSpec:
-    """down(act(gate(h)) * up(h)); `activation` "silu" or "gelu_tanh" (the tanh form of GELU)."""
+    """down(act(gate(h)) * up(h)); `activation` "silu", "gelu_tanh" (the tanh form of GELU) or "glu_clamped": with g = min(gate(h),
+    `limit`) and u = clamp(up(h), -limit, limit) the down product takes g sigmoid(1.702 g) (u + 1)."""
     hidden: int
     intermediate: int
     activation: str = "silu"
+    limit: float = 0.0
     kind: str = "swiglu"
 
 
@@ -159,7 +182,9 @@ class LatentAttentionSpec:
     sigmoid of a per-head gate read from the mixer's input when `gated`.  `own_kv` False: no down-projection
     of its own; the latent and key part of another stage's cache are read.  `q_rank` None: the queries are one product
     of the mixer's input (tensor `q_proj.weight`), without a latent of their own.  `rot_dim` 0: no rotated part at all.
-    `window` w: a query sees itself and the w - 1 positions before it."""
+    `window` w: a query sees itself and the w - 1 positions before it.  `gate_features`: the gates are one number per feature of
+    the joined heads in place of one per head.  `sink`: the softmax's denominator also holds exp of a learned number per head
+    (tensor `sink`) that has no key and no value."""
     hidden: int
     n_heads: int
     dim: int
@@ -173,6 +198,8 @@ class LatentAttentionSpec:
     gated: bool = True
     own_kv: bool = True
     window: Optional[int] = None
+    gate_features: bool = False
+    sink: bool = False
     kind: str = "latent_attention"
 
 
@@ -252,6 +279,17 @@ class InputMixSpec:
     [hidden, 2 hidden] (the stream's half first)."""
     hidden: int
     kind: str = "input_mix"
+
+
+@dataclass(frozen=True)
+class PassStepSpec:
+    """What stands in front of pass `index` of a run of layers that is passed `passes` times: the stream gets, with `again`,
+    the embedded rows of the step once more, and the row `index` of a learned table [passes, hidden] (tensor `step`)."""
+    hidden: int
+    passes: int
+    index: int
+    again: bool
+    kind: str = "pass_step"
 
 
 @dataclass(frozen=True)

@@ -45,6 +45,27 @@ class NormedTerm:
         return v * torch.rsqrt((v * v).mean(-1, keepdim=True) + self.eps) * self.weight
 
 
+@dataclass
+class NormedStep:
+    """What is owed to the stream by layers that norm a sublayer's result: `rows` ([T, d] or partial sums [parts, T, d]), which
+    is RMS-normed (`norm`, a part) before it is added, and what the beginning of a pass adds besides: float rows [T, d] and a float
+    vector [d] for every row."""
+    rows: Optional[torch.Tensor] = None
+    norm: object = None
+    again: Optional[torch.Tensor] = None
+    vector: Optional[torch.Tensor] = None
+
+    def float(self, like: torch.Tensor) -> torch.Tensor:
+        """The addend of `like`'s shape, formed by torch operations (for looking into a model)."""
+        out = torch.zeros_like(like)
+        if self.rows is not None:
+            out += NormedTerm(self.rows, self.norm.weight_f32(), self.norm.spec.eps).float()
+        for extra in (self.again, self.vector):
+            if extra is not None:
+                out += extra
+        return out
+
+
 class ResidualStream:
     def __init__(self, x: torch.Tensor):
         self.x = x                                     # float32 [T, d]
@@ -56,6 +77,7 @@ class ResidualStream:
         #                                                x left them (for sublayers that read the stream un-normed)
         self.terms: Optional[Terms] = None             # not yet added to x either: results with constants of their own
         #                                                (a block that adds scaled sums; whoever reads x calls settle())
+        self.step: Optional[NormedStep] = None         # not yet added to x either: a result that is normed before it is added
         self.origin: Optional[torch.Tensor] = None     # float32 [T, d]: the embedded rows, kept for parts that mix them in
         self.lanes: Optional[torch.Tensor] = None      # float32 [n, T, d]: the residual as n lanes (then x is not the residual)
         self.lane_owed = None                          # (result, link) of the last sublayer, not yet written to the lanes
@@ -104,6 +126,22 @@ class ResidualStream:
             from ..csrc import ops
             ops.add_terms_norm(self.x, self.terms.items)
             self.terms, self.ssq, self.lowp = None, None, None
+        if self.step is not None:
+            self.normed_step()
+
+    def normed_step(self, norm=None, dtype: Optional[torch.dtype] = None) -> Optional[torch.Tensor]:
+        """Adds the owed `step` to x, and with `norm` (an RMS norm) also returns the normed rows of the new x in `dtype`: one
+        pass over the rows for both.  Nothing else may be owed then."""
+        from ..csrc import ops
+        s = self.step if self.step is not None else NormedStep()
+        h = None if norm is None else torch.empty(self.x.shape, dtype=dtype, device=self.x.device)
+        wy, w = None if s.norm is None else s.norm.weight, None if norm is None else norm.weight
+        if wy is not None and w is not None and wy.dtype != w.dtype:
+            wy, w = s.norm.weight_f32(), norm.weight_f32()
+        ops.norm_step(self.x, s.rows, wy, 0.0 if s.norm is None else s.norm.spec.eps, rows=s.again, vector=s.vector, weight=w,
+                      eps=0.0 if norm is None else norm.spec.eps, out=h)
+        self.step, self.ssq, self.lowp = None, None, None
+        return h
 
     def owe(self, addend: torch.Tensor) -> None:
         self.pending, self.ssq, self.lowp = addend, None, None
@@ -139,6 +177,6 @@ class NormedInput:
     def fusable(self):
         """(weight, eps) of the norm when a product may apply it to the stream itself, else None."""
         s = self.stream
-        if self._tensor is not None or s.pending is not None or s.terms is not None or s.ssq is None:
+        if self._tensor is not None or s.pending is not None or s.terms is not None or s.step is not None or s.ssq is None:
             return None
         return getattr(self.norm, "fusion", lambda: None)()

@@ -79,13 +79,13 @@ class TensorCoreProduct:
     def fused(self, T: int, out: torch.Tensor, mode: int, x: Optional[torch.Tensor] = None,
               xf: Optional[torch.Tensor] = None, ssq_in: Optional[torch.Tensor] = None,
               norm_weight: Optional[torch.Tensor] = None, eps: float = 0.0, bias: Optional[torch.Tensor] = None,
-              want_ssq: bool = False) -> Optional[torch.Tensor]:
+              want_ssq: bool = False, limit: float = 0.0) -> Optional[torch.Tensor]:
         """ops.gemm_fused with this weight; returns the sums of squares of the new rows when asked."""
         s = self.fused_splits(T)
         ssq_out = torch.empty((self.tiles * s, 64), dtype=torch.float32, device=out.device) if want_ssq else None
         ops.gemm_fused_unchecked(self._w_ptr, self.n_out, self.k, self._ldw, T, out, mode, x, xf, ssq_in,
                                  None if norm_weight is None else norm_weight.data_ptr(), eps,
-                                 None if bias is None else bias.data_ptr(), ssq_out, s, self._status_ptr)
+                                 None if bias is None else bias.data_ptr(), ssq_out, s, self._status_ptr, limit)
         return ssq_out
 
     ROPE_HEAD_SIZES = (32, 64, 128)      # whole heads in a tile of 128 rows, so that a feature meets its partner
@@ -107,13 +107,14 @@ class TensorCoreProduct:
         have too few 256 x 256 tiles for the pairs of the device."""
         return self.ctx.fuse and T >= PAIR_TOKENS and self.n_out % 128 == 0
 
-    def pair_swiglu(self, x: torch.Tensor, activation: str = "silu") -> torch.Tensor:
+    def pair_swiglu(self, x: torch.Tensor, activation: str = "silu", limit: float = 0.0) -> torch.Tensor:
         """act(gate) * up of x's rows, [T, n_out / 2] bfloat16; the weight's rows are interleaved in blocks of 64; act is
-        silu or the tanh form of GELU."""
+        silu or the tanh form of GELU, or the whole is the clamped form."""
         if x.dtype != torch.bfloat16 or x.stride(1) != 1 or x.shape[1] != self.k or x.stride(0) % 8:
             raise ops.KernelError(f"the tcgen05 product takes contiguous bfloat16 rows of {self.k} features")
         out = torch.empty((x.shape[0], self.n_out // 2), dtype=torch.bfloat16, device=x.device)
-        ops.gemm_pair_unchecked(x, self._w_ptr, self.n_out, self.k, self._ldw, out, ops.PAIR_GLU[activation], self._status_ptr)
+        ops.gemm_pair_unchecked(x, self._w_ptr, self.n_out, self.k, self._ldw, out, ops.PAIR_GLU[activation], self._status_ptr,
+                                limit=limit)
         return out
 
     def pair_residual(self, x: torch.Tensor, bias: Optional[torch.Tensor], stream_x: torch.Tensor) -> None:
