@@ -251,6 +251,22 @@ __global__ void __launch_bounds__(1024) norm_step_vec4_kernel(NormStepParams p) 
     pdl_launch();
     const int d4 = p.d >> 2;
     const size_t base = (size_t)blockIdx.x * p.d;
+    // bfloat16 weights are asked for before the wait for the kernel ahead (no kernel of the step writes them)
+    constexpr bool AHEAD = !std::is_same<TW, float>::value && ITER <= 2;
+    uint2 wy_raw[AHEAD ? ITER : 1], w_raw[AHEAD ? ITER : 1];
+    if constexpr (AHEAD) {
+#pragma unroll
+        for (int it = 0; it < ITER; ++it) {
+            const int c = threadIdx.x + it * blockDim.x;
+            if (c >= d4) continue;
+            if (p.y) wy_raw[it] = *reinterpret_cast<const uint2*>((const TW*)p.wy + 4 * c);
+            if (p.out) w_raw[it] = *reinterpret_cast<const uint2*>((const TW*)p.w + 4 * c);
+        }
+    }
+    auto weight4 = [&](const void* w, const uint2* raw, int it, int c) {
+        if constexpr (AHEAD) return step_load4(reinterpret_cast<const __nv_bfloat16*>(raw + it));
+        else return step_load4((const TW*)w + 4 * c);
+    };
     pdl_wait();
     float4 xv[ITER];
     float inv = 0.0f;
@@ -279,7 +295,7 @@ __global__ void __launch_bounds__(1024) norm_step_vec4_kernel(NormStepParams p) 
             if (c >= d4) continue;
             float4 v = xv[it];
             if (p.y) {
-                const float4 w = step_load4((const TW*)p.wy + 4 * c);
+                const float4 w = weight4(p.wy, wy_raw, it, c);
                 v.x += yv[it].x * inv * w.x; v.y += yv[it].y * inv * w.y; v.z += yv[it].z * inv * w.z; v.w += yv[it].w * inv * w.w;
             }
             if (p.rows) {
@@ -307,7 +323,7 @@ __global__ void __launch_bounds__(1024) norm_step_vec4_kernel(NormStepParams p) 
     for (int it = 0; it < ITER; ++it) {
         const int c = threadIdx.x + it * blockDim.x;
         if (c >= d4) continue;
-        const float4 w = step_load4((const TW*)p.w + 4 * c), v = xv[it];
+        const float4 w = weight4(p.w, w_raw, it, c), v = xv[it];
         step_store4((TO*)p.out + base + 4 * c, make_float4(v.x * inv * w.x, v.y * inv * w.y, v.z * inv * w.z, v.w * inv * w.w));
     }
 }

@@ -264,6 +264,111 @@ __global__ void __launch_bounds__(256) qk_norm_rope_append_vec8_kernel(typename 
             store8(pool + v_base + (size_t)(i / vpad) * p.page_size * p.vs + p.vd + 8 * (i % vpad), zero);
 }
 
+// The same without norms (sizes as for the kernel above, bfloat16 queries and cache): nothing of a row is needed by more than one
+// thread, so nothing passes through shared memory and no thread waits for another.  A thread takes eight features that turn
+// together with the eight at the other side of the rotated part (in neighbouring pairs: eight features), eight that pass, or
+// eight of a value; one block per token.
+template <typename TS, typename TQ, typename TC, int MAPS>
+__global__ void __launch_bounds__(256) rope_append_vec8_kernel(typename QkParamsOf<MAPS>::type p) {
+    pdl_launch();
+    const int t = blockIdx.x;
+    const int n_heads = p.nh + (p.pool ? p.nkv * MAPS : 0), qd = p.nh * p.hd, kd = p.pool ? p.nkv * MAPS * p.hd : 0;
+    const int half = p.rot / 2, turns = p.interleaved ? p.rot / 8 : half / 8, passes = (p.hd - p.rot) / 8;
+    const int n_turn = n_heads * turns, n_pass = n_heads * passes, n_val = p.pool ? p.nkv * p.vd / 8 : 0;
+    const TS* row = (const TS*)p.src + (size_t)t * p.src_stride;
+    const int pos = p.positions[t];
+    long long k_base = -1, v_base = -1;
+    if (p.pool) {
+        const int req = p.row_req[t];
+        const int page = p.block_table[(size_t)req * p.max_pages + pos / p.page_size];
+        if (page < 0 || page >= p.num_pages) {
+            if (p.status && threadIdx.x == 0) atomicOr(p.status, BG_STATUS_BAD_PAGE);
+        } else {
+            const size_t page_elems = (size_t)p.nkv * p.page_size * (p.ks + p.vs);
+            const int slot = pos % p.page_size;
+            k_base = (long long)((size_t)page * page_elems + (size_t)slot * p.ks);
+            v_base = (long long)((size_t)page * page_elems + (size_t)p.nkv * p.page_size * p.ks + (size_t)slot * p.vs);
+        }
+    }
+    TQ* qo = (TQ*)p.q_out + (size_t)t * p.q_stride;
+    TC* pool = (TC*)p.pool;
+    auto fetch = [&](int at, float (&v)[8]) {
+        load8(row + at, v);
+        for (int pp = 1; pp < p.parts; ++pp) {
+            float u[8];
+            load8(row + (size_t)pp * p.part_stride + at, u);
+#pragma unroll
+            for (int e = 0; e < 8; ++e) v[e] += u[e];
+        }
+    };
+    auto put = [&](int h, int f, const float (&v)[8]) {        // feature f of (map) head h: queries first, then keys
+        if (h < p.nh) store8(qo + (size_t)h * p.qs + (h % MAPS) * map_shift(p) + f, v);
+        else if (k_base >= 0) {
+            const int k = h - p.nh;
+            store8(pool + k_base + (size_t)(k / MAPS) * p.page_size * p.ks + (k % MAPS) * map_width(p) + f, v);
+        }
+    };
+    pdl_wait();
+    const float* cs = p.cos_sin ? p.cos_sin + (size_t)t * half * 2 : nullptr;
+    for (int i = threadIdx.x; i < n_turn + n_pass + n_val; i += blockDim.x) {
+        if (i < n_turn) {
+            const int h = i / turns, c = 8 * (i - h * turns);
+            float a[8];
+            fetch(h * p.hd + c, a);
+            if (p.interleaved) {
+#pragma unroll
+                for (int k = 0; k < 4; ++k) {
+                    const float u = a[2 * k], w = a[2 * k + 1];
+                    const float cc = cs[2 * (c / 2 + k)], sn = cs[2 * (c / 2 + k) + 1];
+                    a[2 * k] = u * cc - w * sn;
+                    a[2 * k + 1] = w * cc + u * sn;
+                }
+                put(h, c, a);
+            } else {
+                float b[8], f[16];
+                fetch(h * p.hd + c + half, b);
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float4 q = reinterpret_cast<const float4*>(cs + 2 * c)[e];
+                    f[4 * e] = q.x; f[4 * e + 1] = q.y; f[4 * e + 2] = q.z; f[4 * e + 3] = q.w;
+                }
+#pragma unroll
+                for (int e = 0; e < 8; ++e) {
+                    const float u = a[e], w = b[e];
+                    a[e] = u * f[2 * e] - w * f[2 * e + 1];
+                    b[e] = w * f[2 * e] + u * f[2 * e + 1];
+                }
+                put(h, c, a);
+                put(h, c + half, b);
+            }
+        } else if (i < n_turn + n_pass) {
+            const int j = i - n_turn, h = j / passes, f = p.rot + 8 * (j - h * passes);
+            float a[8];
+            fetch(h * p.hd + f, a);
+            put(h, f, a);
+        } else if (v_base >= 0) {
+            const int j = 8 * (i - n_turn - n_pass), h = j / p.vd, f = j - h * p.vd;
+            float a[8];
+            fetch(qd + kd + j, a);
+            store8(pool + v_base + (size_t)h * p.page_size * p.vs + f, a);
+        }
+    }
+    const float zero[8] = {0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f, 0.0f};
+    const int qpad = (p.qs - p.hd) / 8, kpad = (map_width(p) - p.hd) / 8, vpad = (p.vs - p.vd) / 8;
+    for (int i = threadIdx.x; i < p.nh * qpad; i += blockDim.x) {
+        const int h = i / qpad, r = 8 * (i - h * qpad);
+        store8(qo + (size_t)h * p.qs + (r < (h % MAPS) * map_shift(p) ? r : r + p.hd), zero);
+    }
+    if (k_base >= 0)
+        for (int i = threadIdx.x; i < p.nkv * MAPS * kpad; i += blockDim.x) {
+            const int h = i / kpad;
+            store8(pool + k_base + (size_t)(h / MAPS) * p.page_size * p.ks + (h % MAPS) * map_width(p) + p.hd + 8 * (i % kpad), zero);
+        }
+    if (v_base >= 0)
+        for (int i = threadIdx.x; i < p.nkv * vpad; i += blockDim.x)
+            store8(pool + v_base + (size_t)(i / vpad) * p.page_size * p.vs + p.vd + 8 * (i % vpad), zero);
+}
+
 // out[t][j] = src[t][(j / vd) * head_stride + j % vd] * sigmoid(gate[t][col0 + j / gate_per]) for j < n: the gate is a column
 // range of a wider row (or of its partial sums), one number per feature (gate_per 1) or one per head (gate_per = vd); the
 // source's heads may be stored wider than they are (out == src when they are not).
@@ -327,6 +432,16 @@ static int qk_norm_rope_launch_maps(const QkMapsParams& p, int T, cudaStream_t s
                      p.qs % 8 == 0 && p.ks % 8 == 0 && p.kw % 8 == 0 && p.q_shift % 8 == 0 && p.vs % 8 == 0 && p.src_stride % 8 == 0 && p.part_stride % 8 == 0 &&
                      p.q_stride % 8 == 0 && (uintptr_t)p.src % 16 == 0 && (uintptr_t)p.q_out % 16 == 0 && (uintptr_t)p.pool % 16 == 0 &&
                      (!p.wq || ((uintptr_t)p.wq % 16 == 0 && (uintptr_t)p.wk % 16 == 0)) && width > 0;
+    if (vec && !p.wq && (!p.cos_sin || (uintptr_t)p.cos_sin % 16 == 0)) {
+        const int n_heads = p.nh + (p.pool ? p.nkv * MAPS : 0);
+        const int items = n_heads * ((p.interleaved ? p.rot : p.rot / 2) + p.hd - p.rot) / 8 + (p.pool ? p.nkv * p.vd / 8 : 0);
+        int threads = (items + 31) / 32 * 32;
+        if (threads > 256) threads = (items / ((items + 255) / 256) + 32) / 32 * 32;       // rounds of equal length
+        if (threads > 256) threads = 256;
+        launch(rope_append_vec8_kernel<TS, TQ, TC, MAPS>, dim3(T), dim3(threads), 0, stream, static_cast<const typename QkParamsOf<MAPS>::type&>(p));
+        BG_LAUNCH_CHECK();
+        return BG_OK;
+    }
     auto kern = vec ? qk_norm_rope_append_vec8_kernel<TS, TQ, TC, MAPS> : qk_norm_rope_append_kernel<TS, TQ, TC, MAPS>;
     const size_t smem = (size_t)(p.nh * p.hd + (p.pool ? p.nkv * MAPS * p.hd : 0)) * sizeof(float);
     if (smem > 200 * 1024) return BG_ERR_SHAPE;

@@ -455,10 +455,31 @@ def dinatar_config(width, heads, layers, vocab=32768, max_positions=32768):
                         "mlp": {"kind": "dense", "ff": 4 * width} if i % 3 == 0 else moe} for i in range(n)]}
 
 
+# The Fanitar decoder beside another design at equal layer sizes (--design fanitar): layers in the order differential attention,
+# differential attention, latent attention, ...: heads that are pairs of maps of 64 features over values of 128, whole maps
+# rotated, every position visible; attention through a latent of 512 features (width / 4 up to width 2048) with queries through one
+# of width / 2, heads of 128, a window of 1,024, learned sinks and a gate per feature.  Every layer has a gated feed-forward of the
+# Qwen2 layer's weights and four norms.  Two of the layers are passed twice, so that the number of layer runs is the other
+# model's number of layers.  Random weights.
+def fanitar_config(width, heads, layers, vocab=32768):
+    kv = max(1, heads // 4 if heads % 4 == 0 and heads > 12 else heads // 6)
+    att = {"heads": heads, "kv_heads": kv, "dim": 64, "vdim": 128, "scale": 64 ** -0.5, "diff": 0.8, "rot": {"base": 500000.0, "dims": 64}}
+    lat = {"heads": heads, "dim": 128, "vdim": 128, "q_rank": width // 2, "kv_rank": width // 4 if width <= 2048 else 512,
+           "scale": 128 ** -0.5, "mask": {"size": 1024}}
+    ff = {"kind": "dense", "ff": (8 * width // 3) // 128 * 128, "limit": 7.0}
+    kinds = [("attention", att), ("attention", att), ("latent_attention", lat)]
+    k = 2 if layers >= 5 else 1                    # layers passed twice
+    n = layers - k
+    return {"architecture": "Fanitar", "vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "embedding": {"scale": float(width) ** 0.5},
+            "logit_scale": 0.5, "loop": {"start": 1, "stop": 1 + k, "times": 2},
+            "layers": [{"type": kinds[i % 3][0], "mixer": kinds[i % 3][1], "mlp": ff} for i in range(n)]}
+
+
 DESIGN_SIZES = {"1536": (1536, 12, 8), "4096": (4096, 32, 4)}      # width -> (width, heads, layers)
 DESIGNS = {"sukisun": lambda w, h, l: sukisun_config(w, h, l), "nadilorn": lambda w, h, l: nadilorn_config(w, h, l),
            "nadilorn-v64": lambda w, h, l: nadilorn_config(w, h, l, vdim=64), "sofudra": lambda w, h, l: sofudra_config(w, h, l),
-           "tuzupel": lambda w, h, l: tuzupel_config(w, h, l), "dinatar": lambda w, h, l: dinatar_config(w, h, l)}
+           "tuzupel": lambda w, h, l: tuzupel_config(w, h, l), "dinatar": lambda w, h, l: dinatar_config(w, h, l),
+           "fanitar": lambda w, h, l: fanitar_config(w, h, l)}
 BESIDE = dict(DESIGNS, qwen2=lambda w, h, l: qwen2_like(w, h, l))
 
 

@@ -29,6 +29,13 @@ import torch
 SLOPE = 1.702          # of the sigmoid inside the gated activation
 
 
+def exactly(x: torch.Tensor) -> torch.Tensor:
+    """The default of `low`: nothing is rounded.  (`forward` with another `low` passes through it what an engine in a rounded number
+    format keeps in that format, which tells how far rounding alone moves the logits.)"""
+    return x
+
+
+
 def read_folder(folder: str, dtype: torch.dtype = torch.float64):
     from safetensors import safe_open
 
@@ -55,13 +62,13 @@ def turn_halves(x: torch.Tensor, base: float, dims: int) -> torch.Tensor:
     position * base^(-2i/dims); features from dims on pass."""
     half = dims // 2
     out = x.clone()
-    for t in range(x.shape[0]):
-        for i in range(half):
-            a = t * base ** (-2.0 * i / dims)
-            c, s = math.cos(a), math.sin(a)
-            u, v = x[t, ..., i], x[t, ..., i + half]
-            out[t, ..., i] = u * c - v * s
-            out[t, ..., i + half] = v * c + u * s
+    for i in range(half):
+        f = base ** (-2.0 * i / dims)
+        c = torch.tensor([math.cos(t * f) for t in range(x.shape[0])], dtype=x.dtype).view(-1, *[1] * (x.dim() - 2))
+        s = torch.tensor([math.sin(t * f) for t in range(x.shape[0])], dtype=x.dtype).view(-1, *[1] * (x.dim() - 2))
+        u, v = x[..., i], x[..., i + half]
+        out[..., i] = u * c - v * s
+        out[..., i + half] = v * c + u * s
     return out
 
 
@@ -72,10 +79,10 @@ def visible(t: int, size: Optional[int]) -> List[int]:
 
 
 def plain_softmax_weights(s: torch.Tensor, sink: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """exp(s_j) / (sum_j exp(s_j) + exp(sink)), the last only where given."""
-    top = s.max() if sink is None else torch.maximum(s.max(), sink)
+    """exp(s_j) / (sum_j exp(s_j) + exp(sink)) over the first index, the last term only where given."""
+    top = s.amax(0) if sink is None else torch.maximum(s.amax(0), sink)
     e = torch.exp(s - top)
-    z = e.sum() + (0.0 if sink is None else torch.exp(sink - top))
+    z = e.sum(0) + (0.0 if sink is None else torch.exp(sink - top))
     return e / z
 
 
@@ -84,14 +91,14 @@ def two_maps(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, scale: float):
     map, over the same values; query head h reads kv head h // (H / G)."""
     T, H = q.shape[:2]
     G = k.shape[1]
+    reads = [h // (H // G) for h in range(H)]
+    k, v = k[:, reads], v[:, reads]                                     # what each query head reads
     out = [torch.zeros((T, H, v.shape[2]), dtype=q.dtype) for _ in range(2)]
     for t in range(T):
         keys = visible(t, None)
-        for h in range(H):
-            g = h // (H // G)
-            for c in range(2):
-                p = plain_softmax_weights((k[keys, g, c] @ q[t, h, c]) * scale)
-                out[c][t, h] = p @ v[keys, g]
+        for c in range(2):
+            p = plain_softmax_weights((k[keys, :, c] * q[t, :, c]).sum(-1) * scale)             # [keys, H]
+            out[c][t] = (p[:, :, None] * v[keys]).sum(0)
     return out
 
 
@@ -99,7 +106,7 @@ def difference_weight(w: Dict[str, torch.Tensor], diff: float) -> torch.Tensor:
     return torch.exp((w["lq1"] * w["lk1"]).sum()) - torch.exp((w["lq2"] * w["lk2"]).sum()) + diff
 
 
-def differential_mixer(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float) -> torch.Tensor:
+def differential_mixer(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float, low: Callable = exactly) -> torch.Tensor:
     T = h.shape[0]
     H, G, n, nv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
     q = (h @ w["q"].T + w["q.b"]).view(T, H, 2, n)
@@ -108,25 +115,24 @@ def differential_mixer(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps
     rot = m.get("rot")
     if rot is not None and rot["dims"] > 0:
         q, k = turn_halves(q, rot["base"], rot["dims"]), turn_halves(k, rot["base"], rot["dims"])
-    a1, a2 = two_maps(q, k, v, m["scale"])
+    a1, a2 = two_maps(low(q), low(k), low(v), m["scale"])
     o = rms_unit(a1 - difference_weight(w, m["diff"]) * a2, eps) * (1.0 - m["diff"])
-    return o.reshape(T, H * nv) @ w["o"].T
+    return low(o).reshape(T, H * nv) @ w["o"].T
 
 
-def latent_mixer(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float) -> torch.Tensor:
+def latent_mixer(h: torch.Tensor, w: Dict[str, torch.Tensor], m: dict, eps: float, low: Callable = exactly) -> torch.Tensor:
     T = h.shape[0]
     H, n, nv = m["heads"], m["dim"], m["vdim"]
-    q = (rms_norm(h @ w["dq"].T, w["dq.norm"], eps) @ w["uq"].T).view(T, H, n)
-    c = rms_norm(h @ w["dkv"].T, w["dkv.norm"], eps)
-    k, v = (c @ w["uk"].T).view(T, H, n), (c @ w["uv"].T).view(T, H, nv)
+    q = low(low(rms_norm(h @ w["dq"].T, w["dq.norm"], eps)) @ w["uq"].T).view(T, H, n)
+    c = low(rms_norm(h @ w["dkv"].T, w["dkv.norm"], eps))
+    k, v = low(c @ w["uk"].T).view(T, H, n), low(c @ w["uv"].T).view(T, H, nv)
     size = (m.get("mask") or {}).get("size")
     o = torch.zeros((T, H, nv), dtype=h.dtype)
     for t in range(T):
         keys = visible(t, size)
-        for hh in range(H):
-            p = plain_softmax_weights((k[keys, hh] @ q[t, hh]) * m["scale"], w["sink"][hh])
-            o[t, hh] = p @ v[keys, hh]
-    return (o.reshape(T, H * nv) * torch.sigmoid(h @ w["g"].T)) @ w["o"].T
+        p = plain_softmax_weights((k[keys] * q[t]).sum(-1) * m["scale"], w["sink"])             # [keys, H]
+        o[t] = (p[:, :, None] * v[keys]).sum(0)
+    return low(o.reshape(T, H * nv) * torch.sigmoid(h @ w["g"].T)) @ w["o"].T
 
 
 # ----------------------------------------------------------------------------- feed-forward
@@ -137,10 +143,10 @@ def cut_gate(g: torch.Tensor, u: torch.Tensor, limit: float) -> torch.Tensor:
     return g * torch.sigmoid(SLOPE * g) * (u + 1.0)
 
 
-def feed_forward(h: torch.Tensor, w: Dict[str, torch.Tensor], f: dict) -> torch.Tensor:
+def feed_forward(h: torch.Tensor, w: Dict[str, torch.Tensor], f: dict, low: Callable = exactly) -> torch.Tensor:
     if f["kind"] != "dense":
         raise ValueError(f["kind"])
-    return cut_gate(h @ w["gate"].T, h @ w["up"].T, f["limit"]) @ w["down"].T
+    return low(cut_gate(low(h @ w["gate"].T), low(h @ w["up"].T), f["limit"])) @ w["down"].T
 
 
 # ----------------------------------------------------------------------------- the model
@@ -148,11 +154,11 @@ def sub(weights: Dict[str, torch.Tensor], prefix: str) -> Dict[str, torch.Tensor
     return {k[len(prefix):]: v for k, v in weights.items() if k.startswith(prefix)}
 
 
-def mixer_of(kind: str, h, w, m, eps):
+def mixer_of(kind: str, h, w, m, eps, low=exactly):
     if kind == "attention":
-        return differential_mixer(h, w, m, eps)
+        return differential_mixer(h, w, m, eps, low)
     if kind == "latent_attention":
-        return latent_mixer(h, w, m, eps)
+        return latent_mixer(h, w, m, eps, low)
     raise ValueError(kind)
 
 
@@ -167,7 +173,8 @@ def run_order(n_layers: int, loop: Optional[dict]):
     return out + [(i, None) for i in range(hi, n_layers)]
 
 
-def forward(cfg: dict, weights: Dict[str, torch.Tensor], tokens: Sequence[int], tap: Optional[Callable] = None) -> torch.Tensor:
+def forward(cfg: dict, weights: Dict[str, torch.Tensor], tokens: Sequence[int], tap: Optional[Callable] = None,
+            low: Callable = exactly) -> torch.Tensor:
     """Logits [T, vocab] of a whole sequence from position 0.  `tap(run, rows)` gets the stream behind every layer run."""
     eps = cfg["norm"]["eps"]
     scale = (cfg.get("embedding") or {}).get("scale", 1.0)
@@ -179,12 +186,12 @@ def forward(cfg: dict, weights: Dict[str, torch.Tensor], tokens: Sequence[int], 
             if begins > 0:
                 x = x + e
             x = x + weights["loop.step"][begins]
-        y = mixer_of(layer["type"], rms_norm(x, weights[p + "norm1"], eps), sub(weights, p + "mix."), layer["mixer"], eps)
-        x = x + rms_norm(y, weights[p + "norm1b"], eps)
+        y = mixer_of(layer["type"], low(rms_norm(x, weights[p + "norm1"], eps)), sub(weights, p + "mix."), layer["mixer"], eps, low)
+        x = x + rms_norm(low(y), weights[p + "norm1b"], eps)
         if layer.get("mlp") is not None:
-            y = feed_forward(rms_norm(x, weights[p + "norm2"], eps), sub(weights, p + "mlp."), layer["mlp"])
-            x = x + rms_norm(y, weights[p + "norm2b"], eps)
+            y = feed_forward(low(rms_norm(x, weights[p + "norm2"], eps)), sub(weights, p + "mlp."), layer["mlp"], low)
+            x = x + rms_norm(low(y), weights[p + "norm2b"], eps)
         if tap is not None:
             tap(ri, x)
-    x = rms_norm(x, weights["final.norm"], eps)
+    x = low(rms_norm(x, weights["final.norm"], eps))
     return (x @ weights["head"].T) * cfg.get("logit_scale", 1.0)
