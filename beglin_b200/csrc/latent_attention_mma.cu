@@ -181,6 +181,7 @@ latent_attention_mma_kernel(LatentMmaParams p) {
             fetch(ti + 1, (ti + 1) & 1);
             lm_cp_async_wait<1>();
         } else {
+            if (p.stages == 1 && ti > 0) fetch(ti, 0);             // one tile at a time (the last one has been read)
             lm_cp_async_wait<0>();
         }
         __syncthreads();

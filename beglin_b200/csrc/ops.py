@@ -1151,7 +1151,7 @@ def gemm_f32_nt_batched(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> 
     strides with unit inner stride.  CUDA cores only."""
     _cuda(a, w, out)
     for t in (a, w, out):
-        if t.dtype != torch.float32 or t.dim() != 3 or t.stride(2) != 1:
+        if t.dtype != torch.float32 or t.dim() != 3 or (t.stride(2) != 1 and t.shape[2] != 1):
             raise KernelError("gemm_f32_nt_batched takes float32 [B, rows, cols] views with unit inner stride")
     B, M, K = a.shape
     N = w.shape[1]

@@ -235,6 +235,23 @@ def test_a_long_portion_replayed_as_a_graph(model_root, dtype):
                 assert rel_err(row, full[p]) < tol * float(full.abs().max() / full[p].abs().max()), (rid, p)
 
 
+@pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
+def test_large_heads_and_a_long_latent(model_root, dtype):
+    """Maps of 128 features over values of 256 and maps of 96 (sizes that no tensor-core kernel takes), seventeen query heads on one
+    kv head (more than the decoding kernel takes, while portions run on the tensor cores), a latent of 512 features with few heads:
+    whole, with single tokens at the end, and in portions."""
+    cfg = config(400, 256, 1e-5, [layer(att(4, 2, 128, 256, 0.09, 0.4, rot=(128, 1e5)), dense(512, 2.0)),
+                                  layer(lat(5, 96, 128, 160, 512, 0.1, window=301), dense(320, 1.0)),
+                                  layer(att(17, 1, 32, 64, 0.18, 0.2, rot=(32, 1e4)), dense(128, 1.5)),
+                                  layer(att(3, 3, 96, 64, 0.1, 0.5, rot=(50, 1e4)))], embed_scale=2.0, loop=(1, 4, 2))
+    folder = make_model(model_root, "large", seed=5, dtype=stored(dtype), config_json=cfg)
+    reqs = {"a": seeded_ids(370, 400, 1), "b": seeded_ids(66, 400, 2)}
+    for steps in (rl.whole(reqs), rl.last_one_by_one(reqs, tail=20), rl.portions(reqs)):
+        eng = engine_for(folder, dtype, 384, 64, kv_split=256)
+        check_against_plain(rl.run_in_process(eng, steps), folder, reqs, TOL_F32 if dtype == "float32" else TOL_BF16,
+                            None if dtype == "float32" else torch.bfloat16)
+
+
 def test_a_run_of_layers_passed_three_times_has_caches_of_its_own(model_root):
     """Three passes over a run that holds both kinds of mixer and reaches from the first layer to the last: as many cache stages as
     layer runs, and the logits of the plain implementation, in one step and cut; the learned rows of the passes and the embedded

@@ -392,6 +392,65 @@ def test_both_latents_normed_and_the_cached_row_appended(q_rank, rank, rot, rot_
     assert int(torch.isnan(pool.float()).all(-1).sum()) == 10 * page - T
 
 
+LATENT = [  # heads, latent, rotated part, page, window, positions, queries: rows of 16, 32 and 64 in a CTA, one and two tiles of keys in it
+    (5, 512, 0, 16, 301, 700, 1), (12, 384, 0, 64, 0, 900, 1), (3, 384, 64, 64, 130, 500, 1), (16, 448, 0, 32, 0, 700, 1),
+    (2, 512, 64, 64, 0, 600, 7), (5, 96, 0, 16, 0, 400, 60), (40, 256, 0, 64, 72, 300, 3), (6, 128, 32, 8, 0, 1100, 1), (1, 32, 0, 64, 3, 70, 70),
+]
+
+
+@pytest.mark.parametrize("case", LATENT, ids=["-".join(map(str, c)) for c in LATENT])
+@pytest.mark.parametrize("kernel", ["mma", "cuda_cores", "float"])
+@pytest.mark.parametrize("sinks", [True, False])
+def test_latent_attention_over_many_tiles(case, kernel, sinks):
+    """The kernels that score against the cached rows themselves, over ranges of several tiles of keys, with keys that stand out
+    in every tile so that a tile taken twice or left out shows; NaN in all that may not be read."""
+    H, rank, rot, page, window, S, T = case
+    o = ops()
+    dtype = torch.float32 if kernel == "float" else torch.bfloat16
+    g = torch.Generator().manual_seed(S + H)
+    width, first = rank + rot, S - T
+    rows = torch.randn(S, width, generator=g).to(dtype)
+    q_lat = torch.randn(H, T, rank, generator=g)
+    q_raw = torch.randn(T, H * (8 + rot), generator=g).to(dtype)
+    for p in range(7, S, 50):                                   # every head looks for some of these
+        h = p % H
+        qq = torch.cat([q_lat[h, 0], q_raw.view(T, H, 8 + rot)[0, h, 8:].float()])
+        rows[p] = (1.5 * qq * math.sqrt(width) / qq.norm()).to(dtype)
+    q_lat = 0.3 * q_lat + q_lat[:, :1]
+    sink = 2.0 * torch.randn(H, generator=g) + 2.0 if sinks else None
+    scale = 2.0 / math.sqrt(width)
+    lo = max(0, first - window + 1) if window else 0
+    n_pages = -(-S // page)
+    order = torch.randperm(n_pages + 2, generator=g).tolist()
+    pool = torch.full((n_pages + 2, page, width), NAN).to(dtype)
+    table = torch.full((1, n_pages + 2), -1, dtype=torch.int32)
+    for i in range(n_pages):
+        if (i + 1) * page > lo:
+            table[0, i] = order[i]
+            pool[order[i], :min(page, S - i * page)] = rows[i * page:i * page + min(page, S - i * page)]
+    r, tile = o.latent_attention_plan(rank, rot)
+    stages = 0
+    if kernel == "mma":
+        r, stages = o.latent_attention_mma_plan(rank, rot)
+    hc = min(H, r)
+    bq = 1 if T == 1 else max(1, r // hc)
+    qblk = i32([[0, t, min(bq, T - t)] for t in range(0, T, bq)])
+    out = torch.full((H, T, rank), NAN, dtype=dtype, device=DEV)
+    status = o.new_status(DEV)
+    o.latent_attention(dev(q_lat), dev(q_raw), 8, rot, 0, None, dev(pool), dev(table), i32(list(range(first, S))), qblk, qblk.shape[0],
+                       S - 1, bq, hc, tile, 256, scale, out, status, mma_stages=stages, window=window,
+                       sink_weight=None if sink is None else dev(sink))
+    o.raise_on_status(status)
+    full = torch.cat([q_lat.double().transpose(0, 1), q_raw.double().view(T, H, 8 + rot)[:, :, 8:]], -1)
+    k = rows.double()
+    want = torch.zeros(H, T, rank, dtype=torch.float64)
+    for t in range(T):
+        keys = plain.visible(first + t, window or None)
+        p = plain.plain_softmax_weights((k[keys][:, None, :] * full[t]).sum(-1) * scale, None if sink is None else sink.double())
+        want[:, t] = (p[:, :, None] * k[keys][:, None, :rank]).sum(0)
+    assert rel_err(out, want) < (2e-5 if kernel == "float" else 2e-2)
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 @pytest.mark.parametrize("dim,rank", [(64, 64), (24, 40)])
 def test_a_key_inside_and_outside_the_window_and_the_sink(tmp_path, dtype, dim, rank):

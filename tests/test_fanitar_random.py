@@ -46,7 +46,7 @@ def random_config(case: int, even: bool = False):
     return cfg, rng.choice([4, 8, 16, 32, 64])
 
 
-@pytest.mark.parametrize("case", range(14))
+@pytest.mark.parametrize("case", list(range(14)) + [15, 34])      # 15 and 34: heads, or a latent, of a single feature
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_random_configuration(model_root, case, dtype):
     cfg, page = random_config(case, even=(dtype == "bfloat16"))
@@ -58,7 +58,7 @@ def test_random_configuration(model_root, case, dtype):
     results = {}
     tol = TOL_F32 if dtype == "float32" else TOL_BF16
     for way, (steps, tokens) in {"whole": (rl.whole(reqs), 192), "mixed": (mixed_steps, peak)}.items():
-        eng = Engine.from_folder(folder, dtype=dtype, max_tokens=max(tokens, page), page_size=page, max_requests=4, kv_split=64)
+        eng = Engine.from_folder(folder, dtype=dtype, max_tokens=max(tokens, page), page_size=page, max_requests=4, kv_split=64 if case % 2 else 256)
         poison(eng)
         results[way] = rl.run_in_process(eng, steps)
         eng.cache.check()
