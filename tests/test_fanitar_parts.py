@@ -395,6 +395,7 @@ def test_both_latents_normed_and_the_cached_row_appended(q_rank, rank, rot, rot_
 LATENT = [  # heads, latent, rotated part, page, window, positions, queries: rows of 16, 32 and 64 in a CTA, one and two tiles of keys in it
     (5, 512, 0, 16, 301, 700, 1), (12, 384, 0, 64, 0, 900, 1), (3, 384, 64, 64, 130, 500, 1), (16, 448, 0, 32, 0, 700, 1),
     (2, 512, 64, 64, 0, 600, 7), (5, 96, 0, 16, 0, 400, 60), (40, 256, 0, 64, 72, 300, 3), (6, 128, 32, 8, 0, 1100, 1), (1, 32, 0, 64, 3, 70, 70),
+    (5, 448, 0, 16, 301, 700, 180),        # (every row a CTA of its own: more CTAs than leave room for two tiles in each)
 ]
 
 
@@ -433,7 +434,7 @@ def test_latent_attention_over_many_tiles(case, kernel, sinks):
     if kernel == "mma":
         r, stages = o.latent_attention_mma_plan(rank, rot)
     hc = min(H, r)
-    bq = 1 if T == 1 else max(1, r // hc)
+    bq = 1 if T == 1 or T == 180 else max(1, r // hc)
     qblk = i32([[0, t, min(bq, T - t)] for t in range(0, T, bq)])
     out = torch.full((H, T, rank), NAN, dtype=dtype, device=DEV)
     status = o.new_status(DEV)
