@@ -32,7 +32,7 @@ APPEND = [  # query heads, kv heads, dim, vdim, rotated, interleaved, stored map
     (3, 1, 10, 7, 6, False, 10, 7, 4),
     (4, 2, 5, 13, 0, False, 5, 13, 8),
     (2, 2, 12, 24, 12, True, 32, 64, 16),
-    (4, 2, 48, 96, 48, False, 64, 128, 16),
+    (4, 1, 40, 88, 32, False, 64, 128, 16),
     (6, 2, 64, 128, 32, False, 64, 128, 64),
     (2, 1, 24, 40, 16, True, 32, 64, 8),
     (12, 2, 64, 128, 64, False, 64, 128, 64),
@@ -164,10 +164,10 @@ CASES = [  # kernel, dtype, query heads, kv heads, dim, vdim, stored map, stored
     ("generic", torch.float32, 4, 1, 130, 200, 130, 200, 16, 0, 130, 9),
     ("generic", torch.float32, 1, 1, 1, 1, 1, 1, 4, 0, 33, 33),
     ("generic", torch.bfloat16, 4, 2, 32, 16, 32, 16, 16, 33, 200, 60),
-    ("generic", torch.bfloat16, 4, 2, 48, 96, 64, 128, 16, 0, 200, 60),
+    ("generic", torch.bfloat16, 4, 1, 40, 88, 64, 128, 16, 0, 200, 60),
     ("tc_rows", torch.bfloat16, 4, 2, 32, 64, 32, 64, 16, 0, 300, 300),
     ("tc_rows", torch.bfloat16, 2, 1, 64, 128, 64, 128, 64, 0, 500, 200),
-    ("tc_rows", torch.bfloat16, 4, 2, 48, 96, 64, 128, 16, 0, 140, 140),
+    ("tc_rows", torch.bfloat16, 6, 2, 40, 104, 64, 128, 16, 0, 140, 140),
     ("tc_rows", torch.bfloat16, 6, 1, 24, 40, 32, 64, 64, 72, 1100, 900),
     ("tc_rows", torch.bfloat16, 3, 3, 40, 21, 64, 128, 8, 0, 333, 70),
     ("tc_rows", torch.bfloat16, 1, 1, 64, 128, 64, 128, 32, 0, 63, 63),
@@ -175,7 +175,7 @@ CASES = [  # kernel, dtype, query heads, kv heads, dim, vdim, stored map, stored
     ("tc_rows", torch.bfloat16, 5, 1, 64, 100, 64, 128, 4, 130, 420, 333),
     ("mma_keys", torch.bfloat16, 4, 2, 32, 64, 32, 64, 16, 0, 700, 1),
     ("mma_keys", torch.bfloat16, 2, 1, 64, 128, 64, 128, 64, 300, 1500, 1),
-    ("mma_keys", torch.bfloat16, 16, 2, 48, 96, 64, 128, 64, 0, 2500, 1),
+    ("mma_keys", torch.bfloat16, 16, 2, 56, 88, 64, 128, 64, 0, 2500, 1),
     ("mma_keys", torch.bfloat16, 4, 1, 24, 33, 32, 64, 48, 600, 900, 1),
     ("mma_keys", torch.bfloat16, 4, 4, 64, 128, 64, 128, 32, 0, 1, 1),
 ]
@@ -360,7 +360,7 @@ def test_a_gate_for_every_feature_of_head_major_results(H, T, vd, dtype, gate_ty
     assert rel_err(out, want) < (2e-6 if dtype == torch.float32 else 5e-3)
 
 
-@pytest.mark.parametrize("q_rank,rank,rot,rot_dims", [(80, 96, 0, 0), (768, 384, 0, 0), (0, 512, 64, 64), (12, 20, 6, 4), (11, 17, 0, 0),
+@pytest.mark.parametrize("q_rank,rank,rot,rot_dims", [(72, 104, 0, 0), (768, 384, 0, 0), (0, 512, 64, 64), (12, 20, 6, 4), (11, 17, 0, 0),
                                                       (2048, 512, 64, 32)])
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_both_latents_normed_and_the_cached_row_appended(q_rank, rank, rot, rot_dims, dtype):
@@ -394,7 +394,7 @@ def test_both_latents_normed_and_the_cached_row_appended(q_rank, rank, rot, rot_
 
 LATENT = [  # heads, latent, rotated part, page, window, positions, queries: rows of 16, 32 and 64 in a CTA, one and two tiles of keys in it
     (5, 512, 0, 16, 301, 700, 1), (12, 384, 0, 64, 0, 900, 1), (3, 384, 64, 64, 130, 500, 1), (16, 448, 0, 32, 0, 700, 1),
-    (2, 512, 64, 64, 0, 600, 7), (5, 96, 0, 16, 0, 400, 60), (40, 256, 0, 64, 72, 300, 3), (6, 128, 32, 8, 0, 1100, 1), (1, 32, 0, 64, 3, 70, 70),
+    (2, 512, 64, 64, 0, 600, 7), (5, 160, 0, 16, 0, 400, 60), (40, 256, 0, 64, 72, 300, 3), (6, 128, 32, 8, 0, 1100, 1), (1, 32, 0, 64, 3, 70, 70),
     (5, 448, 0, 16, 301, 700, 180),        # (every row a CTA of its own: more CTAs than leave room for two tiles in each)
 ]
 
